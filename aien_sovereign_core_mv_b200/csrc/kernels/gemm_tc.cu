@@ -220,9 +220,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 // leaves at once) and is multiplied by rows group * N + n0 .. of W.  The roles, the ring and the
 // bounded waits are those of the first form with 128 rows of A.  tile_group comes from a kernel
 // ahead in the stream, so nothing is requested before griddepcontrol.wait here.
-//   EPI 0: store;  EPI 2 / 3: the gelu in its erf / tanh form, then store.
+//   EPI 0: store;  EPI 1: silu(gate) * up over columns interleaved in runs of 8;  EPI 2 / 3: the gelu in its erf / tanh
+//   form, then store;  EPI 4: the square of relu.
 //   row_dest != nullptr: row r of the result goes to row row_dest[r] of out (-1: nowhere) times
-//   row_scale[r]: the weighted outputs of routed experts, back in token order.
+//   row_scale[r] (null: times one): the weighted outputs of routed experts, back in token order.
+//   row_scale without row_dest: the products of row r are multiplied by row_scale[r] before the activation (a weight
+//   on the expert's input).
 // Columns of a tile beyond N belong to the next group's rows of W; they are computed and not stored.
 template <int EPI, typename TC>
 __global__ void __launch_bounds__(192)
@@ -301,15 +304,18 @@ gemm_tc_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_c
         const int row = m0 + quarter * 32 + lane;
         int dest = row;
         float rs = 1.0f;
-        if (row_dest != nullptr) {
-            dest = __ldcg(row_dest + row);
-            rs = __ldcg(row_scale + row);
-        }
+        if (row_dest != nullptr) dest = __ldcg(row_dest + row);
+        if (row_scale != nullptr) rs = __ldcg(row_scale + row);
+        const bool scale_first = row_dest == nullptr && row_scale != nullptr;
 #pragma unroll 1
         for (int c0 = 0; c0 < BN && n0 + c0 < N; c0 += 32) {
             uint32_t r[32];
             tmem_ld32(tmem_acc + ((uint32_t)(quarter * 32) << 16) + (uint32_t)c0, r);
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+            if (scale_first) {
+#pragma unroll
+                for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * rs);
+            }
             if (EPI == 2) {
 #pragma unroll
                 for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(tc_gelu_erf(__uint_as_float(r[j])));
@@ -320,11 +326,11 @@ gemm_tc_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_c
 #pragma unroll
                 for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(tc_relu2(__uint_as_float(r[j])));
             }
-            if (row_dest != nullptr) {
+            if (row_dest != nullptr && row_scale != nullptr) {
 #pragma unroll
                 for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * rs);
             }
-            if (dest >= 0) tc_store_chunk<0, TC>(r, out, ldc, dest, n0, c0, N);
+            if (dest >= 0) tc_store_chunk<(EPI == 1 ? 1 : 0), TC>(r, out, ldc, dest, n0, c0, N);
         }
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -888,20 +894,22 @@ AIEN_API int aien_gemm_tc(const void* A, long lda, const void* W, long ldw, void
 }
 
 // Grouped product (see gemm_tc_grouped_kernel): A [tiles * 128, K] sorted by group, W [groups * N, K].
-// epilogue 0 store, 2 erf gelu, 3 tanh gelu.  row_dest / row_scale (both or neither): scatter rows of
-// the result, scaled, into out (float32).
+// epilogue 0 store, 1 silu(gate) * up (N counts gate and up rows, interleaved in runs of 8; out has N / 2 columns), 2 erf gelu,
+// 3 tanh gelu, 4 relu squared.  row_dest: scatter rows of the result, times row_scale when given, into out; row_scale alone:
+// multiplies before the activation.
 AIEN_API int aien_gemm_tc_grouped(const void* A, long lda, const void* W, long ldw, int groups, void* out, int c_dt, long ldc,
                                   const int* tile_group, int tiles, const int* row_dest, const float* row_scale,
                                   int N, int K, int epilogue, cudaStream_t stream) {
     if (tiles <= 0 || N <= 0) return 0;
     if (K <= 0 || (K & 7) || groups <= 0 || tile_group == nullptr) return AIEN_E_SHAPE;
-    if ((row_dest == nullptr) != (row_scale == nullptr)) return AIEN_E_SHAPE;
+    if (epilogue == 1 && ((N & 15) || row_dest != nullptr)) return AIEN_E_SHAPE;
     if ((lda & 7) || (ldw & 7) || ((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return AIEN_E_ALIGN;
     if ((long)tiles * ((N + 127) / 128) > 2147483647L || (long)groups * N > 2147483647L) return AIEN_E_SHAPE;
     const int rows_a = tiles * 128;
 #define TCG_CASE(EPIV, T) return launch_tc_grouped<EPIV, T>(A, lda, rows_a, W, ldw, groups, out, ldc, tile_group, tiles, row_dest, row_scale, N, K, stream)
     if (c_dt == AIEN_DT_BF16) {
         if (epilogue == 0) TCG_CASE(0, __nv_bfloat16);
+        if (epilogue == 1) TCG_CASE(1, __nv_bfloat16);
         if (epilogue == 2) TCG_CASE(2, __nv_bfloat16);
         if (epilogue == 3) TCG_CASE(3, __nv_bfloat16);
         if (epilogue == 4) TCG_CASE(4, __nv_bfloat16);

@@ -334,14 +334,14 @@ static int launch_latent_tc(const void* q, const void* cache, const int* bt, int
 
 
 // ---------------------------------------------------------------- one product per head, on the tensor cores
-// C[m, h, n] = sum_k A[m, h, k] * W[h, n, k] (see head_project_kernel) for bfloat16 A and W: tiles of 64 x 64 per CTA of
+// C[m, h, n] = sum_k A[m, h, k] * W[h, n, k], times sigmoid(gate[m, h]) when given (see head_project_kernel), for bfloat16 A and W: tiles of 64 x 64 per CTA of
 // four warps, k in steps of 64 through shared memory (cp.async), mma.sync.m16n8k16 with float32 accumulation.
 constexpr int HT_BM = 64, HT_BN = 64, HT_BK = 64, HT_STR = HT_BK + 8;
 
 template <typename TC>
 __global__ void __launch_bounds__(128)
 head_project_tc_kernel(const __nv_bfloat16* __restrict__ A, long lda, long a_head, const __nv_bfloat16* __restrict__ W, long w_head,
-                       TC* __restrict__ C, long ldc, long c_head, int M, int N, int K) {
+                       TC* __restrict__ C, long ldc, long c_head, int M, int N, int K, const float* __restrict__ gate, long ldg) {
     __shared__ __align__(16) __nv_bfloat16 As[HT_BM * HT_STR];
     __shared__ __align__(16) __nv_bfloat16 Ws[HT_BN * HT_STR];
     const uint32_t As_u = (uint32_t)__cvta_generic_to_shared(As), Ws_u = (uint32_t)__cvta_generic_to_shared(Ws);
@@ -388,6 +388,14 @@ head_project_tc_kernel(const __nv_bfloat16* __restrict__ A, long lda, long a_hea
         }
         __syncthreads();
     }
+    float gs[2][2];                                              // sigmoid of the head's gate, for this thread's four rows
+#pragma unroll
+    for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int m = m0 + mh * 32 + mt * 16 + g + r * 8;
+            gs[mt][r] = (gate != nullptr && m < M) ? 1.0f / (1.0f + expf(-gate[(size_t)m * ldg + h])) : 1.0f;
+        }
 #pragma unroll
     for (int mt = 0; mt < 2; ++mt)
 #pragma unroll
@@ -395,7 +403,7 @@ head_project_tc_kernel(const __nv_bfloat16* __restrict__ A, long lda, long a_hea
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int m = m0 + mh * 32 + mt * 16 + g + (e >> 1) * 8, n = n0 + nh * 32 + j * 8 + 2 * c + (e & 1);
-                if (m < M && n < N) C[(size_t)m * ldc + n] = from_f<TC>(acc[mt][j][e]);
+                if (m < M && n < N) C[(size_t)m * ldc + n] = from_f<TC>(acc[mt][j][e] * gs[mt][e >> 1]);
             }
 }
 
@@ -437,13 +445,13 @@ AIEN_API int aien_latent_attention_tc(const void* q, const void* cache, const in
 // A bfloat16 [M, lda] (head h at column h * a_head), W bfloat16 [heads, N, K], C [M, ldc] (head h at column h * c_head).
 // K, lda and a_head multiples of 8, A and W 16-byte aligned.
 AIEN_API int aien_head_project_tc(const void* A, long lda, long a_head, const void* W, void* C, int c_dt, long ldc, long c_head,
-                                  int M, int N, int K, int heads, cudaStream_t stream) {
+                                  int M, int N, int K, int heads, const float* gate, long ldg, cudaStream_t stream) {
     if (M <= 0 || N <= 0 || heads <= 0) return 0;
     if (K <= 0 || heads > 65535) return AIEN_E_SHAPE;
     if ((K & 7) || (lda & 7) || (a_head & 7) || ((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return AIEN_E_ALIGN;
     dim3 grid((N + HT_BN - 1) / HT_BN, (M + HT_BM - 1) / HT_BM, heads);
     if (grid.y > 65535) return AIEN_E_SHAPE;
     AIEN_DISPATCH_DTYPE(c_dt, TC, (head_project_tc_kernel<TC><<<grid, 128, 0, stream>>>((const __nv_bfloat16*)A, lda, a_head, (const __nv_bfloat16*)W,
-                                                                                     (long)N * K, (TC*)C, ldc, c_head, M, N, K)));
+                                                                                     (long)N * K, (TC*)C, ldc, c_head, M, N, K, gate, ldg)));
     return launch_status();
 }

@@ -12,6 +12,9 @@
 //   expert_down  part[c][t, :] = weight(t,c) * W_down[e(t,c)] act[t, c, :]   float32 parts, one per choice,
 //                which the consumer (the norm that takes the branch) adds in index order
 //   act_rows     f applied in place to [T, F] rows (the shared expert's hidden layer)
+//   A gated expert's first matrix holds gate and up rows (w_up [E, 2F, D]): act = silu(gate) * up.  On request the pair's
+//   weight multiplies the expert's input instead of its output: the products are linear, so it multiplies what they give
+//   before the activation, in float32.
 //
 // expert_up / expert_down are one warp per output value with the reduction in a fixed lane order, so a
 // token's result depends on its own row alone; they serve the 32-bit engine and sizes the others do not
@@ -96,28 +99,37 @@ moe_route_kernel(const float* __restrict__ z, int E, int groups, int keep, int t
 }
 
 // The router with a correction on the choice and experts that return their input.  s = softmax(z[t][0..E)) (rows ldz
-// apart); the `top` experts with the largest s + correction are chosen (ties to the lower index); a choice weighs s,
+// apart), or s = sigmoid(z) of every output by itself (`sigmoid`; without a correction the choice then goes by z, which has
+// the same order and does not saturate); the `top` experts with the largest s + correction are chosen (ties to the lower index); a choice weighs s,
 // divided by the sum of the chosen s plus renorm_eps when `renorm` is set.  Experts from `real` on have no tensors:
 // their output is their input, so their weights are summed into w_same[t] and the choice is handed on as expert 0
 // with weight zero (the expert products need no case for it).  One warp per token.
 __global__ void __launch_bounds__(32)
 moe_route_biased_kernel(const float* __restrict__ z, long ldz, int E, int real, int top, int renorm, float renorm_eps,
-                        const void* __restrict__ correction, int cdt, int* __restrict__ ids, float* __restrict__ wts,
+                        const void* __restrict__ correction, int cdt, int sigmoid, int* __restrict__ ids, float* __restrict__ wts,
                         float* __restrict__ w_same, int* __restrict__ expert_count) {
     __shared__ float s[ROUTE_MAX_EXPERTS];
     __shared__ float ch[ROUTE_MAX_EXPERTS];
     const int t = blockIdx.x, lane = threadIdx.x;
     const float* zr = z + (size_t)t * ldz;
-    float m = -INFINITY;
-    for (int e = lane; e < E; e += 32) { const float v = zr[e]; s[e] = v; m = fmaxf(m, v); }
-    m = warp_max(m);
-    float sum = 0.f;
-    for (int e = lane; e < E; e += 32) { const float v = expf(s[e] - m); s[e] = v; sum += v; }
-    sum = warp_sum(sum);
-    const float inv = 1.0f / sum;
-    for (int e = lane; e < E; e += 32) {
-        s[e] *= inv;
-        ch[e] = correction != nullptr ? s[e] + load_dyn(correction, cdt, e) : s[e];
+    if (sigmoid) {
+        for (int e = lane; e < E; e += 32) {
+            const float v = zr[e];
+            s[e] = 1.0f / (1.0f + expf(-v));
+            ch[e] = correction != nullptr ? s[e] + load_dyn(correction, cdt, e) : v;
+        }
+    } else {
+        float m = -INFINITY;
+        for (int e = lane; e < E; e += 32) { const float v = zr[e]; s[e] = v; m = fmaxf(m, v); }
+        m = warp_max(m);
+        float sum = 0.f;
+        for (int e = lane; e < E; e += 32) { const float v = expf(s[e] - m); s[e] = v; sum += v; }
+        sum = warp_sum(sum);
+        const float inv = 1.0f / sum;
+        for (int e = lane; e < E; e += 32) {
+            s[e] *= inv;
+            ch[e] = correction != nullptr ? s[e] + load_dyn(correction, cdt, e) : s[e];
+        }
     }
     __syncwarp();
     float wsum = 0.f;
@@ -156,10 +168,17 @@ moe_route_biased_kernel(const float* __restrict__ z, long ldz, int E, int real, 
 
 // ---------------------------------------------------------------- plain expert products
 // One warp per output value; 8 warps a CTA take 8 consecutive output rows of one (token, choice).
+// Row of w_up that makes gate (up: + up_step) number f of a gated expert: runs of `group` gate and up rows in turn, or all
+// gate rows ahead of all up rows (group 0).
+__device__ __forceinline__ int gated_row(int f, int F, int group, int* up_step) {
+    *up_step = group > 0 ? group : F;
+    return group > 0 ? (f / group) * 2 * group + f % group : f;
+}
+
 template <typename TH, typename TW, typename TO>
 __global__ void __launch_bounds__(256)
 moe_expert_up_kernel(const TH* __restrict__ h, long h_stride, const TW* __restrict__ w_up, const int* __restrict__ ids,
-                     TO* __restrict__ act, int top, int D, int F, int act_kind) {
+                     const float* __restrict__ in_wts, TO* __restrict__ act, int top, int D, int F, int act_kind, int gated, int group) {
     griddep_launch();
     griddep_wait();
     const int pair = blockIdx.x;                       // t * top + c
@@ -167,11 +186,28 @@ moe_expert_up_kernel(const TH* __restrict__ h, long h_stride, const TW* __restri
     const int f = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (f >= F) return;
     const int e = __ldcg(ids + pair);
-    const TW* wr = w_up + ((size_t)e * F + f) * D;
     const TH* hr = h + (size_t)t * h_stride;
+    const float scale = in_wts != nullptr ? __ldcg(in_wts + pair) : 1.0f;
+    if (gated) {
+        int up_step;
+        const int r = gated_row(f, F, group, &up_step);
+        const TW* wg = w_up + ((size_t)e * 2 * F + r) * D;
+        const TW* wu = wg + (size_t)up_step * D;
+        float g = 0.f, u = 0.f;
+        for (int i = lane; i < D; i += 32) {
+            const float hv = ld_act(hr + i);
+            g = fmaf(to_f(wg[i]), hv, g);
+            u = fmaf(to_f(wu[i]), hv, u);
+        }
+        g = warp_sum(g) * scale;
+        u = warp_sum(u) * scale;
+        if (lane == 0) act[(size_t)pair * F + f] = from_f<TO>(g / (1.0f + expf(-g)) * u);
+        return;
+    }
+    const TW* wr = w_up + ((size_t)e * F + f) * D;
     float acc = 0.f;
     for (int i = lane; i < D; i += 32) acc = fmaf(to_f(wr[i]), ld_act(hr + i), acc);
-    acc = warp_sum(acc);
+    acc = warp_sum(acc) * scale;
     if (lane == 0) act[(size_t)pair * F + f] = from_f<TO>(act_apply(acc, act_kind));
 }
 
@@ -191,7 +227,7 @@ moe_expert_down_kernel(const TA* __restrict__ act, const TW* __restrict__ w_down
     float acc = 0.f;
     for (int i = lane; i < F; i += 32) acc = fmaf(to_f(wr[i]), ld_act(ar + i), acc);
     acc = warp_sum(acc);
-    if (lane == 0) parts[((size_t)c * T + t) * D + n] = acc * __ldcg(wts + pair);
+    if (lane == 0) parts[((size_t)c * T + t) * D + n] = acc * (wts != nullptr ? __ldcg(wts + pair) : 1.0f);
 }
 
 // ---------------------------------------------------------------- rows sorted by expert, for the grouped product
@@ -281,7 +317,7 @@ moe_place_rows_kernel(const __nv_bfloat16* __restrict__ h, long h_stride, const 
 // ---------------------------------------------------------------- expert products of a few tokens (bfloat16)
 // A step that decodes brings few (token, choice) pairs, each with a whole expert's matrices to read:
 // the products are bound by that stream.  One warp per output value, 16-byte loads, ROWS output rows
-// of one pair per warp so that as many loads are in flight; K % 256 == 0 keeps every lane on whole vectors.
+// of one pair per warp so that as many loads are in flight; K is a multiple of 8.
 __device__ __forceinline__ float dot8(const uint4 w, const uint4 a) {
     const __nv_bfloat162* wp = reinterpret_cast<const __nv_bfloat162*>(&w);
     const __nv_bfloat162* ap = reinterpret_cast<const __nv_bfloat162*>(&a);
@@ -298,22 +334,38 @@ __device__ __forceinline__ float dot8(const uint4 w, const uint4 a) {
 constexpr int SV_ROWS = 4;        // output rows per warp
 
 // MODE 0: act[pair, f] = f(w[e, f, :] . x[pair / top, :])   (x = the tokens' rows, K = D)
-// MODE 1: parts[c, t, n] = wts[pair] * (w[e, n, :] . x[pair, :])  (x = the pairs' hidden rows, K = F)
+//         (wts given: times wts[pair] before f)
+// MODE 1: parts[c, t, n] = wts[pair] * (w[e, n, :] . x[pair, :])  (x = the pairs' hidden rows, K = F; wts null: no factor)
+// MODE 2: a gated expert: rows of w as gated_row says, act[pair, f] = silu(gate) * up (wts given: both times wts[pair] first)
 template <int MODE>
 __global__ void __launch_bounds__(256)
 moe_expert_rows_bf16_kernel(const __nv_bfloat16* __restrict__ x, long x_stride, const __nv_bfloat16* __restrict__ w,
                             const int* __restrict__ ids, const float* __restrict__ wts, void* __restrict__ out,
-                            int T, int top, int N, int K, int act_kind) {
+                            int T, int top, int N, int K, int act_kind, int group) {
     griddep_launch();
+    constexpr int OUTS = MODE == 2 ? SV_ROWS / 2 : SV_ROWS;      // results a warp makes; a gated one takes two rows
     const int pair = blockIdx.x;
     const int lane = threadIdx.x & 31;
-    const int n0 = (blockIdx.y * 8 + (threadIdx.x >> 5)) * SV_ROWS;
+    const int n0 = (blockIdx.y * 8 + (threadIdx.x >> 5)) * OUTS;
     griddep_wait();
     if (n0 >= N) return;
     const int e = __ldcg(ids + pair);
     const int t = pair / top;
-    const __nv_bfloat16* xr = x + (size_t)(MODE == 0 ? t : pair) * x_stride;
-    const __nv_bfloat16* wr = w + ((size_t)e * N + n0) * K;
+    const __nv_bfloat16* xr = x + (size_t)(MODE == 1 ? pair : t) * x_stride;
+    const __nv_bfloat16* wr[SV_ROWS];
+    bool in[SV_ROWS];
+#pragma unroll
+    for (int j = 0; j < SV_ROWS; ++j) {
+        const int n = n0 + (MODE == 2 ? j >> 1 : j);
+        in[j] = n < N;
+        if (MODE == 2) {
+            int up_step;
+            const int r = gated_row(in[j] ? n : n0, N, group, &up_step);
+            wr[j] = w + ((size_t)e * 2 * N + r + ((j & 1) ? up_step : 0)) * K;
+        } else {
+            wr[j] = w + ((size_t)e * N + (in[j] ? n : n0)) * K;
+        }
+    }
     float acc[SV_ROWS];
 #pragma unroll
     for (int j = 0; j < SV_ROWS; ++j) acc[j] = 0.f;
@@ -322,21 +374,25 @@ moe_expert_rows_bf16_kernel(const __nv_bfloat16* __restrict__ x, long x_stride, 
         uint4 wv[SV_ROWS];
 #pragma unroll
         for (int j = 0; j < SV_ROWS; ++j)
-            wv[j] = (n0 + j < N) ? __ldg(reinterpret_cast<const uint4*>(wr + (size_t)j * K + k)) : make_uint4(0u, 0u, 0u, 0u);
+            wv[j] = in[j] ? __ldg(reinterpret_cast<const uint4*>(wr[j] + k)) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
         for (int j = 0; j < SV_ROWS; ++j) acc[j] += dot8(wv[j], a);
     }
 #pragma unroll
     for (int j = 0; j < SV_ROWS; ++j) acc[j] = warp_sum(acc[j]);
     if (lane == 0) {
+        const float scale = wts != nullptr ? __ldcg(wts + pair) : 1.0f;
 #pragma unroll
-        for (int j = 0; j < SV_ROWS; ++j) {
+        for (int j = 0; j < OUTS; ++j) {
             if (n0 + j >= N) break;
             if (MODE == 0) {
-                reinterpret_cast<__nv_bfloat16*>(out)[(size_t)pair * N + n0 + j] = __float2bfloat16_rn(act_apply(acc[j], act_kind));
+                reinterpret_cast<__nv_bfloat16*>(out)[(size_t)pair * N + n0 + j] = __float2bfloat16_rn(act_apply(acc[j] * scale, act_kind));
+            } else if (MODE == 2) {
+                const float g = acc[2 * j] * scale, u = acc[2 * j + 1] * scale;
+                reinterpret_cast<__nv_bfloat16*>(out)[(size_t)pair * N + n0 + j] = __float2bfloat16_rn(g / (1.0f + expf(-g)) * u);
             } else {
                 const int c = pair - t * top;
-                reinterpret_cast<float*>(out)[((size_t)c * T + t) * N + n0 + j] = acc[j] * __ldcg(wts + pair);
+                reinterpret_cast<float*>(out)[((size_t)c * T + t) * N + n0 + j] = acc[j] * scale;
             }
         }
     }
@@ -368,23 +424,25 @@ AIEN_API int aien_moe_route(const float* z, int T, int E, int groups, int keep, 
 // z float32 [T, ldz]: the first E numbers of a row are the router's; correction [E] in c_dt (or null); experts from
 // `real` on return their input (w_same float32 [T], needed when real < E).
 AIEN_API int aien_moe_route_biased(const float* z, long ldz, int T, int E, int real, int top, int renorm, float renorm_eps,
-                                   const void* correction, int c_dt, int* ids, float* wts, float* w_same, int* expert_count,
+                                   const void* correction, int c_dt, int sigmoid, int* ids, float* wts, float* w_same, int* expert_count,
                                    cudaStream_t stream) {
     if (T <= 0) return 0;
     if (E <= 0 || E > ROUTE_MAX_EXPERTS || real <= 0 || real > E || top <= 0 || top > E || (real < E && w_same == nullptr)) return AIEN_E_SHAPE;
-    moe_route_biased_kernel<<<T, 32, 0, stream>>>(z, ldz, E, real, top, renorm, renorm_eps, correction, c_dt, ids, wts, w_same, expert_count);
+    moe_route_biased_kernel<<<T, 32, 0, stream>>>(z, ldz, E, real, top, renorm, renorm_eps, correction, c_dt, sigmoid, ids, wts, w_same, expert_count);
     return launch_status();
 }
 
-// h [T, D] (row stride h_stride), w_up [E, F, D], act [T * top, F]; act_kind 0: erf gelu, 1: tanh gelu.
-AIEN_API int aien_moe_expert_up(const void* h, int h_dt, long h_stride, const void* w_up, int w_dt, const int* ids,
-                                void* act, int act_dt, int T, int top, int D, int F, int act_kind, cudaStream_t stream) {
+// h [T, D] (row stride h_stride), w_up [E, F, D], act [T * top, F]; act_kind 0: erf gelu, 1: tanh gelu, 2: relu squared.
+// gated != 0: w_up [E, 2F, D] with gate and up rows in runs of `group` (0: all gate rows first).  in_wts [T * top] or null:
+// the pair's weight multiplies the expert's input.
+AIEN_API int aien_moe_expert_up(const void* h, int h_dt, long h_stride, const void* w_up, int w_dt, const int* ids, const float* in_wts,
+                                void* act, int act_dt, int T, int top, int D, int F, int act_kind, int gated, int group, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (T * (long)top > 2147483647L || D <= 0 || F <= 0 || (F + 7) / 8 > 65535) return AIEN_E_SHAPE;
+    if (T * (long)top > 2147483647L || D <= 0 || F <= 0 || (F + 7) / 8 > 65535 || group < 0 || (group > 0 && F % group)) return AIEN_E_SHAPE;
     dim3 grid(T * top, (F + 7) / 8);
     AIEN_DISPATCH_DTYPE(h_dt, TH, AIEN_DISPATCH_DTYPE(w_dt, TW, AIEN_DISPATCH_DTYPE(act_dt, TO,
         (launch_chain(moe_expert_up_kernel<TH, TW, TO>, grid, dim3(256), 0, stream,
-                      (const TH*)h, h_stride, (const TW*)w_up, ids, (TO*)act, top, D, F, act_kind)))));
+                      (const TH*)h, h_stride, (const TW*)w_up, ids, in_wts, (TO*)act, top, D, F, act_kind, gated, group)))));
     return launch_status();
 }
 
@@ -418,21 +476,24 @@ AIEN_API int aien_moe_place_rows(const void* h, long h_stride, const int* ids, c
     return launch_status();
 }
 
-// The expert products of a few tokens, bfloat16: mode 0 = up with activation (out bfloat16 [T*top, N], K = D),
-// mode 1 = down, weighted, into float32 parts [top, T, N] (K = F).  K % 256 == 0, 16-byte aligned rows.
+// The expert products of a few tokens, bfloat16: mode 0 = up with activation (out bfloat16 [T*top, N], K = D), mode 2 = the
+// same for gated experts (w [E, 2N, K], runs of `group` gate and up rows), in both wts (or null) multiplies the input; mode 1 =
+// down into float32 parts [top, T, N] (K = F) times wts (or null).  K a multiple of 8, 16-byte aligned rows.
 AIEN_API int aien_moe_expert_rows_bf16(int mode, const void* x, long x_stride, const void* w, const int* ids, const float* wts,
-                                       void* out, int T, int top, int N, int K, int act_kind, cudaStream_t stream) {
+                                       void* out, int T, int top, int N, int K, int act_kind, int group, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (N <= 0 || K <= 0 || (K & 255) || (x_stride & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return AIEN_E_ALIGN;
-    const int tiles = (N + 8 * SV_ROWS - 1) / (8 * SV_ROWS);
-    if (tiles > 65535 || (long)T * top > 2147483647L) return AIEN_E_SHAPE;
+    if (N <= 0 || K <= 0 || (K & 7) || (x_stride & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return AIEN_E_ALIGN;
+    const int outs = 8 * (mode == 2 ? SV_ROWS / 2 : SV_ROWS);
+    const int tiles = (N + outs - 1) / outs;
+    if (tiles > 65535 || (long)T * top > 2147483647L || group < 0 || (group > 0 && N % group)) return AIEN_E_SHAPE;
     dim3 grid(T * top, tiles);
-    if (mode == 0)
-        launch_chain(moe_expert_rows_bf16_kernel<0>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)x, x_stride,
-                     (const __nv_bfloat16*)w, ids, wts, out, T, top, N, K, act_kind);
-    else
-        launch_chain(moe_expert_rows_bf16_kernel<1>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)x, x_stride,
-                     (const __nv_bfloat16*)w, ids, wts, out, T, top, N, K, act_kind);
+#define MR_CASE(M)                                                                                                       \
+    launch_chain(moe_expert_rows_bf16_kernel<M>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)x, x_stride,           \
+                 (const __nv_bfloat16*)w, ids, wts, out, T, top, N, K, act_kind, group)
+    if (mode == 0) MR_CASE(0);
+    else if (mode == 2) MR_CASE(2);
+    else MR_CASE(1);
+#undef MR_CASE
     return launch_status();
 }
 

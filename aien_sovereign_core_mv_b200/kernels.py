@@ -122,12 +122,12 @@ def _declare(l: ctypes.CDLL) -> None:
         "aien_stream_norm_inplace": [P, P, I, F, P, I, I, I, P],
         "aien_qk_rope_pairs_unit_kv_write": [P, L, I, P, L, P, L, I, I, I, c_size_t, P, L, I, I, I, F, P, P, I, P, P, P, I, I, I, P],
         "aien_moe_route": [P, I, I, I, I, I, I, P, P, P, P],
-        "aien_moe_expert_up": [P, I, L, P, I, P, P, I, I, I, I, I, I, P],
+        "aien_moe_expert_up": [P, I, L, P, I, P, P, P, I, I, I, I, I, I, I, I, P],
         "aien_moe_expert_down": [P, I, P, I, P, P, P, I, I, I, I, P],
         "aien_act_rows": [P, I, c_size_t, I, P],
         "aien_moe_plan_rows": [P, I, I, P, P, P, P],
         "aien_moe_place_rows": [P, L, P, P, P, I, I, P, I, P, P, P],
-        "aien_moe_expert_rows_bf16": [I, P, L, P, P, P, P, I, I, I, I, I, P],
+        "aien_moe_expert_rows_bf16": [I, P, L, P, P, P, P, I, I, I, I, I, I, P],
         "aien_gemm_tc_grouped": [P, L, P, L, I, P, I, L, P, I, P, P, I, I, I, P],
         "aien_argmax_rows": [P, I, I, P, P],
         "aien_sample_rows": [P, I, I, P, P, P, P, P, P, P, P, P],
@@ -167,9 +167,9 @@ def _declare(l: ctypes.CDLL) -> None:
         "aien_latent_prepare": [P, I, L, I, P, P, I, F, P, I, L, I, I, I, I, P, P, P, P, I, I, P],
         "aien_rotate_pairs_rows": [P, I, L, L, P, I, L, L, I, I, I, I, P, P, P],
         "aien_latent_attention_tc": [P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, P, I, P, P, I, P],
-        "aien_head_project_tc": [P, L, L, P, P, I, L, L, I, I, I, I, P],
+        "aien_head_project_tc": [P, L, L, P, P, I, L, L, I, I, I, I, P, L, P],
         "aien_latent_attention_tc_supports": [I, I],
-        "aien_head_project": [P, I, L, L, P, I, L, L, P, I, L, L, I, I, I, I, P],
+        "aien_head_project": [P, I, L, L, P, I, L, L, P, I, L, L, I, I, I, I, P, L, P],
         "aien_latent_attention": [P, L, P, I, P, I, P, P, P, P, I, L, I, I, I, I, I, I, F, P, P],
         "aien_post_norm_add": [P, P, I, I, c_size_t, P, I, F, F, P, I, F, P, I, I, I, P],
         "aien_embed_gather_scaled": [P, I, P, P, I, I, I, F, P],
@@ -195,7 +195,14 @@ def _declare(l: ctypes.CDLL) -> None:
         "aien_clamped_glu": [P, I, L, I, I, P, P, I, F, F, P, I, L, I, I, P],
         "aien_sigmoid_gate": [P, I, L, P, L, F, P, I, L, I, I, P],
         "aien_routed_combine": [P, I, I, c_size_t, P, I, L, P, P, I, I, c_size_t, P, L, P, I, I, P],
-        "aien_moe_route_biased": [P, L, I, I, I, I, I, F, P, I, P, P, P, P, P],
+        "aien_moe_route_biased": [P, L, I, I, I, I, I, F, P, I, I, P, P, P, P, P],
+        "aien_sum_terms_rmsnorm": [P, I] + 3 * [P, I, I, c_size_t, P, L] + [P, I, I, P, I, F, P, I, I, I, P],
+        "aien_pass_rows": [P, I] + 3 * [P, I, I, c_size_t, P, L] + [P, P, I, I, I, P],
+        "aien_matrix_memory_gates": [P, L, I, I, P, P, F, P, c_size_t, c_size_t, P, P, P, P, I, I, I, P],
+        "aien_matrix_memory_walk": [P, I, L, I, I, I, F, P, P, c_size_t, P, P, P, P, P, I, I, I, I, P],
+        "aien_matrix_memory_finish": [P, P, P, P, I, L, P, I, F, F, P, I, L, I, I, I, P],
+        "aien_matrix_memory_token_supports": [I, I],
+        "aien_matrix_memory_token": [P, I, L, I, I, I, I, F, P, L, I, I, P, P, F, P, c_size_t, P, P, P, P, I, F, F, P, I, L, I, I, I, I, P],
         "aien_rope_halves_value_write": [P, L, I, I, I, I, I, I, I, P, P, I, P, P, I, L, P, P, I, I, P],
     }
     for name, args in sigs.items():
@@ -487,18 +494,26 @@ def moe_route(z: torch.Tensor, groups: int, keep: int, top: int, renorm: bool, i
                                 _stream()), "moe_route")
 
 
-def moe_expert_up(h: torch.Tensor, w_up: torch.Tensor, ids: torch.Tensor, act: torch.Tensor, top: int, act_kind: int) -> None:
-    """act[t*top + c] = f(w_up[ids[t,c]] . h[t]); h [T,D], w_up [E,F,D], act [T*top, F]."""
-    _dev(h, w_up, ids, act)
+ACT_GATED = 3                       # experts of the form silu(gate) * up: their first matrix holds gate and up rows
+
+
+def moe_expert_up(h: torch.Tensor, w_up: torch.Tensor, ids: torch.Tensor, act: torch.Tensor, top: int, act_kind: int,
+                  in_wts: Optional[torch.Tensor] = None, group: int = 0) -> None:
+    """act[t*top + c] = f(w_up[ids[t,c]] . h[t]); h [T,D], w_up [E,F,D], act [T*top, F].  ``act_kind`` ACT_GATED: w_up [E,2F,D],
+    gate and up rows in runs of ``group`` (0: all gate rows first).  ``in_wts`` float32 [T,top]: multiplies h[t]."""
+    _dev(h, w_up, ids, act, in_wts)
     T, D = h.shape
+    gated = act_kind == ACT_GATED
     E, Fd, D2 = w_up.shape
+    Fd = Fd // 2 if gated else Fd
     assert D2 == D and h.stride(1) == 1 and w_up.is_contiguous() and act.is_contiguous() and tuple(act.shape) == (T * top, Fd)
-    _check(lib().aien_moe_expert_up(_p(h), dt(h), h.stride(0), _p(w_up), dt(w_up), _p(ids), _p(act), dt(act), T, int(top), D, Fd,
-                                    int(act_kind), _stream()), "moe_expert_up")
+    assert in_wts is None or (in_wts.dtype == torch.float32 and in_wts.is_contiguous() and in_wts.numel() >= T * top)
+    _check(lib().aien_moe_expert_up(_p(h), dt(h), h.stride(0), _p(w_up), dt(w_up), _p(ids), _p(in_wts), _p(act), dt(act), T, int(top), D, Fd,
+                                    0 if gated else int(act_kind), 1 if gated else 0, int(group), _stream()), "moe_expert_up")
 
 
-def moe_expert_down(act: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, parts: torch.Tensor, top: int) -> None:
-    """parts[c, t] = wts[t,c] * (w_down[ids[t,c]] . act[t*top + c]); w_down [E,D,F], parts float32 [top,T,D]."""
+def moe_expert_down(act: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, wts: Optional[torch.Tensor], parts: torch.Tensor, top: int) -> None:
+    """parts[c, t] = wts[t,c] * (w_down[ids[t,c]] . act[t*top + c]) (wts None: no factor); w_down [E,D,F], parts float32 [top,T,D]."""
     _dev(act, w_down, ids, wts, parts)
     E, D, Fd = w_down.shape
     T = act.shape[0] // top
@@ -527,7 +542,7 @@ _MOE_IMPL = __import__("os").environ.get("AIEN_B200_MOE", "").strip().lower()   
 
 
 def moe_grouped_supports(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor) -> bool:
-    D, Fd = w_up.shape[2], w_up.shape[1]
+    D, Fd = w_down.shape[1], w_down.shape[2]
     return (h.dtype == torch.bfloat16 and w_up.dtype == torch.bfloat16 and w_down.dtype == torch.bfloat16 and D % 8 == 0
             and Fd % 8 == 0 and h.stride(1) == 1 and h.stride(0) % 8 == 0 and h.data_ptr() % 16 == 0
             and w_up.data_ptr() % 16 == 0 and w_down.data_ptr() % 16 == 0)
@@ -539,28 +554,34 @@ def moe_takes_grouped(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor)
 
 
 def moe_experts(ctx, h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor,
-                top: int, act_kind: int, expert_count: Optional[torch.Tensor] = None) -> torch.Tensor:
+                top: int, act_kind: int, expert_count: Optional[torch.Tensor] = None, group: int = 0, on_input: bool = False) -> torch.Tensor:
     """Returns parts [top, T, D] with parts[c, t] = wts[t,c] * w_down[e] f(w_up[e] h[t]), e = ids[t,c]: the chosen
     experts of every token, weighted, one part per choice (float32; bfloat16 from the grouped products, whose
     consumer adds them in float32).  ``expert_count``: what moe_route counted; the grouped products need it.
+    ``act_kind`` ACT_GATED: w_up [E, 2F, D] holds gate and up rows in runs of ``group`` (8 for the grouped products; 0: all
+    gate rows first) and f gives silu(gate) * up.  ``on_input``: the weight multiplies h[t] instead of the output, which
+    every path does behind the first product, in float32.
     bfloat16: a few tokens stream their experts' rows (one warp per output value, 16-byte loads); larger
     steps place the (token, choice) pairs in rows sorted by expert and run two grouped tcgen05 products, the activation in
     the first one's epilogue, the weights and the way back to token order in the second's.  float32, and
     sizes those kernels do not take: the plain products."""
     T, D = h.shape
-    E, Fd, _ = w_up.shape
+    gated = act_kind == ACT_GATED
+    E, _, Fd = w_down.shape
     ws = ctx.workspace
     ok = _MOE_IMPL != "plain" and moe_grouped_supports(h, w_up, w_down)
     grouped = ok and T > MOE_ROWS_MAX_TOKENS
     if grouped and expert_count is None:
         raise KernelError("moe_experts: the grouped products need the per-expert counts of moe_route (expert_count)")
+    if grouped and gated and group != 8:
+        raise KernelError("moe_experts: the grouped products take gate and up rows in runs of 8")
     parts = ws.take((top, T, D), torch.bfloat16 if grouped else torch.float32)
-    if ok and T <= MOE_ROWS_MAX_TOKENS and D % 256 == 0 and Fd % 256 == 0:
+    if ok and not grouped:
         act = ws.take((T * top, Fd), torch.bfloat16)
-        _check(lib().aien_moe_expert_rows_bf16(0, _p(h), h.stride(0), _p(w_up), _p(ids), _p(wts), _p(act), T, top, Fd, D,
-                                               int(act_kind), _stream()), "moe_expert_rows(up)")
-        _check(lib().aien_moe_expert_rows_bf16(1, _p(act), Fd, _p(w_down), _p(ids), _p(wts), _p(parts), T, top, D, Fd,
-                                               int(act_kind), _stream()), "moe_expert_rows(down)")
+        _check(lib().aien_moe_expert_rows_bf16(2 if gated else 0, _p(h), h.stride(0), _p(w_up), _p(ids), _p(wts if on_input else None), _p(act), T,
+                                               top, Fd, D, 0 if gated else int(act_kind), int(group), _stream()), "moe_expert_rows(up)")
+        _check(lib().aien_moe_expert_rows_bf16(1, _p(act), Fd, _p(w_down), _p(ids), _p(None if on_input else wts), _p(parts), T, top, D, Fd,
+                                               0, 0, _stream()), "moe_expert_rows(down)")
         return parts
     if grouped:
         tiles = _moe_tiles(T * top, E)
@@ -574,14 +595,15 @@ def moe_experts(ctx, h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, 
         _check(lib().aien_moe_plan_rows(_p(expert_count), E, tiles, _p(cursor), _p(tile_group), _p(row_dest), _stream()), "moe_plan_rows")
         _check(lib().aien_moe_place_rows(_p(h), h.stride(0), _p(ids), _p(wts), _p(cursor), T, top, _p(a_sorted), D, _p(row_dest),
                                          _p(row_scale), _stream()), "moe_place_rows")
-        _check(lib().aien_gemm_tc_grouped(_p(a_sorted), D, _p(w_up), D, E, _p(act), BF16, Fd, _p(tile_group), tiles, None, None,
-                                          Fd, D, 2 + int(act_kind), _stream()), "gemm_tc_grouped(up)")
+        _check(lib().aien_gemm_tc_grouped(_p(a_sorted), D, _p(w_up), D, E, _p(act), BF16, Fd, _p(tile_group), tiles, None,
+                                          _p(row_scale) if on_input else None, w_up.shape[1], D, 1 if gated else 2 + int(act_kind), _stream()),
+               "gemm_tc_grouped(up)")
         _check(lib().aien_gemm_tc_grouped(_p(act), Fd, _p(w_down), Fd, E, _p(parts), BF16, D, _p(tile_group), tiles, _p(row_dest),
-                                          _p(row_scale), D, Fd, 0, _stream()), "gemm_tc_grouped(down)")
+                                          None if on_input else _p(row_scale), D, Fd, 0, _stream()), "gemm_tc_grouped(down)")
         return parts
     act = ws.take((T * top, Fd), ctx.dtype)
-    moe_expert_up(h, w_up, ids, act, top, act_kind)
-    moe_expert_down(act, w_down, ids, wts, parts, top)
+    moe_expert_up(h, w_up, ids, act, top, act_kind, wts if on_input else None, group)
+    moe_expert_down(act, w_down, ids, None if on_input else wts, parts, top)
     return parts
 
 
@@ -1404,8 +1426,10 @@ def rotate_pairs_rows(q: torch.Tensor, q_head: int, col0: int, out: torch.Tensor
                                         int(rot_dim), int(rot_dims), _p(cos), _p(sin), _stream()), "rotate_pairs_rows")
 
 
-def head_project(a: torch.Tensor, a_head: int, a_col0: int, w: torch.Tensor, out: torch.Tensor, o_head: int, o_col0: int) -> None:
+def head_project(a: torch.Tensor, a_head: int, a_col0: int, w: torch.Tensor, out: torch.Tensor, o_head: int, o_col0: int,
+                 gate: Optional[torch.Tensor] = None) -> None:
     """out[t, h*o_head + o_col0 + n] = sum_k a[t, h*a_head + a_col0 + k] * w[h, n, k]: one product per head, w [heads, N, K].
+    ``gate`` float32 [T, heads] (row stride free): the result of head h is multiplied by sigmoid(gate[t, h]).
     bfloat16 operands whose rows are whole aligned 16-byte pieces run on the tensor cores, everything else on the CUDA cores;
     both sum in float32."""
     _dev(a, w, out)
@@ -1413,14 +1437,17 @@ def head_project(a: torch.Tensor, a_head: int, a_col0: int, w: torch.Tensor, out
     M = a.shape[0]
     assert a.stride(1) == 1 and out.stride(1) == 1 and w.is_contiguous() and out.shape[0] == M
     assert (heads - 1) * a_head + a_col0 + K_ <= a.shape[1] and (heads - 1) * o_head + o_col0 + N <= out.shape[1]
+    assert gate is None or (gate.dtype == torch.float32 and tuple(gate.shape) == (M, heads) and gate.stride(1) == 1)
+    _dev(gate)
+    gp, ldg = _p(gate), gate.stride(0) if gate is not None else 0
     av, ov = a[:, a_col0:], out[:, o_col0:]
     if (_LATENT_IMPL != "plain" and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and K_ % 8 == 0 and a.stride(0) % 8 == 0
             and a_head % 8 == 0 and av.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
         _check(lib().aien_head_project_tc(_p(av), a.stride(0), int(a_head), _p(w), _p(ov), dt(out), out.stride(0), int(o_head), M, N, K_,
-                                          heads, _stream()), "head_project_tc")
+                                          heads, gp, ldg, _stream()), "head_project_tc")
         return
     _check(lib().aien_head_project(_p(av), dt(a), a.stride(0), int(a_head), _p(w), dt(w), K_, N * K_, _p(ov), dt(out), out.stride(0),
-                                   int(o_head), M, N, K_, heads, _stream()), "head_project")
+                                   int(o_head), M, N, K_, heads, gp, ldg, _stream()), "head_project")
 
 
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, max_blocks: int, seq_of_token: torch.Tensor,
@@ -1953,8 +1980,9 @@ def routed_combine(parts: torch.Tensor, h: Optional[torch.Tensor], w_same: Optio
 
 def moe_route_biased(z: torch.Tensor, num_experts: int, real: int, top: int, renorm: bool, renorm_eps: float,
                      correction: Optional[torch.Tensor], ids: torch.Tensor, wts: torch.Tensor, w_same: Optional[torch.Tensor],
-                     expert_count: Optional[torch.Tensor] = None) -> None:
-    """Router with a correction on the choice: s = softmax(z[:, :num_experts]) (float32); the ``top`` largest s + correction
+                     expert_count: Optional[torch.Tensor] = None, sigmoid: bool = False) -> None:
+    """Router with a correction on the choice: s = softmax(z[:, :num_experts]), or with ``sigmoid`` the sigmoid of every
+    output by itself (float32); the ``top`` largest s + correction
     are chosen; weights s (``renorm``: divided by their sum + renorm_eps).  Experts from ``real`` on return their input:
     their weights are summed into ``w_same`` [T] and their choices handed on as expert 0 with weight zero."""
     _dev(z, correction, ids, wts, w_same, expert_count)
@@ -1964,8 +1992,8 @@ def moe_route_biased(z: torch.Tensor, num_experts: int, real: int, top: int, ren
     assert correction is None or (correction.is_contiguous() and correction.numel() == num_experts)
     assert w_same is None or (w_same.dtype == torch.float32 and w_same.is_contiguous() and w_same.numel() >= T)
     _check(lib().aien_moe_route_biased(_p(z), z.stride(0), T, int(num_experts), int(real), int(top), 1 if renorm else 0, float(renorm_eps),
-                                       _p(correction), dt(correction) if correction is not None else F32, _p(ids), _p(wts), _p(w_same),
-                                       _p(expert_count), _stream()), "moe_route_biased")
+                                       _p(correction), dt(correction) if correction is not None else F32, 1 if sigmoid else 0, _p(ids), _p(wts),
+                                       _p(w_same), _p(expert_count), _stream()), "moe_route_biased")
 
 
 def rope_halves_value_write(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, nq: int, nkv: int, hd: int, hdv: int,
@@ -1983,3 +2011,120 @@ def rope_halves_value_write(proj: torch.Tensor, q_off: int, k_off: int, v_off: i
     _check(lib().aien_rope_halves_value_write(_p(proj), proj.stride(0), int(q_off), int(k_off), int(v_off), int(nq), int(nkv), int(hd), int(hdv),
                                               _p(cos), _p(sin), int(rot), _p(slot_map), _p(q_out), dt(q_out), q_out.stride(0), _p(k_cache),
                                               _p(v_cache), dt(k_cache), T, _stream()), "rope_halves_value_write")
+
+
+# ---------------------------------------------------------------------------- several branches pending at once
+MAX_SUM_TERMS = 3
+
+
+def _term_args(terms, T: int, H: int) -> list:
+    """The kernels' arguments for ``terms``: (tensor [T,H] or [P,T,H], gate float32 [T] (stride free) or None) pairs."""
+    assert len(terms) <= MAX_SUM_TERMS
+    args = []
+    for t, gate in terms:
+        _dev(t, gate)
+        assert t.is_contiguous() and tuple(t.shape[-2:]) == (T, H) and t.dim() in (2, 3)
+        assert gate is None or (gate.dtype == torch.float32 and gate.numel() >= T)
+        args += [_p(t), dt(t), t.shape[0] if t.dim() == 3 else 1, T * H if t.dim() == 3 else 0, _p(gate), gate.stride(0) if gate is not None else 0]
+    return args + [0, F32, 0, 0, 0, 0] * (MAX_SUM_TERMS - len(terms))
+
+
+def sum_terms_rmsnorm(x: torch.Tensor, terms, bias: Optional[torch.Tensor], replace: bool, weight: Optional[torch.Tensor], eps: float,
+                      out: Optional[torch.Tensor]) -> None:
+    """x += the terms + bias (``replace``: x = them), float32 [T,H] in place; a term is (tensor [T,H] or parts [P,T,H], gate or
+    None) and counts times sigmoid(gate[t]).  With ``out``: out = rmsnorm(x) * weight."""
+    _dev(x, bias, weight, out)
+    T, H = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and (bias is None or (bias.numel() == H and bias.is_contiguous()))
+    assert out is None or (out.is_contiguous() and out.shape == x.shape and weight.numel() == H and weight.is_contiguous())
+    _check(lib().aien_sum_terms_rmsnorm(_p(x), len(terms), *_term_args(terms, T, H), _p(bias), dt(bias) if bias is not None else F32, 1 if replace else 0,
+                                        _p(weight), dt(weight) if weight is not None else F32, float(eps), _p(out), dt(out) if out is not None else F32,
+                                        T, H, _stream()), "sum_terms_rmsnorm")
+
+
+def pass_rows(x: torch.Tensor, terms, x0: torch.Tensor, out: torch.Tensor) -> None:
+    """Rows of a product over the stream with its pending terms and x0 (float32 [T,H]): out bfloat16 [T,3H] = [hi | lo | x0],
+    hi the rounded stream and lo the rounded rest, or float32 [T,2H] = [x | x0].  x itself stays."""
+    _dev(x, x0, out)
+    T, H = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and x0.dtype == torch.float32 and x0.is_contiguous() and x0.shape == x.shape
+    assert out.is_contiguous() and tuple(out.shape) == (T, (2 if out.dtype == torch.float32 else 3) * H)
+    _check(lib().aien_pass_rows(_p(x), len(terms), *_term_args(terms, T, H), _p(x0), _p(out), dt(out), T, H, _stream()), "pass_rows")
+
+
+# ---------------------------------------------------------------------------- matrix memory
+def _state_args(state: torch.Tensor, slot_map: torch.Tensor, q_start: torch.Tensor, positions: torch.Tensor) -> None:
+    _dev(state, slot_map, q_start, positions)
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous()
+    for t in (slot_map, q_start, positions):
+        assert t.dtype == torch.int32
+
+
+def matrix_memory_state_floats(heads: int, dim: int, vdim: int) -> int:
+    """Floats of one request's slot: S [heads, dim, vdim], n [heads, dim], m [heads], rounded up to whole float4."""
+    return (heads * (dim * vdim + dim + 1) + 3) // 4 * 4
+
+
+def matrix_memory_gates(z: torch.Tensor, i_off: int, f_off: int, bi: torch.Tensor, bf: torch.Tensor, cap: float, state: torch.Tensor,
+                        slot_map: torch.Tensor, q_start: torch.Tensor, positions: torch.Tensor, gates: torch.Tensor, num_seqs: int,
+                        heads: int, dim: int, vdim: int) -> None:
+    """gates float32 [T, 3*heads] = log keep | take | m of every token, from the gates' projections z float32 [T, *]; the
+    running maximum continues from the slots and is left there."""
+    _dev(z, bi, bf, gates)
+    _state_args(state, slot_map, q_start, positions)
+    T = z.shape[0]
+    assert z.dtype == torch.float32 and z.stride(1) == 1 and max(i_off, f_off) + heads <= z.shape[1]
+    assert bi.dtype == torch.float32 and bf.dtype == torch.float32 and bi.numel() == heads and bf.numel() == heads
+    assert gates.dtype == torch.float32 and gates.is_contiguous() and tuple(gates.shape) == (T, 3 * heads)
+    assert state.shape[1] >= matrix_memory_state_floats(heads, dim, vdim)
+    _check(lib().aien_matrix_memory_gates(_p(z), z.stride(0), int(i_off), int(f_off), _p(bi), _p(bf), float(cap), _p(state), state.stride(0),
+                                          heads * (dim * vdim + dim), _p(slot_map), _p(q_start), _p(positions), _p(gates), T, int(num_seqs),
+                                          int(heads), _stream()), "matrix_memory_gates")
+
+
+def matrix_memory_walk(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_scale: float, gates: torch.Tensor, state: torch.Tensor,
+                       slot_map: torch.Tensor, q_start: torch.Tensor, positions: torch.Tensor, num: torch.Tensor, nq: torch.Tensor,
+                       num_seqs: int, heads: int, dim: int, vdim: int) -> None:
+    """The recurrence token by token: num float32 [T, heads*vdim] = S^T q, nq float32 [T, heads] = n . q (q times q_scale), with
+    q, k, v columns of ``proj`` [T, *]; S and n continue from the slots and are left there."""
+    _dev(proj, gates, num, nq)
+    _state_args(state, slot_map, q_start, positions)
+    T = proj.shape[0]
+    assert proj.stride(1) == 1 and max(q_off, k_off) + heads * dim <= proj.shape[1] and v_off + heads * vdim <= proj.shape[1]
+    assert gates.is_contiguous() and tuple(gates.shape) == (T, 3 * heads) and state.shape[1] >= matrix_memory_state_floats(heads, dim, vdim)
+    assert num.dtype == torch.float32 and num.is_contiguous() and num.numel() == T * heads * vdim and nq.is_contiguous() and nq.numel() == T * heads
+    _check(lib().aien_matrix_memory_walk(_p(proj), dt(proj), proj.stride(0), int(q_off), int(k_off), int(v_off), float(q_scale), _p(gates), _p(state),
+                                         state.stride(0), _p(slot_map), _p(q_start), _p(positions), _p(num), _p(nq), int(num_seqs), int(heads),
+                                         int(dim), int(vdim), _stream()), "matrix_memory_walk")
+
+
+def matrix_memory_finish(num: torch.Tensor, nq: torch.Tensor, gates: torch.Tensor, g: torch.Tensor, weight: torch.Tensor, eps: float,
+                         den_eps: float, out: torch.Tensor, heads: int, vdim: int) -> None:
+    """out [T, heads*vdim] = o / rms(o of the head) * weight * sigmoid(g) with o = num / (max(|nq|, exp(-m)) + den_eps)."""
+    _dev(num, nq, gates, g, weight, out)
+    T = num.shape[0]
+    assert g.stride(1) == 1 and tuple(g.shape) == (T, heads * vdim) and out.stride(1) == 1 and tuple(out.shape) == (T, heads * vdim)
+    assert weight.is_contiguous() and weight.numel() == heads * vdim
+    _check(lib().aien_matrix_memory_finish(_p(num), _p(nq), _p(gates), _p(g), dt(g), g.stride(0), _p(weight), dt(weight), float(eps), float(den_eps),
+                                           _p(out), dt(out), out.stride(0), T, int(heads), int(vdim), _stream()), "matrix_memory_finish")
+
+
+def matrix_memory_token_supports(dim: int, vdim: int) -> bool:
+    return bool(lib().aien_matrix_memory_token_supports(int(dim), int(vdim)))
+
+
+def matrix_memory_token(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, q_scale: float, z: torch.Tensor, i_off: int,
+                        f_off: int, bi: torch.Tensor, bf: torch.Tensor, cap: float, state: torch.Tensor, slot_map: torch.Tensor,
+                        q_start: torch.Tensor, positions: torch.Tensor, weight: torch.Tensor, eps: float, den_eps: float, out: torch.Tensor,
+                        num_seqs: int, heads: int, dim: int, vdim: int) -> None:
+    """Gates, recurrence, denominator, norm and gate in one kernel for a step in which every request brings one token."""
+    _dev(proj, z, bi, bf, weight, out)
+    _state_args(state, slot_map, q_start, positions)
+    assert proj.stride(1) == 1 and z.dtype == torch.float32 and z.stride(1) == 1 and out.stride(1) == 1
+    assert max(q_off, k_off) + heads * dim <= proj.shape[1] and max(v_off, g_off) + heads * vdim <= proj.shape[1]
+    assert max(i_off, f_off) + heads <= z.shape[1] and bi.dtype == torch.float32 and bf.dtype == torch.float32
+    assert state.shape[1] >= matrix_memory_state_floats(heads, dim, vdim) and weight.is_contiguous() and weight.numel() == heads * vdim
+    _check(lib().aien_matrix_memory_token(_p(proj), dt(proj), proj.stride(0), int(q_off), int(k_off), int(v_off), int(g_off), float(q_scale), _p(z),
+                                          z.stride(0), int(i_off), int(f_off), _p(bi), _p(bf), float(cap), _p(state), state.stride(0), _p(slot_map),
+                                          _p(q_start), _p(positions), _p(weight), dt(weight), float(eps), float(den_eps), _p(out), dt(out),
+                                          out.stride(0), int(num_seqs), int(heads), int(dim), int(vdim), _stream()), "matrix_memory_token")

@@ -12,7 +12,7 @@ import torch
 
 from .. import kernels as K
 from ..config.spec import LayerSpec, ModelSpec, PartSpec
-from ..parts.base import Prenormed, Block, CacheNeed, Mixer, NormedStream, RunBinding, ScaledSum, StepContext, StreamCopy, add_to_residual
+from ..parts.base import Prenormed, Block, CacheNeed, Mixer, NormedStream, RunBinding, ScaledSum, StepContext, StreamCopy, SumTerms, add_to_residual
 from ..registry import make_part, part_factory
 
 
@@ -196,11 +196,14 @@ class Decoder:
                     part.tie_embedding(self.embedding)
         if pending or waiting:
             raise RuntimeError("bind: some parts did not receive all their tensors")
+        for block in self.blocks:
+            block.finish_bind()
 
     # ------------------------------------------------------------------ sizes
     def layer_workspace_bytes(self, lim) -> int:
         head = lim.max_tokens * self.hidden_size * (4 + lim.itemsize) + 4096
-        return max(max(b.workspace_bytes(lim) for b in self.blocks), head) + (1 << 16)
+        enter = self.pass_input.workspace_bytes(lim) if self.pass_input is not None else 0      # taken ahead of the pass's first block
+        return max(max(b.workspace_bytes(lim) for b in self.blocks) + enter, head) + (1 << 16)
 
     def step_workspace_bytes(self, lim) -> int:
         n = self.streams * lim.max_tokens * self.hidden_size * 4 + 4096
@@ -233,9 +236,12 @@ class Decoder:
             ws.begin_layer()
             block = self.blocks[run.layer]
             if run.enter >= 0:
-                add_to_residual(ctx, x, delta)                  # the pass starts from the stream as it stands
-                delta = None
-                self.pass_input.forward(ctx, x, x0, run.enter)
+                if self.pass_input.takes_pending:
+                    delta = self.pass_input.forward(ctx, x, x0, run.enter, delta)
+                else:
+                    add_to_residual(ctx, x, delta)              # the pass starts from the stream as it stands
+                    delta = None
+                    self.pass_input.forward(ctx, x, x0, run.enter)
             if block.chains_norm:
                 # the norm that will take this block's result, so that the block's last product may work for it
                 nxt = self.blocks[runs[i + 1].layer].first_norm() if i + 1 < len(runs) else None
@@ -245,7 +251,7 @@ class Decoder:
         ws.end_layers()
         if isinstance(delta, (Prenormed, StreamCopy, NormedStream)):    # nothing is pending: the last block summed into the stream itself
             delta = None
-        if isinstance(delta, ScaledSum):                                # a pending sum that the row gather cannot take
+        if isinstance(delta, (ScaledSum, SumTerms)):                    # a pending sum that the row gather cannot take
             add_to_residual(ctx, x, delta)
             delta = None
         if num_rows > 0:

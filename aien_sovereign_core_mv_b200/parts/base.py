@@ -251,6 +251,19 @@ class ScaledSum:
 
 
 @dataclass
+class SumTerms:
+    """What a block whose sublayers share one input hands on: several branches still to be added to the stream.  A term
+    is (tensor [T, H] or parts [P, T, H], gate) and counts times sigmoid(gate[t]) (a float32 column of the step's tokens)
+    or, without a gate, as it is.  ``bias`` [H] is added for every token; with ``replace`` the sum takes the stream's
+    place instead of being added to it.  The next block of that kind makes the sum inside its first norm's kernel; every
+    other consumer calls ``add_to_residual``."""
+
+    terms: Tuple[Tuple[torch.Tensor, Optional[torch.Tensor]], ...]
+    bias: Optional[torch.Tensor] = None
+    replace: bool = False
+
+
+@dataclass
 class ResidualSink:
     """Offered to a part whose last product ends a residual branch: instead of returning the
     branch's output for the next norm to add, the product may add it to ``x`` itself and return a
@@ -317,6 +330,12 @@ class Position(Part):
 class Mixer(Part):
     takes_prenormed = False      # True: forward() accepts a Prenormed as h
     feeds_residual = False       # True: forward() accepts sink=ResidualSink and may return a Prenormed
+    takes_riders = False         # True: set_riders() may be called once, after bind()
+
+    def set_riders(self, weight: torch.Tensor) -> None:
+        """Rows [R, hidden] of a neighbour that reads the same h: they ride in this mixer's first product, and forward()
+        then returns (y, float32 [T, R] = h . weight^T)."""
+        raise NotImplementedError
 
     def cache_need(self) -> Optional[CacheNeed]:
         return None
@@ -331,6 +350,15 @@ class FeedForward(Part):
 
     def forward(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
+
+    def rider_rows(self) -> Optional[torch.Tensor]:
+        """The rows of a small product over h that may ride in a neighbour's product (``Mixer.takes_riders``), whose float32
+        result then comes as ``riders=`` of terms(); None: there are none."""
+        return None
+
+    def terms(self, ctx: StepContext, h: torch.Tensor, riders: Optional[torch.Tensor] = None):
+        """The branch as terms of a :class:`SumTerms`."""
+        return ((self.forward(ctx, h), None),)
 
     def pending_bias(self) -> Optional[torch.Tensor]:
         """A float32 vector [H] that belongs to the result of forward() and that the consumer of the branch adds with
@@ -371,6 +399,9 @@ def add_to_residual(ctx: StepContext, x: torch.Tensor, delta) -> None:
     from .. import kernels as K
     if delta is None or isinstance(delta, (Prenormed, StreamCopy, NormedStream)):
         return
+    if isinstance(delta, SumTerms):
+        K.sum_terms_rmsnorm(x, delta.terms, delta.bias, delta.replace, None, 0.0, None)
+        return
     if isinstance(delta, ScaledSum):
         K.scaled_add_rmsnorm(x, delta.delta, delta.vec, delta.bias, None, 0.0, None)
         return
@@ -391,6 +422,9 @@ class Block(Part):
 
     def workspace_bytes(self, lim: "StepLimits") -> int:
         return sum(p.workspace_bytes(lim) for p in self.parts().values())
+
+    def finish_bind(self) -> None:
+        """Called once when every part of the block has its tensors."""
 
     def first_norm(self) -> Optional[Norm]:
         """The norm that takes the previous block's result, if the block starts with one."""

@@ -7,7 +7,7 @@ import torch
 
 from ..registry import register_block
 from .. import kernels as K
-from .base import Block, FeedForward, Mixer, Norm, Part, Prenormed, RunBinding, ScaledSum, StepContext, StreamCopy, add_to_residual
+from .base import Block, FeedForward, Mixer, Norm, Part, Prenormed, RunBinding, ScaledSum, StepContext, StreamCopy, SumTerms, add_to_residual
 
 
 @register_block("prenorm")
@@ -197,3 +197,48 @@ class ScaledPreNormMixerBlock(ScaledPreNormBlock):
         if feed_forward is not None:
             raise ValueError("the block kind 'prenorm_scaled_mixer' takes no feed-forward")
         super().__init__(mixer, None, norm_in, None, residual_mult, layer_scale)
+
+
+@register_block("parallel")
+class ParallelBlock(Block):
+    """x <- x + (mixer(h) + ff(h)) with h = norm_in(x): both sublayers read one norm's output (a layer without a
+    feed-forward: x <- x + mixer(h)).  The branches stay pending (``SumTerms``) until the next norm's kernel adds them, in
+    float32.  Small rows of the feed-forward that read h (a router's) ride in the mixer's first product where the mixer
+    takes them.  The norm is an RMS norm with a plain weight."""
+
+    norm_slots = ("norm_in",)
+
+    def __init__(self, mixer: Mixer, feed_forward: Optional[FeedForward], norm_in: Norm):
+        if not hasattr(norm_in, "weight") or not hasattr(norm_in, "eps") or getattr(norm_in, "weight_offset", 0.0) != 0.0:
+            raise ValueError("the norm of a parallel block is an RMS norm with a plain weight")
+        self.mixer, self.feed_forward, self.norm_in = mixer, feed_forward, norm_in
+        self._riders = False
+
+    def parts(self):
+        out = {"norm_in": self.norm_in, "mixer": self.mixer}
+        if self.feed_forward is not None:
+            out["feed_forward"] = self.feed_forward
+        return out
+
+    def first_norm(self):
+        return self.norm_in
+
+    def finish_bind(self):
+        rows = self.feed_forward.rider_rows() if self.feed_forward is not None and self.mixer.takes_riders else None
+        if rows is not None:
+            self.mixer.set_riders(rows)
+            self._riders = True
+
+    def forward(self, ctx: StepContext, x: torch.Tensor, delta, run: RunBinding):
+        if not isinstance(delta, SumTerms):
+            add_to_residual(ctx, x, delta)             # whatever another kind of block left pending
+            delta = SumTerms(())
+        h = ctx.workspace.take(tuple(x.shape), ctx.dtype)
+        K.sum_terms_rmsnorm(x, delta.terms, delta.bias, delta.replace, self.norm_in.weight, self.norm_in.eps, h)
+        a, riders = self.mixer.forward(ctx, h, run), None
+        if self._riders:
+            a, riders = a
+        terms = ((a, None),)
+        if self.feed_forward is not None:
+            terms += tuple(self.feed_forward.terms(ctx, h, riders))
+        return SumTerms(terms)

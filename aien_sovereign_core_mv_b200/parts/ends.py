@@ -7,7 +7,7 @@ import torch
 
 from .. import kernels as K
 from ..registry import make_part, register_embedding, register_head, register_pass_input
-from .base import Embedding, Head, Part, StepContext
+from .base import Embedding, Head, Part, StepContext, SumTerms, add_to_residual
 from .linear import linear
 
 
@@ -128,6 +128,8 @@ class StepVectorInput(Part):
     embedding's output once more (``add_embedding``; every pass but the first), then the row t of ``steps`` [times,
     hidden] for every token.  The sums are float32."""
 
+    takes_pending = False          # True: forward() takes the pending sum and returns what is pending behind it
+
     def __init__(self, hidden_size: int, times: int, add_embedding: bool = True):
         self.hidden_size, self.times, self.add_embedding = int(hidden_size), int(times), bool(add_embedding)
         if self.times <= 0:
@@ -149,3 +151,49 @@ class StepVectorInput(Part):
         if not (0 <= t < self.times):
             raise ValueError(f"pass {t} of {self.times}")
         K.pass_input(x, embedded if (self.add_embedding and t > 0) else None, self.steps[t])
+
+
+@register_pass_input("step_projection")
+class StepProjectionInput(Part):
+    """Before pass t = 0, 1, ... of a repeated stretch of layers the stream x becomes W_in [x; e] + steps[t], e the embedding's
+    output: tensors ``in_proj`` [hidden, 2 hidden] (the stream's columns first) and ``steps`` [times, hidden].
+
+    The stream is float32 and the product's operands in a bfloat16 engine are not, so the stream enters it twice, as its
+    rounded value and as the rounded rest, each against the same columns of W_in: the product sees 16 bits of it.  The
+    result stays pending (``SumTerms`` that replaces the stream) with the pass's vector as its bias, so the next norm's
+    kernel writes the stream."""
+
+    takes_pending = True
+    wants_embedding = True
+
+    def __init__(self, hidden_size: int, times: int):
+        self.hidden_size, self.times = int(hidden_size), int(times)
+        if self.times <= 0:
+            raise ValueError(f"times {times!r} must be positive")
+        self.w_in: Optional[torch.Tensor] = None
+        self.steps: Optional[torch.Tensor] = None
+
+    def param_shapes(self):
+        H = self.hidden_size
+        return {"in_proj": ((H, 2 * H), "matrix"), "steps": ((self.times, H), "small")}
+
+    def bind(self, tensors):
+        w, H = tensors["in_proj"], self.hidden_size
+        self.w_in = torch.cat([w[:, :H], w[:, :H], w[:, H:]], dim=1).contiguous() if w.dtype == torch.bfloat16 else w.contiguous()
+        self.steps = tensors["steps"].contiguous()
+
+    def workspace_bytes(self, lim):
+        return lim.max_tokens * self.hidden_size * (3 * lim.itemsize + 4) + 4096 + K.PARTIALS_MAX_BYTES
+
+    def forward(self, ctx: StepContext, x: torch.Tensor, embedded: torch.Tensor, t: int, delta):
+        if not (0 <= t < self.times):
+            raise ValueError(f"pass {t} of {self.times}")
+        terms = ()
+        if isinstance(delta, SumTerms) and delta.bias is None and not delta.replace:
+            terms = delta.terms
+        else:
+            add_to_residual(ctx, x, delta)
+        rows = ctx.workspace.take((ctx.num_tokens, self.w_in.shape[1]), self.w_in.dtype)
+        K.pass_rows(x, terms, embedded, rows)
+        y = linear(ctx, rows, self.w_in, out_dtype=torch.float32, may_defer_sum=True)
+        return SumTerms(((y, None),), self.steps[t], True)

@@ -8,7 +8,7 @@ import torch
 from .. import kernels as K
 from ..registry import register_mixer
 from .base import CacheNeed, Mixer, Position, RunBinding, StepContext
-from .linear import linear
+from .linear import linear, stack_rows
 
 
 @register_mixer("latent_attention")
@@ -18,7 +18,8 @@ class LatentAttention(Mixer):
     rows; the first kv_rank, RMS-normed (weight ``dkv_norm``), are the latent c, the rest one rotated key part shared by
     all heads.  Per head the unrotated key is W_uk c and the value W_uv c; score = (q_unrot . k_unrot + q_rot . k_rot) *
     ``scale``; causal, optionally only the last ``window`` positions (the token itself included); optionally a learned
-    sink per head in the softmax denominator; W_o on the heads.  The rotation turns neighbouring pairs of the first
+    sink per head in the softmax denominator; optionally (``head_gate``) head h's output times sigmoid(W_g h)_h; W_o on the
+    heads.  The rotation turns neighbouring pairs of the first
     ``rotary_dim`` numbers of the rotated part (the position part's table).
 
     The cache keeps one row [c | k_rot] per token and nothing per head.  The kernels never build a head's keys or
@@ -29,7 +30,7 @@ class LatentAttention(Mixer):
 
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, value_dim: int, kv_rank: int, q_rank: int,
                  position: Position, scale: Optional[float] = None, window: int = 0, cache_window: Optional[int] = None,
-                 sink: bool = False, norm_eps: float = 1e-6, own_cache: bool = True):
+                 sink: bool = False, norm_eps: float = 1e-6, own_cache: bool = True, head_gate: bool = False):
         self.hidden_size, self.num_heads, self.head_dim, self.rot_dim = int(hidden_size), int(num_heads), int(head_dim), int(rot_dim)
         self.value_dim, self.kv_rank, self.q_rank = int(value_dim), int(kv_rank), int(q_rank)
         if min(self.num_heads, self.head_dim, self.value_dim, self.kv_rank, self.q_rank) <= 0 or self.rot_dim < 0:
@@ -46,6 +47,8 @@ class LatentAttention(Mixer):
         if self.window < 0 or (self.window == 0) != (self.cache_window == 0) or self.cache_window < self.window:
             raise ValueError("cache_window must cover window (0 for both: every earlier position is seen)")
         self.sink, self.norm_eps, self.own_cache = bool(sink), float(norm_eps), bool(own_cache)
+        self.head_gate = bool(head_gate)
+        self.side_rows, self.riders = (self.num_heads if self.head_gate else 0), 0     # rows of the first product behind the query latent
         self.q_head = self.head_dim + self.rot_dim
         self.row = self.kv_rank + self.rot_dim
         self.w_down = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = self.dq_norm = self.dkv_norm = self.sinks = None
@@ -60,13 +63,27 @@ class LatentAttention(Mixer):
             shapes.update({"dkv_proj": ((self.row, H), "matrix"), "dkv_norm": ((self.kv_rank,), "norm")})
         if self.sink:
             shapes["sink"] = ((n,), "vector")
+        if self.head_gate:
+            shapes["g_proj"] = ((n, H), "matrix")
         return shapes
 
+    takes_riders = True
+
+    def _stack(self, dq, side, dkv):
+        """Rows query latent | head gates and riders, filled up to whole vectors | key/value latent | shared key part."""
+        head = stack_rows([dq] + side, 8) if side else dq
+        self.side_rows = head.shape[0] - self.q_rank
+        self.w_down = stack_rows([head] + ([dkv] if dkv is not None else []))
+
+    def set_riders(self, weight):
+        w = self.w_down
+        gates = [w[self.q_rank:self.q_rank + self.num_heads]] if self.head_gate else []
+        dkv = w[self.q_rank + self.side_rows:] if self.own_cache else None
+        self.riders = weight.shape[0]
+        self._stack(w[:self.q_rank], gates + [weight], dkv)
+
     def bind(self, tensors):
-        rows = [tensors["dq_proj"]] + ([tensors["dkv_proj"]] if self.own_cache else [])
-        if len({t.dtype for t in rows}) > 1:
-            rows = [t.float() for t in rows]
-        self.w_down = torch.cat(rows, dim=0).contiguous()              # rows query latent | key/value latent | shared key part
+        self._stack(tensors["dq_proj"], [tensors["g_proj"]] if self.head_gate else [], tensors["dkv_proj"] if self.own_cache else None)
         self.w_uq, self.w_o = tensors["uq_proj"].contiguous(), tensors["o_proj"].contiguous()
         n = self.num_heads
         # per head [kv_rank, head_dim]: the matrix that takes a head's unrotated query to the latent
@@ -84,7 +101,7 @@ class LatentAttention(Mixer):
 
     def workspace_bytes(self, lim):
         n = self.num_heads
-        per_token = (self.q_rank + self.row) * 4 + self.q_rank * lim.itemsize + n * self.q_head * 4 + n * self.row * 4 \
+        per_token = (self.q_rank + self.side_rows + self.row) * 4 + self.q_rank * lim.itemsize + n * self.q_head * 4 + n * self.row * 4 \
             + n * self.kv_rank * lim.itemsize + n * self.value_dim * lim.itemsize + self.hidden_size * 4
         # the partial results of a step with few tiles: tokens * heads * ksplit rows, which latent_attention_tc_ksplit keeps
         # below 296 tiles' worth of 64 rows
@@ -99,12 +116,13 @@ class LatentAttention(Mixer):
         writes = run.writes and self.own_cache
         if run.writes and not self.own_cache:
             raise RuntimeError("a latent-attention layer without its own key/value projection was bound to write a cache")
-        w_down = self.w_down if writes else self.w_down[:self.q_rank]
+        kv_off = self.q_rank + self.side_rows
+        w_down = self.w_down if writes else self.w_down[:kv_off]
         d = linear(ctx, h, w_down, out_dtype=torch.float32)
         rot = self.position.rotary(ctx) if self.rotary_dim else None
         cos, sin, rdims = rot if rot is not None else (None, None, 0)
         cq = ws.take((T, self.q_rank), ctx.dtype)
-        K.latent_prepare(d, self.q_rank, self.dq_norm, self.norm_eps, cq, self.q_rank, self.kv_rank, self.rot_dim, rdims,
+        K.latent_prepare(d, self.q_rank, self.dq_norm, self.norm_eps, cq, kv_off, self.kv_rank, self.rot_dim, rdims,
                          self.dkv_norm, cos, sin, group.slot_map if writes else None, cache if writes else None)
         tc = K.latent_attention_tc_supports(cache.dtype, self.kv_rank, self.rot_dim) and ctx.dtype == torch.bfloat16
         # per head: unrotated | rotated part, before rotation; an operand of the tensor-core products where those run
@@ -124,5 +142,10 @@ class LatentAttention(Mixer):
             K.latent_attention(qf, cache, group.block_table, group.max_blocks, ctx.seq_of_token, ctx.positions, mixed, n, self.kv_rank,
                                self.rot_dim, group.page_size, self.window, self.scale, self.sinks)
         o = ws.take((T, n * self.value_dim), ctx.dtype)
-        K.head_project(mixed, self.kv_rank, 0, self.w_uv, o, self.value_dim, 0)
-        return linear(ctx, o, self.w_o, out_dtype=torch.float32, may_defer_sum=True)     # the branch norm adds partial products
+        K.head_project(mixed, self.kv_rank, 0, self.w_uv, o, self.value_dim, 0,
+                       gate=d[:, self.q_rank:self.q_rank + n] if self.head_gate else None)
+        y = linear(ctx, o, self.w_o, out_dtype=torch.float32, may_defer_sum=True)        # the consumer's norm adds partial products
+        if not self.riders:
+            return y
+        r0 = self.q_rank + (n if self.head_gate else 0)
+        return y, d[:, r0:r0 + self.riders]

@@ -63,6 +63,17 @@ def linear(ctx: StepContext, a: torch.Tensor, w: torch.Tensor, out_dtype: Option
     return out
 
 
+def stack_rows(rows, multiple: int = 1) -> torch.Tensor:
+    """Weights of products over one input as one matrix, rows one below the other; zero rows fill it up to a multiple of
+    ``multiple`` (products store whole vectors of a row then)."""
+    if len({t.dtype for t in rows}) > 1:
+        rows = [t.float() for t in rows]
+    pad = -sum(t.shape[0] for t in rows) % multiple
+    if pad:
+        rows = list(rows) + [rows[0].new_zeros((pad, rows[0].shape[1]))]
+    return torch.cat(list(rows), dim=0).contiguous()
+
+
 def _choose(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, M: int) -> str:
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         return "simple"

@@ -47,12 +47,8 @@ class SwiGLU(FeedForward):
     takes_prenormed = True
     feeds_residual = True
 
-    def forward(self, ctx: StepContext, h, sink: Optional[ResidualSink] = None):
-        if isinstance(h, Prenormed):
-            act = linear_prenormed(ctx, h, self.w_gate_up, epilogue=1) if self.group == 8 else None
-            if act is not None:
-                return linear_into_residual(ctx, act, self.w_down, sink) or linear(ctx, act, self.w_down, may_defer_sum=True)
-            h = h.materialise(ctx)
+    def hidden(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
+        """silu(h Wg^T) * (h Wu^T)."""
         act = ctx.workspace.take((ctx.num_tokens, self.intermediate_size), ctx.dtype)
         if self.group == 8 and h.shape[0] <= K.GEMV_ROUTE_ROWS and K.gemv_supports(h, self.w_gate_up, act):
             K.gemv(h, self.w_gate_up, act, epilogue=1)          # silu(gate)*up inside the product
@@ -61,6 +57,15 @@ class SwiGLU(FeedForward):
         else:
             gu = linear(ctx, h, self.w_gate_up)
             K.swiglu(gu, act, self.group)
+        return act
+
+    def forward(self, ctx: StepContext, h, sink: Optional[ResidualSink] = None):
+        if isinstance(h, Prenormed):
+            act = linear_prenormed(ctx, h, self.w_gate_up, epilogue=1) if self.group == 8 else None
+            if act is not None:
+                return linear_into_residual(ctx, act, self.w_down, sink) or linear(ctx, act, self.w_down, may_defer_sum=True)
+            h = h.materialise(ctx)
+        act = self.hidden(ctx, h)
         return linear_into_residual(ctx, act, self.w_down, sink) or linear(ctx, act, self.w_down, may_defer_sum=True)
 
 

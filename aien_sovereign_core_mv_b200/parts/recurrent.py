@@ -8,7 +8,7 @@ import torch
 from .. import kernels as K
 from ..registry import register_mixer
 from .base import CacheNeed, Mixer, RunBinding, StepContext
-from .linear import linear
+from .linear import linear, stack_rows
 
 
 @register_mixer("decay_linear_attention")
@@ -190,3 +190,78 @@ class GatedDeltaRule(Mixer):
         y = ctx.workspace.take((T, self.v_dim), ctx.dtype)
         K.grouped_gated_rmsnorm(o, proj[:, g_off:g_off + self.v_dim], self.norm_w, self.norm_eps, y, self.value_dim, "silu")
         return linear(ctx, y, self.w_o, out_dtype=torch.float32, may_defer_sum=True)
+
+
+@register_mixer("matrix_memory")
+class MatrixMemory(Mixer):
+    """A matrix memory with exponential gates (the mLSTM of xLSTM).  q = W_q h * head_dim^-1/2 and k = W_k h (heads x
+    ``head_dim``), v = W_v h (heads x ``value_dim``); per head a log input gate i = cap tanh((W_i h + i_bias) / cap) and a
+    log forget gate f = logsigmoid(cap tanh((W_f h + f_bias) / cap)), cap = ``gate_cap``.  With a running maximum m that
+    starts at 0: m_t = max(f + m, i); S <- e^(f + m - m_t) S + e^(i - m_t) k v^T, n the same with k alone;
+    o = S^T q / (max(|n . q|, e^(-m_t)) + ``denominator_eps``).  Each head's o is divided by its root mean square
+    (``norm_eps``), the heads together are multiplied by the weight ``norm`` and by sigmoid(W_g h) and projected by W_o.
+
+    One float32 state slot per request holds S, n and m; it starts from zeros.  Gates, m, the recurrence, the denominator and
+    the norm are float32 in both engine precisions.  One product makes q | k | v | g | i | f (with riders behind);
+    in steps with portions of prompts a bfloat16 engine makes q | k | v | g in bfloat16 and the rest in float32."""
+
+    takes_riders = True
+
+    def __init__(self, hidden_size: int, num_heads: int, head_dim: int, value_dim: int, gate_cap: float, norm_eps: float = 1e-6,
+                 denominator_eps: float = 1e-6, position=None):
+        self.hidden_size, self.num_heads, self.head_dim, self.value_dim = int(hidden_size), int(num_heads), int(head_dim), int(value_dim)
+        self.cap, self.norm_eps, self.den_eps = float(gate_cap), float(norm_eps), float(denominator_eps)
+        if min(self.num_heads, self.head_dim, self.value_dim) <= 0 or self.head_dim > 256:
+            raise ValueError(f"heads, head_dim and value_dim must be positive; head_dim {head_dim}: the kernels keep up to 256 rows of a state column")
+        if not self.cap > 0.0:
+            raise ValueError(f"gate_cap {gate_cap!r} must be positive")
+        self.qk_dim, self.v_dim = self.num_heads * self.head_dim, self.num_heads * self.value_dim
+        self.main = 2 * self.qk_dim + 2 * self.v_dim                    # q | k | v | g
+        self.riders, self.rows = 0, self.main + 2 * self.num_heads
+        self.w_in = self.w_o = self.norm_w = self.b_i = self.b_f = None
+
+    def param_shapes(self):
+        H, n = self.hidden_size, self.num_heads
+        return {"q_proj": ((self.qk_dim, H), "matrix"), "k_proj": ((self.qk_dim, H), "matrix"), "v_proj": ((self.v_dim, H), "matrix"),
+                "g_proj": ((self.v_dim, H), "matrix"), "o_proj": ((H, self.v_dim), "matrix"), "norm": ((self.v_dim,), "norm"),
+                "i_proj": ((n, H), "matrix"), "i_bias": ((n,), "small"), "f_proj": ((n, H), "matrix"), "f_bias": ((n,), "open_gate")}
+
+    def bind(self, tensors):
+        self.w_in = stack_rows([tensors[k] for k in ("q_proj", "k_proj", "v_proj", "g_proj", "i_proj", "f_proj")], 8)
+        self.rows = self.w_in.shape[0]
+        self.w_o, self.norm_w = tensors["o_proj"].contiguous(), tensors["norm"].contiguous()
+        self.b_i, self.b_f = tensors["i_bias"].float().contiguous(), tensors["f_bias"].float().contiguous()
+
+    def set_riders(self, weight):
+        self.riders = weight.shape[0]
+        self.w_in = stack_rows([self.w_in[:self.main + 2 * self.num_heads], weight], 8)
+        self.rows = self.w_in.shape[0]
+
+    def cache_need(self):
+        return CacheNeed("state", state_shape=(K.matrix_memory_state_floats(self.num_heads, self.head_dim, self.value_dim),), state_dtype="float32")
+
+    def workspace_bytes(self, lim):
+        n = self.num_heads
+        return lim.max_tokens * ((self.rows + self.v_dim + 4 * n) * 4 + self.v_dim * lim.itemsize + self.hidden_size * 4) + 16384 + K.PARTIALS_MAX_BYTES
+
+    def forward(self, ctx: StepContext, h: torch.Tensor, run: RunBinding):
+        T, n, D, V = ctx.num_tokens, self.num_heads, self.head_dim, self.value_dim
+        ws = ctx.workspace
+        group = ctx.groups[run.group]
+        state, slots = group.storage["state"][run.slot], group.slot_map
+        k0, v0, g0, m0 = self.qk_dim, 2 * self.qk_dim, 2 * self.qk_dim + self.v_dim, self.main
+        q_scale = D ** -0.5
+        proj = linear(ctx, h, self.w_in, out_dtype=torch.float32)
+        z = proj[:, m0:]
+        y = ws.take((T, self.v_dim), ctx.dtype)
+        if ctx.decode_only and K.matrix_memory_token_supports(D, V):
+            K.matrix_memory_token(proj, 0, k0, v0, g0, q_scale, z, 0, n, self.b_i, self.b_f, self.cap, state, slots, ctx.q_start, ctx.positions,
+                                  self.norm_w, self.norm_eps, self.den_eps, y, ctx.num_seqs, n, D, V)
+        else:
+            gates = ws.take((T, 3 * n), torch.float32)
+            K.matrix_memory_gates(z, 0, n, self.b_i, self.b_f, self.cap, state, slots, ctx.q_start, ctx.positions, gates, ctx.num_seqs, n, D, V)
+            num, nq = ws.take((T, self.v_dim), torch.float32), ws.take((T, n), torch.float32)
+            K.matrix_memory_walk(proj, 0, k0, v0, q_scale, gates, state, slots, ctx.q_start, ctx.positions, num, nq, ctx.num_seqs, n, D, V)
+            K.matrix_memory_finish(num, nq, gates, proj[:, g0:g0 + self.v_dim], self.norm_w, self.norm_eps, self.den_eps, y, n, V)
+        out = linear(ctx, y, self.w_o, out_dtype=torch.float32, may_defer_sum=True)
+        return (out, z[:, 2 * n:2 * n + self.riders]) if self.riders else out

@@ -31,7 +31,7 @@ def random_tensor(name: str, shape: Tuple[int, ...], kind: str, seed: int,
     (a vector of scales stored around zero), "vector" (free numbers of order one, e.g. softmax sinks), "fraction"
     (numbers in [0, 1), e.g. a mixing weight), "near_identity" (a square matrix: the identity plus N(0, 0.1)), "small"
     (N(0, 0.1): biases), "log_rate" (U(-4, 1): logarithms of decay rates) or "rate_bias" (U(-4.5, -1): what a softplus
-    turns into a small step size)."""
+    turns into a small step size) or "open_gate" (U(3, 6): the bias of a gate that mostly stays open)."""
     g = torch.Generator(device=device)
     g.manual_seed(_tensor_seed(seed, name))
     if kind == "norm":
@@ -46,6 +46,8 @@ def random_tensor(name: str, shape: Tuple[int, ...], kind: str, seed: int,
         t = torch.rand(shape, generator=g, device=device, dtype=torch.float32) * 5.0 - 4.0
     elif kind == "rate_bias":
         t = torch.rand(shape, generator=g, device=device, dtype=torch.float32) * 3.5 - 4.5
+    elif kind == "open_gate":
+        t = torch.rand(shape, generator=g, device=device, dtype=torch.float32) * 3.0 + 3.0
     elif kind == "fraction":
         t = torch.rand(shape, generator=g, device=device, dtype=torch.float32)
     elif kind == "near_identity":
