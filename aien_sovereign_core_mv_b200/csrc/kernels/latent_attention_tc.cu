@@ -1,5 +1,6 @@
 // Attention over cached latent rows on the tensor cores (bfloat16 engine): the same result as the plain kernel in
-// latent_attention.cu, for latent sizes of 64, 128, 256 or 512 and a rotated part that is a multiple of 16.
+// latent_attention.cu, for latents of up to 512 numbers and rotated parts that are multiples of 8.  A latent that is not
+// 64, 128, 256 or 512 numbers long runs in the next of these sizes: its rows are filled up with zeros in shared memory.
 //
 // A cached row [c | k_rot] serves every head as key and (its first R numbers) as value, so the rows of the score
 // product are (token, head) pairs: the queries of a request's portion, laid out [token][head][R + rot], are one
@@ -16,6 +17,9 @@
 namespace aien {
 
 constexpr int LX_BM = 64, LX_BN = 64, LX_PSTR = LX_BN + 8;
+
+// Numbers a row of D numbers takes in shared memory (without its padding): whole k-steps of 16, and all R columns of the sum.
+__host__ __device__ __forceinline__ int lx_row_width(int R, int D) { return (D + 15) / 16 * 16 > R ? (D + 15) / 16 * 16 : R; }
 
 __device__ __forceinline__ void lx_cp_async16(uint32_t dst, const void* src, bool valid) {
     const int n = valid ? 16 : 0;
@@ -51,12 +55,13 @@ __global__ void __launch_bounds__(WARPS * 32, SLABS == 1 ? 2 : 1)
 latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ cache,
                            const int* __restrict__ block_table, int max_blocks, const int* __restrict__ q_start,
                            const int* __restrict__ positions, int S, __nv_bfloat16* __restrict__ out,
-                           int H, int rd, int page_size, int window, float scale_log2e, const float* __restrict__ sinks,
+                           int H, int r_lat, int rd, int page_size, int window, float scale_log2e, const float* __restrict__ sinks,
                            int ksplit, float* __restrict__ part_o, float* __restrict__ part_ml) {
     constexpr int BM = SLABS * 16, PARTS = WARPS / SLABS, KP = LX_BN / PARTS, NJ = KP / 8, CHP = R / PARTS, THREADS = WARPS * 32;
     constexpr int DT = CHP / 8;                  // n8 tiles of this warp's share of the channels
     static_assert(DT >= 2 && DT % 2 == 0, "a warp's share of the latent must be whole pairs of n8 tiles");
-    const int D = R + rd, STR = D + 8, CH = D / 8, KS = D / 16;
+    // r_lat <= R: the latent's own size; a row's D numbers are read, the rest of its width in shared memory is zeros
+    const int D = r_lat + rd, CH = D / 8, KS = (D + 15) / 16, W = lx_row_width(R, D), CHW = W / 8, STR = W + 8;
     extern __shared__ __align__(16) uint8_t lx_smem[];
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(lx_smem);          // [BM][STR]
     __nv_bfloat16* Ks = Qs + BM * STR;                                      // [64][STR]
@@ -90,10 +95,10 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
     const int g = lane >> 2, c = lane & 3;
 
     const __nv_bfloat16* qbase = q + ((size_t)qs * H + row0) * D;
-    for (int idx = tid; idx < BM * CH; idx += THREADS) {
-        const int r = idx / CH, ch = idx - r * CH;
-        const bool valid = r < nrows;
-        lx_cp_async16(Qs_u + (uint32_t)(r * STR + ch * 8) * 2, qbase + (size_t)(valid ? r : 0) * D + ch * 8, valid);
+    for (int idx = tid; idx < BM * CHW; idx += THREADS) {
+        const int r = idx / CHW, ch = idx - r * CHW;
+        const bool valid = r < nrows && ch < CH;
+        lx_cp_async16(Qs_u + (uint32_t)(r * STR + ch * 8) * 2, qbase + (valid ? (size_t)r * D + ch * 8 : 0), valid);
     }
     lx_cp_async_commit();
 
@@ -115,8 +120,8 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
         __syncthreads();
     }
     for (int kb = kb_begin + (int)blockIdx.y; kb <= kb_end; kb += ksplit) {
-        for (int idx = tid; idx < LX_BN * CH; idx += THREADS) {
-            const int r = idx / CH, ch = idx - r * CH;
+        for (int idx = tid; idx < LX_BN * CHW; idx += THREADS) {
+            const int r = idx / CHW, ch = idx - r * CHW;
             const int key = kb * LX_BN + r;
             bool valid = key >= first && key <= pos_hi;
             long slot = 0;
@@ -125,7 +130,8 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
                 valid = page >= 0;
                 slot = (long)page * page_size + key % page_size;
             }
-            lx_cp_async16(Ks_u + (uint32_t)(r * STR + ch * 8) * 2, cache + (size_t)(valid ? slot : 0) * D + ch * 8, valid);
+            const bool copy = valid && ch < CH;
+            lx_cp_async16(Ks_u + (uint32_t)(r * STR + ch * 8) * 2, cache + (copy ? (size_t)slot * D + ch * 8 : 0), copy);
             if (ch == 0) key_there[r] = valid ? 1 : 0;
         }
         lx_cp_async_commit();
@@ -250,9 +256,10 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
                 part_ml[slot * 2] = m_run[r];
                 part_ml[slot * 2 + 1] = l_run[r];
             }
-            float* dst = part_o + slot * R + half * CHP;
+            float* dst = part_o + slot * r_lat + half * CHP;
 #pragma unroll
-            for (int d = 0; d < DT; ++d) *reinterpret_cast<float2*>(dst + d * 8 + 2 * c) = make_float2(o[d][2 * r], o[d][2 * r + 1]);
+            for (int d = 0; d < DT; ++d)
+                if (half * CHP + d * 8 < r_lat) *reinterpret_cast<float2*>(dst + d * 8 + 2 * c) = make_float2(o[d][2 * r], o[d][2 * r + 1]);
         }
         return;
     }
@@ -282,16 +289,15 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
             l_run[r] = l_run[r] * corr + exp2f(sk - mn);
         }
         const float inv = l_run[r] > 0.f ? corr / l_run[r] : 0.f;
-        __nv_bfloat16* dst = out + ((size_t)qs * H + row0 + row) * R + half * CHP;
+        __nv_bfloat16* dst = out + ((size_t)qs * H + row0 + row) * r_lat + half * CHP;
 #pragma unroll
         for (int d = 0; d < DT; ++d)
-            *reinterpret_cast<uint32_t*>(dst + d * 8 + 2 * c) = lx_pack(o[d][2 * r] * inv, o[d][2 * r + 1] * inv);
+            if (half * CHP + d * 8 < r_lat) *reinterpret_cast<uint32_t*>(dst + d * 8 + 2 * c) = lx_pack(o[d][2 * r] * inv, o[d][2 * r + 1] * inv);
     }
 }
 
 // out[row] = sum_s 2^(m_s - M) o_s / (sum_s 2^(m_s - M) l_s + 2^(sink - M)), M = max over the row's parts and the sink
-template <int R>
-__global__ void latent_attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int ksplit,
+__global__ void latent_attention_merge_kernel(int R, const float* __restrict__ part_o, const float* __restrict__ part_ml, int ksplit,
                                               const float* __restrict__ sinks, int H, __nv_bfloat16* __restrict__ out) {
     const size_t row = blockIdx.x;
     const float sk = sinks != nullptr ? sinks[row % H] * 1.4426950408889634f : -INFINITY;
@@ -315,20 +321,20 @@ __global__ void latent_attention_merge_kernel(const float* __restrict__ part_o, 
 
 template <int R, int SLABS, int WARPS>
 static int launch_latent_tc(const void* q, const void* cache, const int* bt, int max_blocks, const int* q_start, const int* positions,
-                            int T, int S, void* out, int H, int rd, int page_size, int window, float scale, const float* sinks,
+                            int T, int S, void* out, int H, int r_lat, int rd, int page_size, int window, float scale, const float* sinks,
                             int ksplit, float* part_o, float* part_ml, cudaStream_t stream) {
-    const int D = R + rd;
+    const int D = r_lat + rd;
     constexpr int BM = SLABS * 16;
-    const size_t smem = (size_t)(BM + LX_BN) * (D + 8) * 2 + (size_t)BM * LX_PSTR * 2 + (size_t)WARPS * 16 * sizeof(float);
+    const size_t smem = (size_t)(BM + LX_BN) * (lx_row_width(R, D) + 8) * 2 + (size_t)BM * LX_PSTR * 2 + (size_t)WARPS * 16 * sizeof(float);
     if (smem > 227 * 1024) return AIEN_E_SHAPE;
     auto kern = latent_attention_tc_kernel<R, SLABS, WARPS>;
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return AIEN_E_STATE;
     const long tiles = ((long)T * H) / BM + S;
     kern<<<dim3((unsigned)tiles, ksplit), WARPS * 32, smem, stream>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, bt, max_blocks, q_start,
-                                                                     positions, S, (__nv_bfloat16*)out, H, rd, page_size, window,
+                                                                     positions, S, (__nv_bfloat16*)out, H, r_lat, rd, page_size, window,
                                                                      scale * 1.4426950408889634f, sinks, ksplit, part_o, part_ml);
     if (ksplit > 1)
-        latent_attention_merge_kernel<R><<<dim3((unsigned)((long)T * H)), 128, 0, stream>>>(part_o, part_ml, ksplit, sinks, H, (__nv_bfloat16*)out);
+        latent_attention_merge_kernel<<<dim3((unsigned)((long)T * H)), 128, 0, stream>>>(r_lat, part_o, part_ml, ksplit, sinks, H, (__nv_bfloat16*)out);
     return launch_status();
 }
 
@@ -411,9 +417,11 @@ head_project_tc_kernel(const __nv_bfloat16* __restrict__ A, long lda, long a_hea
 
 using namespace aien;
 
+static int lx_padded_rank(int kv_rank) { return kv_rank <= 64 ? 64 : (kv_rank <= 128 ? 128 : (kv_rank <= 256 ? 256 : 512)); }
+
 AIEN_API int aien_latent_attention_tc_supports(int kv_rank, int rot_dim) {
-    if (!(kv_rank == 64 || kv_rank == 128 || kv_rank == 256 || kv_rank == 512) || rot_dim < 0 || (rot_dim & 15)) return 0;
-    const size_t smem = (size_t)(LX_BM + LX_BN) * (kv_rank + rot_dim + 8) * 2 + (size_t)LX_BM * LX_PSTR * 2 + 16 * 16 * sizeof(float);
+    if (kv_rank <= 0 || kv_rank > 512 || (kv_rank & 7) || rot_dim < 0 || (rot_dim & 7)) return 0;
+    const size_t smem = (size_t)(LX_BM + LX_BN) * (lx_row_width(lx_padded_rank(kv_rank), kv_rank + rot_dim) + 8) * 2 + (size_t)LX_BM * LX_PSTR * 2 + 16 * 16 * sizeof(float);
     return smem <= 227 * 1024 ? 1 : 0;
 }
 
@@ -421,7 +429,7 @@ AIEN_API int aien_latent_attention_tc_supports(int kv_rank, int rot_dim) {
 // The step's T tokens are the portions q_start[s] .. q_start[s + 1] of S requests; positions[t] is token t's position.
 // ksplit > 1: the key blocks of every tile are dealt out to ksplit CTAs (for steps with few tiles); part_o (float32,
 // T * H * ksplit * kv_rank) and part_ml (float32, T * H * ksplit * 2) hold their partial results for the merging launch.
-// small_tiles != 0: tiles of 16 rows instead of 64 (steps in which every request brings one token), for latents of 128 and more.
+// small_tiles != 0: tiles of 16 rows instead of 64 (steps in which every request brings one token), for latents of more than 64.
 AIEN_API int aien_latent_attention_tc(const void* q, const void* cache, const int* block_table, int max_blocks, const int* q_start,
                                       const int* positions, void* out, int T, int S, int H, int kv_rank, int rot_dim, int page_size,
                                       int window, float scale, const float* sinks, int ksplit, float* part_o, float* part_ml,
@@ -430,11 +438,12 @@ AIEN_API int aien_latent_attention_tc(const void* q, const void* cache, const in
     if (H <= 0 || page_size <= 0 || window < 0 || !aien_latent_attention_tc_supports(kv_rank, rot_dim)) return AIEN_E_SHAPE;
     if (((uintptr_t)q & 15) || ((uintptr_t)cache & 15) || ((uintptr_t)out & 3)) return AIEN_E_ALIGN;
     if (ksplit < 1 || ksplit > 65535 || (ksplit > 1 && (part_o == nullptr || part_ml == nullptr || ((uintptr_t)part_o & 7)))) return AIEN_E_SHAPE;
+    const int padded = lx_padded_rank(kv_rank);
 #define LX_CASE(RV, SL)                                                                                                          \
-    if (kv_rank == RV)                                                                                                           \
-        return launch_latent_tc<RV, SL, (SL == 4 ? 16 : 8)>(q, cache, block_table, max_blocks, q_start, positions, T, S, out, H, rot_dim, page_size,  \
+    if (padded == RV)                                                                                                            \
+        return launch_latent_tc<RV, SL, (SL == 4 ? 16 : 8)>(q, cache, block_table, max_blocks, q_start, positions, T, S, out, H, kv_rank, rot_dim, page_size,  \
                                         window, scale, sinks, ksplit, part_o, part_ml, stream);
-    if (small_tiles && kv_rank >= 128) {                   // tiles of 16 rows: a latent of 64 would leave a warp half a pair of n8 tiles
+    if (small_tiles && padded >= 128) {                    // tiles of 16 rows: a latent of 64 would leave a warp half a pair of n8 tiles
         LX_CASE(128, 1) LX_CASE(256, 1) LX_CASE(512, 1)
     }
     LX_CASE(64, 4) LX_CASE(128, 4) LX_CASE(256, 4) LX_CASE(512, 4)

@@ -1,6 +1,6 @@
 // A matrix memory with exponential gates (the mLSTM recurrence).  Per head, with log gates i (input) and f (forget),
 // a running maximum m that starts at 0, S [dim, vdim], n [dim]:
-//     m_t = max(f + m_(t-1), i)      keep = exp(f + m_(t-1) - m_t)      take = exp(i - m_t)
+//     m_t = max(f + m_(t-1), i)      keep = exp(f - (m_t - m_(t-1)))      take = exp(i - m_t)
 //     S_t = keep S_(t-1) + take k v^T      n_t = keep n_(t-1) + take k
 //     o_t = S_t^T q / (max(|n_t . q|, exp(-m_t)) + eps_den),      q already times dim^(-1/2)
 // and then y = o / rms(o of the head) * w * sigmoid(g).  The log gates are i = cap tanh((z_i + b_i) / cap) and
@@ -33,7 +33,7 @@ __device__ __forceinline__ size_t mm_n_off(MmSizes z) { return (size_t)z.H * z.D
 __device__ __forceinline__ size_t mm_m_off(MmSizes z) { return mm_n_off(z) + (size_t)z.H * z.D; }
 
 // ---------------------------------------------------------------- gates and the running maximum
-// gates [T, 3 * H]: log keep = f + m_(t-1) - m_t, then take = exp(i - m_t), then m_t.  One CTA per (request, head), 32 tokens a
+// gates [T, 3 * H]: log keep = f - (m_t - m_(t-1)), then take = exp(i - m_t), then m_t.  One CTA per (request, head), 32 tokens a
 // warp: the map of a run of tokens on m is m -> max(m + a, b), so the warps scan their own runs, the runs' maps follow one
 // another from the state's m, and every token gets its m from its run's start.  The slot's m is rewritten at the end.
 __global__ void __launch_bounds__(1024)
@@ -75,7 +75,7 @@ matrix_memory_gates_kernel(const float* __restrict__ z, long ldz, int i_off, int
         if (lane == 0) mp = m_start;
         if (in) {
             float* g = gates + (size_t)t * 3 * H + h;
-            g[0] = lf + mp - mt;
+            g[0] = lf - (mt - mp);          // exact to the last bit of lf while m only decays: m is far larger than lf
             g[H] = expf(li - mt);
             g[2 * H] = mt;
         }
@@ -206,7 +206,7 @@ matrix_memory_token_kernel(const TP* __restrict__ proj, long ld, int q_off, int 
     const float li = mm_input_gate(z[(size_t)t * ldz + i_off + h] + bi[h], cap);
     const float lf = mm_forget_gate(z[(size_t)t * ldz + f_off + h] + bf[h], cap);
     const float m1 = fmaxf(lf + m0, li);
-    const float keep = expf(lf + m0 - m1), take = expf(li - m1);
+    const float keep = expf(lf - (m1 - m0)), take = expf(li - m1);
     float nqp = 0.f;
     for (int d = tid; d < D; d += MT_THREADS) {
         const float q = to_f(row[q_off + h * D + d]) * q_scale, k = to_f(row[k_off + h * D + d]) * take;

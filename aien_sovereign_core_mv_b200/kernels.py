@@ -202,6 +202,8 @@ def _declare(l: ctypes.CDLL) -> None:
         "aien_matrix_memory_walk": [P, I, L, I, I, I, F, P, P, c_size_t, P, P, P, P, P, I, I, I, I, P],
         "aien_matrix_memory_finish": [P, P, P, P, I, L, P, I, F, F, P, I, L, I, I, I, P],
         "aien_matrix_memory_token_supports": [I, I],
+        "aien_matrix_memory_chunks_supports": [I, I],
+        "aien_matrix_memory_chunked": [P, L, I, I, I, I, F, P, P, c_size_t, P, P, P, P, I, F, F, P, L, P, I, I, I, I, I, P],
         "aien_matrix_memory_token": [P, I, L, I, I, I, I, F, P, L, I, I, P, P, F, P, c_size_t, P, P, P, P, I, F, F, P, I, L, I, I, I, I, P],
         "aien_rope_halves_value_write": [P, L, I, I, I, I, I, I, I, P, P, I, P, P, I, L, P, P, I, I, P],
     }
@@ -1471,7 +1473,7 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Te
 
 
 def latent_attention_tc_supports(dtype: torch.dtype, kv_rank: int, rot_dim: int) -> bool:
-    """Whether the tensor-core kernel takes this case: bfloat16, a latent of 64 / 128 / 256 / 512, a rotated part that is a multiple of 16."""
+    """Whether the tensor-core kernel takes this case: bfloat16, a latent of up to 512 numbers and a rotated part, both multiples of 8."""
     return _LATENT_IMPL != "plain" and dtype == torch.bfloat16 and bool(lib().aien_latent_attention_tc_supports(int(kv_rank), int(rot_dim)))
 
 
@@ -1484,7 +1486,7 @@ def latent_attention_tc(q: torch.Tensor, cache: torch.Tensor, block_table: torch
     table), each portion's positions counting up from positions[q_start[s]].  ``ksplit`` > 1 deals the key blocks of every
     tile out to that many CTAs and merges their results in a second launch (steps with few tiles); ``scratch`` is then
     float32 with ``latent_attention_tc_scratch(T, heads, kv_rank, ksplit)`` numbers.  ``small_tiles``: tiles of 16 rows
-    instead of 64, for steps in which every request brings one token (latents of 128 and more)."""
+    instead of 64, for steps in which every request brings one token (latents of more than 64)."""
     _dev(q, cache, block_table, q_start, positions, out, sinks)
     T, D = q.shape[0], kv_rank + rot_dim
     assert q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
@@ -1514,7 +1516,7 @@ def latent_attention_tc_scratch(num_tokens: int, heads: int, kv_rank: int, kspli
 
 def latent_attention_tc_small_tiles(decode_only: bool, kv_rank: int) -> bool:
     """Whether a step takes the tiles of 16 rows: every request brings one token, and the latent is wide enough."""
-    return bool(decode_only) and kv_rank >= 128
+    return bool(decode_only) and kv_rank > 64
 
 
 def latent_attention_tc_ksplit(num_tokens: int, num_seqs: int, heads: int, max_ctx: int, window: int, small_tiles: bool = False) -> int:
@@ -2128,3 +2130,34 @@ def matrix_memory_token(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, 
                                           z.stride(0), int(i_off), int(f_off), _p(bi), _p(bf), float(cap), _p(state), state.stride(0), _p(slot_map),
                                           _p(q_start), _p(positions), _p(weight), dt(weight), float(eps), float(den_eps), _p(out), dt(out),
                                           out.stride(0), int(num_seqs), int(heads), int(dim), int(vdim), _stream()), "matrix_memory_token")
+
+
+_MATRIX_MEMORY_IMPL = __import__("os").environ.get("AIEN_B200_MATRIX_MEMORY", "chunks").strip().lower()     # "chunks" | "walk": pins the plain form
+
+
+def matrix_memory_chunks_supports(dtype: torch.dtype, dim: int, vdim: int) -> bool:
+    """Whether portions may take the chunked tensor-core form: bfloat16, dim and vdim multiples of 16 up to 256."""
+    return _MATRIX_MEMORY_IMPL != "walk" and dtype == torch.bfloat16 and bool(lib().aien_matrix_memory_chunks_supports(int(dim), int(vdim)))
+
+
+def matrix_memory_chunks_scratch(num_tokens: int, num_seqs: int, heads: int, dim: int, vdim: int) -> int:
+    """float32 numbers the chunked form needs: a state and a decay for every chunk of 64 tokens and head, at most T / 64 + S chunks."""
+    return (num_tokens // 64 + num_seqs) * heads * (dim * vdim + dim + 1)
+
+
+def matrix_memory_chunked(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, q_scale: float, gates: torch.Tensor, state: torch.Tensor,
+                          slot_map: torch.Tensor, q_start: torch.Tensor, positions: torch.Tensor, weight: torch.Tensor, eps: float, den_eps: float,
+                          out: torch.Tensor, scratch: torch.Tensor, num_seqs: int, heads: int, dim: int, vdim: int) -> None:
+    """matrix_memory_walk and matrix_memory_finish for portions, chunks of 64 tokens side by side: proj and out bfloat16."""
+    _dev(proj, gates, weight, out, scratch)
+    _state_args(state, slot_map, q_start, positions)
+    T = proj.shape[0]
+    assert proj.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and proj.stride(1) == 1 and out.stride(1) == 1
+    assert max(q_off, k_off) + heads * dim <= proj.shape[1] and max(v_off, g_off) + heads * vdim <= proj.shape[1]
+    assert gates.is_contiguous() and tuple(gates.shape) == (T, 3 * heads) and state.shape[1] >= matrix_memory_state_floats(heads, dim, vdim)
+    assert out.shape[0] == T and out.shape[1] == heads * vdim and weight.is_contiguous() and weight.numel() == heads * vdim
+    assert scratch.dtype == torch.float32 and scratch.is_contiguous() and scratch.numel() >= matrix_memory_chunks_scratch(T, num_seqs, heads, dim, vdim)
+    _check(lib().aien_matrix_memory_chunked(_p(proj), proj.stride(0), int(q_off), int(k_off), int(v_off), int(g_off), float(q_scale), _p(gates),
+                                            _p(state), state.stride(0), _p(slot_map), _p(q_start), _p(positions), _p(weight), dt(weight), float(eps),
+                                            float(den_eps), _p(out), out.stride(0), _p(scratch), T, int(num_seqs), int(heads), int(dim), int(vdim),
+                                            _stream()), "matrix_memory_chunked")

@@ -242,7 +242,8 @@ class MatrixMemory(Mixer):
 
     def workspace_bytes(self, lim):
         n = self.num_heads
-        return lim.max_tokens * ((self.rows + self.v_dim + 4 * n) * 4 + self.v_dim * lim.itemsize + self.hidden_size * 4) + 16384 + K.PARTIALS_MAX_BYTES
+        return lim.max_tokens * ((self.rows + self.v_dim + 4 * n) * 4 + self.v_dim * lim.itemsize + self.hidden_size * 4) + 16384 + K.PARTIALS_MAX_BYTES \
+            + 4 * K.matrix_memory_chunks_scratch(lim.max_tokens, lim.max_seqs, n, self.head_dim, self.value_dim)
 
     def forward(self, ctx: StepContext, h: torch.Tensor, run: RunBinding):
         T, n, D, V = ctx.num_tokens, self.num_heads, self.head_dim, self.value_dim
@@ -251,17 +252,26 @@ class MatrixMemory(Mixer):
         state, slots = group.storage["state"][run.slot], group.slot_map
         k0, v0, g0, m0 = self.qk_dim, 2 * self.qk_dim, 2 * self.qk_dim + self.v_dim, self.main
         q_scale = D ** -0.5
-        proj = linear(ctx, h, self.w_in, out_dtype=torch.float32)
-        z = proj[:, m0:]
+        gate_args = (0, n, self.b_i, self.b_f, self.cap, state, slots, ctx.q_start, ctx.positions)
         y = ws.take((T, self.v_dim), ctx.dtype)
-        if ctx.decode_only and K.matrix_memory_token_supports(D, V):
-            K.matrix_memory_token(proj, 0, k0, v0, g0, q_scale, z, 0, n, self.b_i, self.b_f, self.cap, state, slots, ctx.q_start, ctx.positions,
-                                  self.norm_w, self.norm_eps, self.den_eps, y, ctx.num_seqs, n, D, V)
-        else:
+        if not ctx.decode_only and self.main % 8 == 0 and K.matrix_memory_chunks_supports(ctx.dtype, D, V):
+            proj = linear(ctx, h, self.w_in[:m0])
+            z = linear(ctx, h, self.w_in[m0:], out_dtype=torch.float32)
             gates = ws.take((T, 3 * n), torch.float32)
-            K.matrix_memory_gates(z, 0, n, self.b_i, self.b_f, self.cap, state, slots, ctx.q_start, ctx.positions, gates, ctx.num_seqs, n, D, V)
-            num, nq = ws.take((T, self.v_dim), torch.float32), ws.take((T, n), torch.float32)
-            K.matrix_memory_walk(proj, 0, k0, v0, q_scale, gates, state, slots, ctx.q_start, ctx.positions, num, nq, ctx.num_seqs, n, D, V)
-            K.matrix_memory_finish(num, nq, gates, proj[:, g0:g0 + self.v_dim], self.norm_w, self.norm_eps, self.den_eps, y, n, V)
+            K.matrix_memory_gates(z, *gate_args, gates, ctx.num_seqs, n, D, V)
+            scratch = ws.take((K.matrix_memory_chunks_scratch(T, ctx.num_seqs, n, D, V),), torch.float32)
+            K.matrix_memory_chunked(proj, 0, k0, v0, g0, q_scale, gates, state, slots, ctx.q_start, ctx.positions, self.norm_w, self.norm_eps,
+                                    self.den_eps, y, scratch, ctx.num_seqs, n, D, V)
+        else:
+            proj = linear(ctx, h, self.w_in, out_dtype=torch.float32)
+            z = proj[:, m0:]
+            if ctx.decode_only and K.matrix_memory_token_supports(D, V):
+                K.matrix_memory_token(proj, 0, k0, v0, g0, q_scale, z, *gate_args, self.norm_w, self.norm_eps, self.den_eps, y, ctx.num_seqs, n, D, V)
+            else:
+                gates = ws.take((T, 3 * n), torch.float32)
+                K.matrix_memory_gates(z, *gate_args, gates, ctx.num_seqs, n, D, V)
+                num, nq = ws.take((T, self.v_dim), torch.float32), ws.take((T, n), torch.float32)
+                K.matrix_memory_walk(proj, 0, k0, v0, q_scale, gates, state, slots, ctx.q_start, ctx.positions, num, nq, ctx.num_seqs, n, D, V)
+                K.matrix_memory_finish(num, nq, gates, proj[:, g0:g0 + self.v_dim], self.norm_w, self.norm_eps, self.den_eps, y, n, V)
         out = linear(ctx, y, self.w_o, out_dtype=torch.float32, may_defer_sum=True)
         return (out, z[:, 2 * n:2 * n + self.riders]) if self.riders else out
