@@ -1,7 +1,7 @@
 #!/usr/bin/env python3
 """Headline measurement: decode tokens per second of the Qwen3-8B-shaped model on one B200.
 
-    python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch B] [--prompt-len L] [--prefill-tokens T] [--layers N] [--workload decode|llama3_8b|serving|mixed_step|dulisun|ripesun|botalorn|mumazen]
+    python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch B] [--prompt-len L] [--prefill-tokens T] [--layers N] [--workload decode|llama3_8b|serving|mixed_step|dulisun|ripesun|botalorn|mumazen|kuvidra]
 
 A step is one decode step of a batch of requests that each hold a 1,024-token prompt (context
 limit 4,096, pages of 16 tokens), random bfloat16 weights, synthetic uniform token ids.  One JSON
@@ -676,6 +676,111 @@ def mumazen_workload(only: str = "") -> int:
     return 0
 
 
+def _kuvidra_config(width, heads, dim, vdim, kv_rank, q_rank, mem_heads, mem_dim, mem_vdim, ff, experts, top, expert_ff, shared_ff, layers, vocab):
+    lat = {"type": "latent_attention", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank, "scale": dim ** -0.5}}
+    mem = {"type": "mlstm", "mixer": {"heads": mem_heads, "dim": mem_dim, "vdim": mem_vdim, "gate_cap": 15.0}}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared_ff}}
+    mlps = ({"kind": "dense", "ff": ff}, moe)
+    # mixers alternate; of every four layers one mixer of each kind carries the dense and one the routed feed-forward
+    return {"architecture": "Kuvidra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "loop": None,
+            "layers": [dict(mem if i % 2 == 0 else lat, mlp=mlps[(i // 2) % 2]) for i in range(layers)]}
+
+
+# (name, Kuvidra sizes).  Beside each: the Ripesun model of the same width, heads, head sizes, latent, layers and vocabulary (linear
+# attention with decay and latent attention with a rotated part of half a head, every position seen) and the dense
+# Qwen3-style model, at equal per-token feed-forward arithmetic of the dense layers.
+KUVIDRA_SHAPES = (
+    ("w2048_h16", dict(width=2048, heads=16, dim=128, vdim=128, kv_rank=512, q_rank=1536, mem_heads=16, mem_dim=128, mem_vdim=128, ff=6144,
+                       experts=16, top=4, expert_ff=1024, shared_ff=1024, layers=8, vocab=32768)),
+    ("w4096_h32", dict(width=4096, heads=32, dim=128, vdim=128, kv_rank=512, q_rank=1536, mem_heads=32, mem_dim=128, mem_vdim=128, ff=12288,
+                       experts=16, top=4, expert_ff=2048, shared_ff=2048, layers=4, vocab=32768)),
+    ("w1024_h16", dict(width=1024, heads=16, dim=64, vdim=64, kv_rank=256, q_rank=512, mem_heads=16, mem_dim=64, mem_vdim=64, ff=3072,
+                       experts=8, top=2, expert_ff=512, shared_ff=512, layers=8, vocab=32768)),
+)
+
+
+def kuvidra_workload(only: str = "") -> int:
+    """Prefill and decode throughput of the Kuvidra design at a few sizes that resemble a real model's layers (random
+    bfloat16 weights), each beside the Ripesun model and the dense Qwen3-style model of equal size.  Prefill: one prompt of 2,048
+    tokens; decode: 8 and 64 requests at 1,024 tokens of context, captured graphs.  Timed on the device with CUDA events
+    after warm-up; every step reads more weights than L2 holds.  The timed steps lie between cudaProfilerStart and
+    cudaProfilerStop.  AIEN_BENCH_MODELS names the models to run (default: all)."""
+    import torch
+    from aien_sovereign_core_mv_b200 import Engine, EngineConfig
+    from aien_sovereign_core_mv_b200 import kernels as K
+    results = []
+    P, CTX = 2048, 1024
+    which_only = os.environ.get("AIEN_BENCH_MODELS", "").split(",") if os.environ.get("AIEN_BENCH_MODELS") else None
+    for name, sz in KUVIDRA_SHAPES:
+        if only and only != name:
+            continue
+        lat = {"type": "latent_attention", "mixer": {"heads": sz["heads"], "dim": sz["dim"], "rot_dim": sz["dim"] // 2, "vdim": sz["vdim"],
+                                                     "kv_rank": sz["kv_rank"], "q_rank": sz["q_rank"], "scale": (1.5 * sz["dim"]) ** -0.5,
+                                                     "rot": {"base": 10000.0, "dims": sz["dim"] // 2}}}
+        lin = {"type": "lightning", "mixer": {"heads": sz["mem_heads"], "dim": sz["mem_dim"], "vdim": sz["mem_vdim"],
+                                              "decay": [1.0 - 2.0 ** -(5.0 + 3.0 * i / sz["mem_heads"]) for i in range(sz["mem_heads"])]}}
+        ripesun = {"architecture": "Ripesun", "vocab": sz["vocab"], "width": sz["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+                   "residual_mult": 1.0, "logit_softcap": 30.0, "token_side": {"dim": sz["width"] // 16},
+                   "layers": [dict(lin if i % 2 == 0 else lat, mlp={"kind": "dense", "ff": sz["ff"]}) for i in range(sz["layers"])]}
+        dense = dict(architectures=["Qwen3ForCausalLM"], model_type="qwen3", num_hidden_layers=sz["layers"], hidden_size=sz["width"],
+                     num_attention_heads=sz["heads"], num_key_value_heads=max(1, sz["heads"] // 4), head_dim=sz["dim"], intermediate_size=sz["ff"] * 2 // 3,
+                     vocab_size=sz["vocab"], rope_theta=10000.0, rms_norm_eps=1e-6, tie_word_embeddings=True,
+                     max_position_embeddings=8192, hidden_act="silu", attention_bias=False, eos_token_id=0)
+        row = {"shape": name, "sizes": dict(sz), "dense_intermediate": sz["ff"] * 2 // 3}
+        for which, cfg in (("kuvidra", _kuvidra_config(**sz)), ("ripesun", ripesun), ("dense", dense)):
+            if which_only and which not in which_only:
+                continue
+            ec = EngineConfig(dtype="bfloat16", page_size=16, max_cache_tokens=64 * (CTX + 64) + P + 64, max_requests=64,
+                              max_batch_tokens=P, max_context=4096, max_batch_size=64)
+            eng = Engine.from_config(cfg, seed=5, engine_config=ec, init_std=0.02, device_init=True)
+            V = sz["vocab"]
+            toks = lambda n, s: [(7 * i + 13 * s) % V for i in range(n)]
+
+            def timed(fn, warm, reps):
+                for i in range(warm):
+                    fn(i)
+                torch.cuda.synchronize()
+                ms = []
+                for i in range(reps):
+                    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                    e0.record()
+                    fn(warm + i)
+                    e1.record()
+                    torch.cuda.synchronize()
+                    ms.append(e0.elapsed_time(e1))
+                return sorted(ms)[len(ms) // 2]
+
+            def prefill(i):
+                eng.step([(9000 + i, toks(P, i), [P - 1])])
+                eng.end_request(9000 + i)
+
+            out = {}
+            torch.cuda.profiler.start()
+            t = timed(prefill, 3, 5)
+            out["prefill_2048"] = {"ms": round(t, 3), "tokens_per_s": round(P / t * 1e3, 1)}
+            for batch in (8, 64):
+                for r in range(0, batch, 2):
+                    eng.step([(r, toks(CTX, r), []), (r + 1, toks(CTX, r + 1), [])])
+                t = timed(lambda i: eng.step([(r, [(i + r) % V], [0]) for r in range(batch)]), 4, 12)
+                out[f"decode_b{batch}"] = {"ms": round(t, 3), "tokens_per_s": round(batch / t * 1e3, 1)}
+                for r in range(batch):
+                    eng.end_request(r)
+            torch.cuda.profiler.stop()
+            eng.check_waits()
+            out["wait_errors"] = sum(1 for w in K.read_wait_errors() if w != 0)
+            out["weight_bytes"] = int(sum(t.numel() * t.element_size() for p in eng.model.parts() for t in vars(p).values()
+                                          if isinstance(t, torch.Tensor) and t.dim() >= 2))
+            row[which] = out
+            del eng
+            torch.cuda.empty_cache()
+        results.append(row)
+    print(json.dumps({"metric": "kuvidra_beside_ripesun_and_dense", "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True,
+                      "dtype": "bf16", "data": "synthetic", "impl": "ours", "shapes": results,
+                      "config": {"prefill_tokens": P, "decode_context": CTX, "page_size": 16, "seed": 5,
+                                 "l2": "weights read per step exceed L2"}}))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -694,18 +799,19 @@ def main() -> int:
     ap.add_argument("--top-k", type=int, default=0, help="top-k of the end-to-end run")
     ap.add_argument("--align-step-tokens", type=int, default=0,
                     help="serving workload: the scheduler cuts portions so that a step's tokens fill whole tiles of this many rows")
-    ap.add_argument("--shape", default="", help="dulisun, ripesun, botalorn and mumazen workloads: only this shape (default: all)")
+    ap.add_argument("--shape", default="", help="dulisun, ripesun, botalorn, mumazen and kuvidra workloads: only this shape (default: all)")
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--skip-prefill", action="store_true")
     ap.add_argument("--skip-e2e", action="store_true")
-    ap.add_argument("--workload", default="decode", choices=["decode", "llama3_8b", "serving", "mixed_step", "dulisun", "ripesun", "botalorn", "mumazen"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "llama3_8b", "serving", "mixed_step", "dulisun", "ripesun", "botalorn", "mumazen", "kuvidra"],
                     help="decode: the headline decode-step measurement (Qwen3-8B shape, 1,024-token prompts); llama3_8b: the same "
                          "line for the Llama-3-8B shape, 16 requests at contexts ending at 8,192 tokens; serving: continuous batching "
                          "of 32 requests on the Qwen3-4B shape (prompts of 64..4096 tokens, portions of 512, 256 new tokens each); "
                          "mixed_step: one step of a 512-token portion beside 24 decoding requests on that shape, timed alone; "
                          "dulisun: prefill and decode of the Dulisun design at a few sizes beside the dense model of equal size; "
                          "ripesun: the same for the Ripesun design; botalorn: the Botalorn design beside Ripesun and the dense model; "
-                         "mumazen: the Mumazen design beside Botalorn and the dense model")
+                         "mumazen: the Mumazen design beside Botalorn and the dense model; "
+                         "kuvidra: the Kuvidra design beside Ripesun and the dense model")
     ap.add_argument("--fill", default="prefill", choices=["prefill", "cache"],
                     help="how requests get their prompt: real prefill, or (development only) cache pages "
                          "filled with random keys/values without running the model")
@@ -731,6 +837,8 @@ def main() -> int:
         return botalorn_workload(args.shape)
     if args.workload == "mumazen":
         return mumazen_workload(args.shape)
+    if args.workload == "kuvidra":
+        return kuvidra_workload(args.shape)
 
     import numpy as np
     import torch
