@@ -287,7 +287,7 @@ AIEN_API int aien_matrix_memory_walk(const void* proj, int p_dt, long ld, int q_
                                      const float* gates, float* state, size_t state_stride, const int* slot_map, const int* q_start,
                                      const int* positions, float* num, float* nq, int S, int H, int D, int V, cudaStream_t stream) {
     if (S <= 0) return 0;
-    if (H <= 0 || D <= 0 || V <= 0 || D > 256 || S > 65535) return AIEN_E_SHAPE;
+    if (H <= 0 || D <= 0 || V <= 0 || D > 512 || S > 65535) return AIEN_E_SHAPE;
     const MmSizes z{H, D, V};
     const dim3 grid((unsigned)(((long)H * (V + 1) + MW_THREADS / 32 - 1) / (MW_THREADS / 32)), S);
 #define MW_CASE(CHV, UV)                                                                                                                  \
@@ -296,7 +296,8 @@ AIEN_API int aien_matrix_memory_walk(const void* proj, int p_dt, long ld, int q_
     if (D <= 32) MW_CASE(1, 4);
     else if (D <= 64) MW_CASE(2, 4);
     else if (D <= 128) MW_CASE(4, 4);
-    else MW_CASE(8, 2);
+    else if (D <= 256) MW_CASE(8, 2);
+    else MW_CASE(16, 1);
 #undef MW_CASE
     return launch_status();
 }

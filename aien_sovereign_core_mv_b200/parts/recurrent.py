@@ -211,8 +211,8 @@ class MatrixMemory(Mixer):
                  denominator_eps: float = 1e-6, position=None):
         self.hidden_size, self.num_heads, self.head_dim, self.value_dim = int(hidden_size), int(num_heads), int(head_dim), int(value_dim)
         self.cap, self.norm_eps, self.den_eps = float(gate_cap), float(norm_eps), float(denominator_eps)
-        if min(self.num_heads, self.head_dim, self.value_dim) <= 0 or self.head_dim > 256:
-            raise ValueError(f"heads, head_dim and value_dim must be positive; head_dim {head_dim}: the kernels keep up to 256 rows of a state column")
+        if min(self.num_heads, self.head_dim, self.value_dim) <= 0 or self.head_dim > 512:
+            raise ValueError(f"heads, head_dim and value_dim must be positive; head_dim {head_dim}: the kernels keep up to 512 rows of a state column")
         if not self.cap > 0.0:
             raise ValueError(f"gate_cap {gate_cap!r} must be positive")
         self.qk_dim, self.v_dim = self.num_heads * self.head_dim, self.num_heads * self.value_dim

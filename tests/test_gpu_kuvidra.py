@@ -223,7 +223,7 @@ def _memory_want(off, rows, z, bi, bf, heads, D, V, cap, w, eps):
 
 
 @pytest.mark.parametrize("form", ["walk", "token", "chunks"])
-@pytest.mark.parametrize("heads,D,V,cap", [(4, 16, 16, 15.0), (3, 48, 80, 6.0), (2, 64, 128, 15.0), (2, 128, 64, 30.0), (1, 256, 256, 9.0), (3, 20, 12, 15.0), (2, 7, 9, 12.0)])
+@pytest.mark.parametrize("heads,D,V,cap", [(4, 16, 16, 15.0), (3, 48, 80, 6.0), (2, 64, 128, 15.0), (2, 128, 64, 30.0), (1, 256, 256, 9.0), (3, 20, 12, 15.0), (2, 7, 9, 12.0), (1, 300, 8, 15.0)])
 def test_matrix_memory_cut_any_way(form, heads, D, V, cap):
     """Whole, in portions down to one token, beside one another: the same rows and states as token by token in float64.
     A used slot must not leak into a new request, and slots of others stay as they are."""
