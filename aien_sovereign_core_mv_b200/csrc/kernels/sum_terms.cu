@@ -19,12 +19,18 @@ __device__ __forceinline__ float term_gate(const SumTerm& a, size_t t) {
     return a.gate == nullptr ? 1.0f : 1.0f / (1.0f + expf(-a.gate[t * a.ldg]));
 }
 
+__device__ __forceinline__ float4 load4(const SumTerm& a, size_t at) {
+    return a.dt == AIEN_DT_F32 ? ld_act4(reinterpret_cast<const float*>(a.p) + at) : ld_act4(reinterpret_cast<const __nv_bfloat16*>(a.p) + at);
+}
+// the loads of four parts in flight, then their sum in order
 __device__ __forceinline__ float4 term_load4(const SumTerm& a, size_t at) {
-    float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int p = 0; p < a.parts; ++p) {
-        const float4 v = a.dt == AIEN_DT_F32 ? ld_act4(reinterpret_cast<const float*>(a.p) + (size_t)p * a.stride + at)
-                                             : ld_act4(reinterpret_cast<const __nv_bfloat16*>(a.p) + (size_t)p * a.stride + at);
-        s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
+    float4 s = load4(a, at);
+    for (int p = 1; p < a.parts; p += 4) {
+        float4 v[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) v[i] = p + i < a.parts ? load4(a, (size_t)(p + i) * a.stride + at) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { s.x += v[i].x; s.y += v[i].y; s.z += v[i].z; s.w += v[i].w; }
     }
     return s;
 }
@@ -135,6 +141,37 @@ pass_rows_kernel(const float* __restrict__ x, SumTerms a, const float* __restric
     }
 }
 
+// The same, four numbers a thread.
+template <typename TO>
+__global__ void __launch_bounds__(256)
+pass_rows_vec_kernel(const float* __restrict__ x, SumTerms a, const float* __restrict__ x0, TO* __restrict__ out, int H) {
+    const size_t t = blockIdx.y, row = t * H;
+    const int c = 4 * (blockIdx.x * 256 + threadIdx.x);
+    if (c >= H) return;
+    float4 v = ld_act4(x + row + c);
+    const float4 e = ld_act4(x0 + row + c);
+#pragma unroll
+    for (int k = 0; k < 3; ++k) {
+        if (k < a.n) {
+            const float g = term_gate(a.t[k], t);
+            const float4 d = term_load4(a.t[k], row + c);
+            v.x = fmaf(g, d.x, v.x);
+            v.y = fmaf(g, d.y, v.y);
+            v.z = fmaf(g, d.z, v.z);
+            v.w = fmaf(g, d.w, v.w);
+        }
+    }
+    if (sizeof(TO) == 4) {
+        store4<TO>(out + t * 2 * H + c, v);
+        store4<TO>(out + t * 2 * H + H + c, e);
+    } else {
+        store4<TO>(out + t * 3 * H + c, v);
+        store4<TO>(out + t * 3 * H + H + c, make_float4(v.x - to_f(from_f<TO>(v.x)), v.y - to_f(from_f<TO>(v.y)), v.z - to_f(from_f<TO>(v.z)),
+                                                        v.w - to_f(from_f<TO>(v.w))));
+        store4<TO>(out + t * 3 * H + 2 * H + c, e);
+    }
+}
+
 }  // namespace aien
 
 using namespace aien;
@@ -187,6 +224,8 @@ AIEN_API int aien_pass_rows(const float* x, int terms, TERM_ARGS(0), TERM_ARGS(1
     const SumTerms a{{TERM_SET(0), TERM_SET(1), TERM_SET(2)}, terms};
     bool vec = true;
     if (!terms_ok(a, H, &vec)) return AIEN_E_SHAPE;
-    AIEN_DISPATCH_DTYPE(o_dt, TO, (pass_rows_kernel<TO><<<dim3((H + 255) / 256, T), 256, 0, stream>>>(x, a, x0, (TO*)out, H)));
+    if (((uintptr_t)x | (uintptr_t)x0 | (uintptr_t)out) & 15) vec = false;
+    if (vec) AIEN_DISPATCH_DTYPE(o_dt, TO, (pass_rows_vec_kernel<TO><<<dim3((H + 1023) / 1024, T), 256, 0, stream>>>(x, a, x0, (TO*)out, H)));
+    else AIEN_DISPATCH_DTYPE(o_dt, TO, (pass_rows_kernel<TO><<<dim3((H + 255) / 256, T), 256, 0, stream>>>(x, a, x0, (TO*)out, H)));
     return launch_status();
 }

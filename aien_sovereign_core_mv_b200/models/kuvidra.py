@@ -9,8 +9,8 @@ x, e = embed[token] and N(y, w) = y / sqrt(mean y^2 + eps) * w:
 
 * x = e; logits = embed N(x, w_final) (the head is the embedding's table);
 * a layer: h = N(x, norm1); x <- x + mixer(h) + ff(h);
-* ``loop`` {start, stop, times}: layers start .. stop - 1 run ``times`` times in a row with the same tensors, every pass
-  with a cache and state of its own; ahead of pass t = 0, 1, ... the stream becomes loop.in [x; e] + loop.step[t];
+* ``loop`` {start, stop, times}: the stretch start .. stop - 1 is gone through ``times`` times on one set of tensors, each
+  pass keeping its own cache and states; ahead of pass t, the first one included, x <- loop.in [x; e] + loop.step[t];
 * mixer ``latent_attention``: :class:`~..parts.latent_attention.LatentAttention` without a rotated part, with a gate per head;
 * mixer ``mlstm``: :class:`~..parts.recurrent.MatrixMemory`;
 * feed-forward ``dense``: W_down gelu(W_up h), the erf form; ``moe``: :class:`~..parts.moe.RoutedExperts` with sigmoid scores

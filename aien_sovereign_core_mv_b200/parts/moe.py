@@ -36,7 +36,7 @@ class RoutedExperts(FeedForward):
     the first four needs ``combined`` or a block that takes the branch as ``terms()`` (and no expert groups).
     ``score``: "softmax", or "sigmoid" (every router output by itself).  ``act`` "swiglu": experts and shared expert are
     W_down (silu(W_gate h) * (W_up h)) (tensors ``experts.<e>.gate`` and ``shared.gate_proj`` beside the others).
-    ``weight_on_input``: a choice's weight multiplies the expert's input, expert(w h), not its output.
+    ``weight_on_input``: a choice counts as expert(w h) instead of w expert(h).
 
     ``terms`` gives the routed parts and the shared expert's output with its gate as they are, for a block that adds
     several terms in one kernel; the router's rows (and the shared gate's) may then have ridden in a neighbour's product."""

@@ -194,12 +194,12 @@ class GatedDeltaRule(Mixer):
 
 @register_mixer("matrix_memory")
 class MatrixMemory(Mixer):
-    """A matrix memory with exponential gates (the mLSTM of xLSTM).  q = W_q h * head_dim^-1/2 and k = W_k h (heads x
+    """A matrix memory with exponential gates (the mLSTM recurrence).  q = W_q h * head_dim^-1/2 and k = W_k h (heads x
     ``head_dim``), v = W_v h (heads x ``value_dim``); per head a log input gate i = cap tanh((W_i h + i_bias) / cap) and a
     log forget gate f = logsigmoid(cap tanh((W_f h + f_bias) / cap)), cap = ``gate_cap``.  With a running maximum m that
     starts at 0: m_t = max(f + m, i); S <- e^(f + m - m_t) S + e^(i - m_t) k v^T, n the same with k alone;
-    o = S^T q / (max(|n . q|, e^(-m_t)) + ``denominator_eps``).  Each head's o is divided by its root mean square
-    (``norm_eps``), the heads together are multiplied by the weight ``norm`` and by sigmoid(W_g h) and projected by W_o.
+    o = S^T q / (max(|n . q|, e^(-m_t)) + ``denominator_eps``).  The output is W_o (o / rms(o) * ``norm`` *
+    sigmoid(W_g h)), rms over one head's numbers (``norm_eps``), ``norm`` a weight over all heads'.
 
     One float32 state slot per request holds S, n and m; it starts from zeros.  Gates, m, the recurrence, the denominator and
     the norm are float32 in both engine precisions.  One product makes q | k | v | g | i | f (with riders behind);

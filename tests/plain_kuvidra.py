@@ -122,7 +122,7 @@ def moe_ff(f, Wt, p, h):
 
 
 def run_order(cfg):
-    """[(layer, pass number or None, first of its pass)]: layers start..stop-1 run ``times`` times in a row."""
+    """[(layer, pass number or None, whether it opens the pass)] of every layer run in order."""
     n = len(cfg["layers"])
     loop = cfg.get("loop")
     if not loop:
