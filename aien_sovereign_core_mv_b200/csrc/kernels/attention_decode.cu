@@ -18,7 +18,9 @@
 // Formulas: crates/aien-inference-abi/src/backend.rs:311-379 (online softmax over pages, scale
 // 1/sqrt(head_dim)).
 //
-// Needs head_dim % 16 == 0 and <= 256, at most 16 query heads per kv head, bfloat16 q and cache.
+// Needs head_dim % 8 == 0 and <= 256, at most 16 query heads per kv head, bfloat16 q and cache.  Values may have a size
+// of their own (a multiple of 16 up to 256), one value head may serve several neighbouring key heads (attention maps over
+// the same values), and the result may leave in float32.
 #include "common.cuh"
 #include "attention_decode_merge.cuh"
 #include <math.h>
@@ -93,6 +95,13 @@ __device__ __forceinline__ void ad_norm_rope_head(const __nv_bfloat16* src, floa
     }
 }
 
+// Values of hdv numbers, one value head for v_share neighbouring key heads; out_f32: float32 results; from_first: key blocks
+// (blockIdx.x) are counted from the block of the first key the token sees, as under a chunk mask, and the launch has only
+// as many as a window can touch.
+struct ValueForm {
+    int hdv, v_share, out_f32, from_first;
+};
+
 // HS = ceil(head_dim / 32) dim steps of the score product, NT = ceil(G / 8) head tiles
 template <int HS, int NT>
 __global__ void __launch_bounds__(AD_WARPS * 32)
@@ -101,9 +110,9 @@ paged_decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long q_stride
                               const int* __restrict__ block_table, int max_blocks,
                               const int* __restrict__ seq_of_token, const int* __restrict__ positions,
                               const int* __restrict__ token_list, float* __restrict__ part_out, float* __restrict__ part_ml, int* __restrict__ counters,
-                              __nv_bfloat16* __restrict__ out, long out_stride,
+                              void* __restrict__ out, long out_stride,
                               int nq, int nkv, int hd, int page_size, int window, float scale, int max_splits, int misc_bytes,
-                              FusedQK fq, int kchunk, const float* __restrict__ sinks, HeadTerms ht) {
+                              FusedQK fq, int kchunk, const float* __restrict__ sinks, HeadTerms ht, ValueForm vf) {
     constexpr int NH = NT * 8;
     extern __shared__ float smem[];
     __shared__ int s_slot[AD_CHUNK];
@@ -123,7 +132,8 @@ paged_decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long q_stride
     int first = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
     if (kchunk > 0) first = max(first, (pos / kchunk) * kchunk);
     const int psplit = blockIdx.x;                                  // where this block's partial results go
-    const int split = kchunk > 0 ? first / AD_CHUNK + (int)blockIdx.x : (int)blockIdx.x;
+    const bool rel = kchunk > 0 || vf.from_first;
+    const int split = rel ? first / AD_CHUNK + (int)blockIdx.x : (int)blockIdx.x;
     // In a decode-only step token t is request t (seq_of_token may be null): the table row does not
     // hang on another load, so the page lookups go out together with the position load.
     const int* bt = block_table + (size_t)(seq_of_token ? seq_of_token[t] : t) * max_blocks;
@@ -147,7 +157,8 @@ paged_decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long q_stride
     // their index flipped instead.  Other row sizes are padded to 4 (mod 8) pieces.
     const bool swz = (CH % 8) == 0;
     const int k_stride = swz ? hd * 2 : (CH + ((4 - CH % 8) + 8) % 8) * 16;
-    const int v_stride = hd * 2 + 16;                        // an odd number of pieces: ldmatrix rows fall on different banks
+    const int hdv = vf.hdv, CHV = hdv / 8, nv = nkv / vf.v_share, vh = kvh / vf.v_share;
+    const int v_stride = hdv * 2 + 16;                       // an odd number of pieces: ldmatrix rows fall on different banks
     const uint32_t K_u = (uint32_t)__cvta_generic_to_shared(smem) + misc_bytes;
     const uint32_t V_u = K_u + AD_CHUNK * k_stride;
     for (int idx = tid; idx < AD_CHUNK * CH; idx += AD_WARPS * 32) {
@@ -159,12 +170,12 @@ paged_decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long q_stride
         ad_cp_async16(K_u + r * k_stride + pc * 16, k_cache + ((size_t)(valid ? sl : 0) * nkv + kvh) * hd + ch * 8, valid);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
-    for (int idx = tid; idx < AD_CHUNK * CH; idx += AD_WARPS * 32) {
-        const int r = idx / CH, ch = idx - r * CH;
+    for (int idx = tid; idx < AD_CHUNK * CHV; idx += AD_WARPS * 32) {
+        const int r = idx / CHV, ch = idx - r * CHV;
         const int key = chunk_base + r, sl = s_slot[r];
         if (fq.k != nullptr && key == pos) continue;
         const bool valid = key >= lo && key <= hi && sl >= 0;
-        ad_cp_async16(V_u + r * v_stride + ch * 16, v_cache + ((size_t)(valid ? sl : 0) * nkv + kvh) * hd + ch * 8, valid);
+        ad_cp_async16(V_u + r * v_stride + ch * 16, v_cache + ((size_t)(valid ? sl : 0) * nv + vh) * hdv + ch * 8, valid);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
 
@@ -300,7 +311,7 @@ paged_decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long q_stride
     // ---- phase 3: out^T[dims, heads] = V^T[dims, keys] . P[keys, heads]; a warp owns 16 dims at a time, so
     // no sum over warps is needed.  V^T fragments by transposing ldmatrix reads of the V rows.
     const int s_lo = first / AD_CHUNK, s_hi = pos / AD_CHUNK;
-    for (int mt = warp; mt * 16 < hd; mt += AD_WARPS) {
+    for (int mt = warp; mt * 16 < hdv; mt += AD_WARPS) {
         float oacc[NT][4];
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) oacc[nt][0] = oacc[nt][1] = oacc[nt][2] = oacc[nt][3] = 0.f;
@@ -324,8 +335,8 @@ paged_decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long q_stride
                 const int h = nt * 8 + 2 * c + e;
                 if (h < G) {
                     const size_t row = ((size_t)zt * nq + kvh * G + h) * max_splits + psplit;
-                    part_out[row * hd + mt * 16 + g] = oacc[nt][e];
-                    part_out[row * hd + mt * 16 + g + 8] = oacc[nt][2 + e];
+                    part_out[row * hdv + mt * 16 + g] = oacc[nt][e];
+                    part_out[row * hdv + mt * 16 + g + 8] = oacc[nt][2 + e];
                 }
             }
     }
@@ -347,15 +358,20 @@ paged_decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long q_stride
     __syncthreads();
     if (!is_last) return;
     __threadfence();
-    const int part_lo = kchunk > 0 ? 0 : s_lo;                      // index of the first block's partial results
+    const int part_lo = rel ? 0 : s_lo;                      // index of the first block's partial results
     const float* hs = sinks != nullptr ? sinks + kvh * G : nullptr;
     const float* hg = ht.gate != nullptr ? ht.gate + (size_t)t * ht.ldg + kvh * G : nullptr;
-    if (hd <= 128)
-        ad_merge_chunks<NH, 1>(smem, part_out, part_ml, out + (size_t)t * out_stride + (size_t)kvh * G * hd, (size_t)zt * nq + kvh * G,
-                               G, hd, max_splits, part_lo, s_hi - s_lo + 1, threadIdx.x, AD_WARPS * 32, [] { __syncthreads(); }, hs, hg);
-    else
-        ad_merge_chunks<NH, 2>(smem, part_out, part_ml, out + (size_t)t * out_stride + (size_t)kvh * G * hd, (size_t)zt * nq + kvh * G,
-                               G, hd, max_splits, part_lo, s_hi - s_lo + 1, threadIdx.x, AD_WARPS * 32, [] { __syncthreads(); }, hs, hg);
+    const size_t at = (size_t)t * out_stride + (size_t)kvh * G * hdv;
+    auto merge = [&](auto* row) {
+        if (hdv <= 128)
+            ad_merge_chunks<NH, 1>(smem, part_out, part_ml, row, (size_t)zt * nq + kvh * G, G, hdv, max_splits, part_lo, s_hi - s_lo + 1,
+                                   threadIdx.x, AD_WARPS * 32, [] { __syncthreads(); }, hs, hg);
+        else
+            ad_merge_chunks<NH, 2>(smem, part_out, part_ml, row, (size_t)zt * nq + kvh * G, G, hdv, max_splits, part_lo, s_hi - s_lo + 1,
+                                   threadIdx.x, AD_WARPS * 32, [] { __syncthreads(); }, hs, hg);
+    };
+    if (vf.out_f32) merge(reinterpret_cast<float*>(out) + at);
+    else merge(reinterpret_cast<__nv_bfloat16*>(out) + at);
 }
 
 template <int HS, int NT>
@@ -363,18 +379,18 @@ static int launch_decode(const void* q, long q_stride, const void* kc, const voi
                          const int* seq_of_token, const int* positions, const int* token_list, float* part_out, float* part_ml, int* counters,
                          void* out, long out_stride,
                          int nq, int nkv, int hd, int page_size, int window, float scale, int max_splits, int T,
-                         const FusedQK& fq, int kchunk, const float* sinks, const HeadTerms& ht, cudaStream_t stream) {
+                         const FusedQK& fq, int kchunk, const float* sinks, const HeadTerms& ht, const ValueForm& vf, cudaStream_t stream) {
     const int NH = NT * 8;
     size_t loop_bytes = ((size_t)AD_CHUNK * NH + 2 * NH) * 4 + (size_t)NH * AD_CHUNK * 2;          // scores, max/denominator, probabilities
     if (fq.k != nullptr) loop_bytes += (size_t)AD_WARPS * 256 * 4 + (size_t)NH * hd * 2 + 16;      // fused q/k scratch, q
     const size_t comb_bytes = 0;
-    const size_t merge_bytes = ad_merge_scratch_floats(max_splits, nq / nkv, hd) * 4;
+    const size_t merge_bytes = ad_merge_scratch_floats(max_splits, nq / nkv, vf.hdv) * 4;
     size_t smem = loop_bytes > comb_bytes ? loop_bytes : comb_bytes;
     if (merge_bytes > smem) smem = merge_bytes;
     const int misc_bytes = (int)((smem + 127) & ~(size_t)127);           // per-warp scratch, combine and merge areas
     const int CH = hd / 8;
     const int k_stride = (CH % 8) == 0 ? hd * 2 : (CH + ((4 - CH % 8) + 8) % 8) * 16;
-    const size_t kv_bytes = (size_t)AD_CHUNK * k_stride + (size_t)AD_CHUNK * (hd * 2 + 16);   // K and V of the chunk
+    const size_t kv_bytes = (size_t)AD_CHUNK * k_stride + (size_t)AD_CHUNK * (vf.hdv * 2 + 16);   // K and V of the chunk
     smem = (size_t)misc_bytes + kv_bytes;
     if (smem > 200 * 1024) return AIEN_E_SHAPE;
     auto kern = paged_decode_attention_kernel<HS, NT>;
@@ -388,8 +404,8 @@ static int launch_decode(const void* q, long q_stride, const void* kc, const voi
     // on the kernel ahead while holding the slots its own tail needs).
     kern<<<grid, AD_WARPS * 32, smem, stream>>>((const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)kc,
                  (const __nv_bfloat16*)vc, bt, max_blocks, seq_of_token, positions, token_list,
-                 part_out, part_ml, counters, (__nv_bfloat16*)out, out_stride, nq, nkv, hd, page_size, window, scale, max_splits,
-                 misc_bytes, fq, kchunk, sinks, ht);
+                 part_out, part_ml, counters, out, out_stride, nq, nkv, hd, page_size, window, scale, max_splits,
+                 misc_bytes, fq, kchunk, sinks, ht, vf);
     return launch_status();
 }
 
@@ -405,7 +421,8 @@ static int decode_dispatch(
     const void* q, long q_stride, const void* k_cache, const void* v_cache, const int* block_table, int max_blocks,
     const int* seq_of_token, const int* positions, const int* token_list, void* out, long out_stride, float* part_out,
     float* part_ml, int* counters, int nq, int nkv, int hd, int page_size, int window, float scale, int max_splits, int T,
-    const FusedQK& fq, cudaStream_t stream, int kchunk = 0, const float* sinks = nullptr, const HeadTerms& ht = HeadTerms{});
+    const FusedQK& fq, cudaStream_t stream, int kchunk = 0, const float* sinks = nullptr, const HeadTerms& ht = HeadTerms{},
+    const ValueForm* vf = nullptr);
 
 // The same under a chunk mask (kchunk > 0: a token sees only the keys of its own chunk of that many positions) and
 // with per-head softmax sinks (float32 [nq], may be null).  With kchunk > 0, max_splits counts the key blocks a
@@ -420,6 +437,23 @@ AIEN_API int aien_paged_attention_decode_masked(
     return decode_dispatch(q, q_stride, k_cache, v_cache, block_table, max_blocks, seq_of_token, positions, token_list, out,
                            out_stride, part_out, part_ml, counters, nq, nkv, hd, page_size, window, scale, max_splits, T, none, stream,
                            kchunk, sinks);
+}
+
+// Values of hdv numbers (v_cache [slots, nkv / v_share, hdv], out [T, nq * hdv]; part_out [T * nq * max_splits * hdv]), one
+// value head for v_share neighbouring key heads, float32 results with out_f32, an optional chunk mask, an optional cap on
+// the scaled score.  from_first: see ValueForm; max_splits then counts the key blocks a window can touch.
+AIEN_API int aien_paged_attention_decode_values(
+    const void* q, long q_stride, const void* k_cache, const void* v_cache, const int* block_table, int max_blocks,
+    const int* seq_of_token, const int* positions, const int* token_list, void* out, long out_stride, float* part_out,
+    float* part_ml, int* counters, int nq, int nkv, int hd, int page_size, int window, float scale, int max_splits, int T,
+    int kchunk, float softcap, int hdv, int v_share, int out_f32, int from_first, cudaStream_t stream) {
+    if (kchunk < 0 || hdv <= 0 || hdv > 256 || (hdv & 15) || v_share <= 0 || nkv % v_share != 0) return AIEN_E_SHAPE;
+    FusedQK none = {};
+    const HeadTerms ht{nullptr, nullptr, nullptr, 0, softcap > 0.f ? softcap : 0.f};
+    const ValueForm vf{hdv, v_share, out_f32 ? 1 : 0, from_first ? 1 : 0};
+    return decode_dispatch(q, q_stride, k_cache, v_cache, block_table, max_blocks, seq_of_token, positions, token_list, out,
+                           out_stride, part_out, part_ml, counters, nq, nkv, hd, page_size, window, scale, max_splits, T, none, stream,
+                           kchunk, nullptr, ht, &vf);
 }
 
 // The plain split-key kernel with terms per query head (see HeadTerms; each pointer may be null): head_scale and
@@ -464,19 +498,20 @@ static int decode_dispatch(
     const void* q, long q_stride, const void* k_cache, const void* v_cache, const int* block_table, int max_blocks,
     const int* seq_of_token, const int* positions, const int* token_list, void* out, long out_stride, float* part_out,
     float* part_ml, int* counters, int nq, int nkv, int hd, int page_size, int window, float scale, int max_splits, int T,
-    const FusedQK& fq, cudaStream_t stream, int kchunk, const float* sinks, const HeadTerms& ht) {
+    const FusedQK& fq, cudaStream_t stream, int kchunk, const float* sinks, const HeadTerms& ht, const ValueForm* values) {
     if (T <= 0) return 0;
-    if (hd <= 0 || hd > 256 || (hd & 15) || nkv <= 0 || nq % nkv != 0 || page_size <= 0 || max_splits <= 0) return AIEN_E_SHAPE;
+    if (hd <= 0 || hd > 256 || (hd & (values ? 7 : 15)) || nkv <= 0 || nq % nkv != 0 || page_size <= 0 || max_splits <= 0) return AIEN_E_SHAPE;
+    const ValueForm vf = values ? *values : ValueForm{hd, 1, 0, 0};
     const int G = nq / nkv;
     if (G > 16 || T > 65535 || nkv > 65535) return AIEN_E_SHAPE;
-    if ((q_stride & 7) || ((uintptr_t)q & 15) || ((uintptr_t)k_cache & 15)) return AIEN_E_ALIGN;
+    if ((q_stride & 7) || ((uintptr_t)q & 15) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15)) return AIEN_E_ALIGN;
     const int HS = (hd + 31) / 32, NT = (G + 7) / 8;
     int rc = AIEN_E_SHAPE;
 #define AD_CASE(hs, nt)                                                                                              \
     if (HS == hs && NT == nt)                                                                                        \
         rc = launch_decode<hs, nt>(q, q_stride, k_cache, v_cache, block_table, max_blocks, seq_of_token, positions,  \
                                    token_list, part_out, part_ml, counters, out, out_stride, nq, nkv, hd, page_size, window, scale,        \
-                                   max_splits, T, fq, kchunk, sinks, ht, stream);
+                                   max_splits, T, fq, kchunk, sinks, ht, vf, stream);
     AD_CASE(1, 1) AD_CASE(2, 1) AD_CASE(3, 1) AD_CASE(4, 1) AD_CASE(5, 1) AD_CASE(6, 1) AD_CASE(7, 1) AD_CASE(8, 1)
     AD_CASE(1, 2) AD_CASE(2, 2) AD_CASE(3, 2) AD_CASE(4, 2) AD_CASE(5, 2) AD_CASE(6, 2) AD_CASE(7, 2) AD_CASE(8, 2)
 #undef AD_CASE

@@ -30,9 +30,9 @@ __host__ __device__ inline size_t ad_merge_scratch_floats(int max_splits, int G,
 // head's first query head among part_out's rows; out_row: where that head's output starts.  Every one of
 // the `nthreads` threads (a multiple of 32) calls this; `sync` is a barrier over exactly those threads.
 // hd % 4 == 0, hd <= 128 * PER (PER: float4 a lane takes per chunk and head, 1 or 2).
-template <int NH, int PER, typename Sync>
+template <int NH, int PER, typename TO, typename Sync>
 __device__ __forceinline__ void ad_merge_chunks(float* scratch, const float* __restrict__ part_out, const float* __restrict__ part_ml,
-                                                __nv_bfloat16* __restrict__ out_row, size_t row0, int G, int hd, int max_splits,
+                                                TO* __restrict__ out_row, size_t row0, int G, int hd, int max_splits,
                                                 int s_lo, int nsp, int tid, int nthreads, Sync sync,
                                                 const float* __restrict__ sinks = nullptr,
                                                 const float* __restrict__ gate = nullptr) {
@@ -113,7 +113,7 @@ __device__ __forceinline__ void ad_merge_chunks(float* scratch, const float* __r
             float o = 0.f;
 #pragma unroll
             for (int v = 0; v < AD_MERGE_WAYS; ++v) o += Ps[(size_t)v * hd + d];
-            out_row[(size_t)h * hd + d] = __float2bfloat16_rn(o * Fi[h]);
+            out_row[(size_t)h * hd + d] = from_f<TO>(o * Fi[h]);
         }
         sync();
     }

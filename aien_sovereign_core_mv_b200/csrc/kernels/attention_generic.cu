@@ -6,7 +6,8 @@
 // `token_list` names (T of them).  Optional per head: a factor on the scaled score (`head_scale`), a distance bias
 // (`slopes`: slope[h] * (query position - key position) is taken off the score) and an output gate (`gate` float32
 // [T, ldg]: the head's output is multiplied by sigmoid(gate[t][h])).  `softcap` c > 0: the scaled score s becomes
-// c * tanh(s / c) before the other terms.
+// c * tanh(s / c) before the other terms.  One value head may serve `v_share` neighbouring key heads (attention maps over
+// the same values).
 //
 // It serves the true-32-bit engine for every kind of step (whole prompts, portions with an
 // offset, single decoded tokens) and is the plain kernel the faster attention kernels are
@@ -33,7 +34,7 @@ paged_attention_generic_kernel(const TQ* __restrict__ q, long q_stride,
                                int nq, int nkv, int hd, int page_size, int window, float scale,
                                int chunk, const float* __restrict__ sinks, int hdv, const int* __restrict__ token_list,
                                const float* __restrict__ head_scale, const float* __restrict__ slopes,
-                               const float* __restrict__ gate, long ldg, float softcap) {
+                               const float* __restrict__ gate, long ldg, float softcap, int v_share) {
     __shared__ float qs[256];
     __shared__ float p[AG_THREADS];
     __shared__ int slots[AG_THREADS];
@@ -42,6 +43,7 @@ paged_attention_generic_kernel(const TQ* __restrict__ q, long q_stride,
     const int pos = positions[t];
     const int* bt = block_table + (size_t)seq_of_token[t] * max_blocks;
     const int kvh = h / (nq / nkv);
+    const int nv = nkv / v_share, vh = kvh / v_share;
     int start = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
     if (chunk > 0 && (pos / chunk) * chunk > start) start = (pos / chunk) * chunk;
 
@@ -92,7 +94,7 @@ paged_attention_generic_kernel(const TQ* __restrict__ q, long q_stride,
             const int sl = slots[jj];
             if (sl < 0) continue;
             const float pj = p[jj];
-            const TKV* vp = v_cache + ((size_t)sl * nkv + kvh) * hdv;
+            const TKV* vp = v_cache + ((size_t)sl * nv + vh) * hdv;
             if (tid < hdv) part0 = fmaf(pj, to_f(vp[tid]), part0);
             if (tid + AG_THREADS < hdv) part1 = fmaf(pj, to_f(vp[tid + AG_THREADS]), part1);
         }
@@ -125,16 +127,18 @@ AIEN_API int aien_paged_attention_generic(
     const int* block_table, int max_blocks, const int* seq_of_token, const int* positions,
     void* out, long out_stride, int nq, int nkv, int hd, int page_size, int window, float scale,
     int act_dt, int kv_dt, int T, int chunk, const float* sinks, int hdv, const int* token_list,
-    const float* head_scale, const float* slopes, const float* gate, long ldg, float softcap, cudaStream_t stream) {
+    const float* head_scale, const float* slopes, const float* gate, long ldg, float softcap, int v_share,
+    int out_dt, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (hdv <= 0) hdv = hd;
-    if (hd <= 0 || hd > 256 || hdv > 256 || nkv <= 0 || nq % nkv != 0 || page_size <= 0 || chunk < 0) return AIEN_E_SHAPE;
+    if (hd <= 0 || hd > 256 || hdv > 256 || nkv <= 0 || nq % nkv != 0 || page_size <= 0 || chunk < 0 || v_share <= 0 || nkv % v_share != 0)
+        return AIEN_E_SHAPE;
     if (T > 65535) return AIEN_E_SHAPE;
     dim3 grid(nq, T);
-    AIEN_DISPATCH_DTYPE(act_dt, TQ, AIEN_DISPATCH_DTYPE(kv_dt, TKV,
-        (paged_attention_generic_kernel<TQ, TKV, TQ><<<grid, AG_THREADS, 0, stream>>>(
+    AIEN_DISPATCH_DTYPE(act_dt, TQ, AIEN_DISPATCH_DTYPE(kv_dt, TKV, AIEN_DISPATCH_DTYPE(out_dt, TO,
+        (paged_attention_generic_kernel<TQ, TKV, TO><<<grid, AG_THREADS, 0, stream>>>(
             (const TQ*)q, q_stride, (const TKV*)k_cache, (const TKV*)v_cache, block_table, max_blocks,
-            seq_of_token, positions, (TQ*)out, out_stride, nq, nkv, hd, page_size, window, scale, chunk, sinks, hdv, token_list,
-            head_scale, slopes, gate, ldg, softcap))));
+            seq_of_token, positions, (TO*)out, out_stride, nq, nkv, hd, page_size, window, scale, chunk, sinks, hdv, token_list,
+            head_scale, slopes, gate, ldg, softcap, v_share)))));
     return launch_status();
 }

@@ -2,7 +2,11 @@
 //
 // Same job and same arguments as the mma.sync prefill kernel (portions of prompts of any length
 // at any offset, causal, grouped-query, optional window; the host lists tiles of 128 query tokens),
-// for head sizes 64 and 128 and pages of 8..128 tokens that divide 128.
+// for head sizes 64 and 128 and pages of 8..128 tokens that divide 128.  Keys and values may have sizes of
+// their own, any multiples of 8 up to 128: a tile is then padded to 64 or 128 columns by the copies themselves,
+// which see every head as a matrix of its own and fill zeros beyond its columns.  A value head may serve
+// several neighbouring key heads (v_share: attention maps over the same values), and the result may
+// leave in float32.
 //
 // One CTA handles one tile of 128 query tokens for TWO query heads that share a key/value head,
 // so every key/value block it brings into shared memory is used twice.  Ten warps:
@@ -63,10 +67,14 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
 constexpr int PT_BM = 128, PT_BN = 128, PT_THREADS = 320;
 constexpr int PT_SMEM_MAX = 227 * 1024;
 
-template <int HD> struct PtShape {
-    static constexpr int CHUNKS = HD / 64;                       // 64-column (128-byte) chunks of a row
-    static constexpr int Q_BYTES = PT_BM * HD * 2;               // one head's query tile
-    static constexpr int SLOT_BYTES = PT_BN * HD * 2;            // one K or V block
+// HD / HDV: columns of a key / value tile (the head sizes, padded to 64 or 128)
+template <int HD, int HDV> struct PtShape {
+    static constexpr int WIDE = HD > HDV ? HD : HDV;
+    static constexpr int CHUNKS = HD / 64, CHUNKS_V = HDV / 64;  // 64-column (128-byte) chunks of a row
+    static constexpr int Q_LOAD = PT_BM * HD * 2;                // one head's query tile
+    static constexpr int Q_BYTES = PT_BM * WIDE * 2;             // and its buffer, which may serve as a slot of the ring
+    static constexpr int K_LOAD = PT_BN * HD * 2, V_LOAD = PT_BN * HDV * 2;
+    static constexpr int SLOT_BYTES = PT_BN * WIDE * 2;          // one K or V block
     static constexpr int FIXED = 2 * Q_BYTES + 1024 /*align*/ + 256 /*barriers*/;
     static constexpr int SLOTS_FIT = (PT_SMEM_MAX - FIXED) / SLOT_BYTES;
     static constexpr int SLOTS = SLOTS_FIT > 6 ? 6 : SLOTS_FIT;
@@ -88,15 +96,22 @@ struct PtMaps {
     CUtensorMap blk;
 };
 
-template <int HD>
+// Sizes that the tiles' padding hides: hd and hdv columns of a head are real.  by_head: the maps are
+// [rows][heads][head size] (boxes of one head's 64 columns), for head sizes that are not whole chunks; the bit 0
+// stands for q and k, bit 1 for v.  v_share neighbouring key heads share a value head.  out_f32: float32 results.
+struct PtSizes {
+    int hdv, by_head, v_share, out_f32;
+};
+
+template <int HD, int HDV>
 __global__ void __launch_bounds__(PT_THREADS, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ PtMaps maps_k,
                   const __grid_constant__ PtMaps maps_v, const int* __restrict__ block_table, int max_blocks,
                   const int* __restrict__ q_start, const int* __restrict__ ctx_len, const int* __restrict__ tile_seq,
-                  const int* __restrict__ tile_q0, int num_tiles, __nv_bfloat16* __restrict__ out, long out_stride,
+                  const int* __restrict__ tile_q0, int num_tiles, void* __restrict__ out_v, long out_stride,
                   int nq, int nkv, int page_size, int window, float scale_log2e, int cache_rows, int heads_per_cta, int big_boxes,
-                  int nsplit, float* __restrict__ part_o, float* __restrict__ part_ml, int chunk, const float* __restrict__ sinks, HeadTerms ht) {
-    using S = PtShape<HD>;
+                  int nsplit, float* __restrict__ part_o, float* __restrict__ part_ml, int chunk, const float* __restrict__ sinks, HeadTerms ht, PtSizes sz) {
+    using S = PtShape<HD, HDV>;
     extern __shared__ uint8_t pt_smem[];
     const uint32_t base = (smem_u32(pt_smem) + 1023u) & ~1023u;
     const uint32_t sQ = base, sKV = sQ + 2 * S::Q_BYTES;
@@ -193,10 +208,13 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
         // memory before it has data from this one.
         griddep_wait();
         if (lane == 0) {
-            mbar_expect_tx(q_full, (has_b ? 2 : 1) * S::Q_BYTES);
+            mbar_expect_tx(q_full, (has_b ? 2 : 1) * S::Q_LOAD);
             for (int h = 0; h < (has_b ? 2 : 1); ++h)
-                for (int c = 0; c < S::CHUNKS; ++c)
-                    tma_load_2d(sQ + h * S::Q_BYTES + c * (PT_BM * 128), &map_q, q_full, (head_a + h) * HD + c * 64, qs + q0);
+                for (int c = 0; c < S::CHUNKS; ++c) {
+                    const uint32_t dst = sQ + h * S::Q_BYTES + c * (PT_BM * 128);
+                    if (sz.by_head & 1) tma_load_3d(dst, &map_q, q_full, c * 64, head_a + h, qs + q0);
+                    else tma_load_2d(dst, &map_q, q_full, (head_a + h) * HD + c * 64, qs + q0);
+                }
         }
         for (int item = 0; item < 2 * nb; ++item) {                 // K0 V0 K1 V1 ...; one head alone: K0 K1 V0 K2 V1 ...
             const int slot = single ? item % NS1 : item % S::SLOTS;
@@ -205,7 +223,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
             if (item + 1 < 2 * nb) page_next = page_of(item_block(item + 1));
             if (round > 0) mbar_wait(kv_free0 + 8 * slot, (round - 1) & 1, 1);
             const bool is_v = item_is_v(item);
-            if (lane == 0) mbar_expect_tx(kv_full0 + 8 * slot, S::SLOT_BYTES);
+            if (lane == 0) mbar_expect_tx(kv_full0 + 8 * slot, is_v ? S::V_LOAD : S::K_LOAD);
             __syncwarp();
             // lane i's page continues lane i-1's in the pool; the largest aligned group of 2, 4, ... pages
             // around this lane whose pages all continue one another is fetched by its first lane
@@ -222,11 +240,15 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                 const int row = page >= 0 ? page * page_size : cache_rows;     // out of range: zeros
                 const PtMaps& maps = is_v ? maps_v : maps_k;
                 const uint32_t dst = slot_addr(slot) + lane * page_size * 128;
-                if (g == pages_per_block && big_boxes) {
-                    tma_load_3d(dst, &maps.blk, kv_full0 + 8 * slot, 0, row, kvh * S::CHUNKS);      // the whole block in one copy
+                const int head = is_v ? kvh / sz.v_share : kvh, chunks = is_v ? S::CHUNKS_V : S::CHUNKS;
+                if (sz.by_head & (is_v ? 2 : 1)) {
+                    for (int c = 0; c < chunks; ++c)
+                        tma_load_3d(dst + c * (PT_BN * 128), &maps.m[level], kv_full0 + 8 * slot, c * 64, head, row);
+                } else if (g == pages_per_block && big_boxes) {
+                    tma_load_3d(dst, &maps.blk, kv_full0 + 8 * slot, 0, row, head * chunks);         // the whole block in one copy
                 } else {
-                    for (int c = 0; c < S::CHUNKS; ++c)
-                        tma_load_2d(dst + c * (PT_BN * 128), &maps.m[level], kv_full0 + 8 * slot, kvh * HD + c * 64, row);
+                    for (int c = 0; c < chunks; ++c)
+                        tma_load_2d(dst + c * (PT_BN * 128), &maps.m[level], kv_full0 + 8 * slot, (head * chunks + c) * 64, row);
                 }
             }
         }
@@ -237,7 +259,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
         {
             const bool issuer = lane == 0;
             const uint32_t idesc_qk = umma_idesc_bf16(PT_BM, PT_BN, false);
-            const uint32_t idesc_pv = umma_idesc_bf16(PT_BM, HD, true);
+            const uint32_t idesc_pv = umma_idesc_bf16(PT_BM, HDV, true);
             const uint64_t desc_q0 = make_desc_sw128(sQ);
             // S[region] = Q(head) K^T from the K block in the slot at `b`
             auto qk = [&](int head, int region, uint32_t b, uint32_t bar) {
@@ -257,7 +279,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                 if (issuer) {
 #pragma unroll
                     for (int kk = 0; kk < PT_BN / 16; ++kk)
-                        umma_bf16_ts(tO0 + head * HD, tS0 + region * PT_BN + kk * 8, db + (uint64_t)((kk * 16 * 128) >> 4), idesc_pv, (kk > 0 || !first_block) ? 1u : 0u);
+                        umma_bf16_ts(tO0 + head * HDV, tS0 + region * PT_BN + kk * 8, db + (uint64_t)((kk * 16 * 128) >> 4), idesc_pv, (kk > 0 || !first_block) ? 1u : 0u);
                     umma_commit(bar);
                 }
             };
@@ -317,7 +339,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
         const int r = quarter * 32 + lane;
         const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
         // one head alone alternates between two score regions and two probability buffers (h is 0 then)
-        const uint32_t tS_base = tS0 + h * PT_BN + lane_off, tO = tO0 + h * HD + lane_off;
+        const uint32_t tS_base = tS0 + h * PT_BN + lane_off, tO = tO0 + h * HDV + lane_off;
         const int hi = r < rows ? pos0 + r : -1;                                 // last key this row sees
         const int lo = max((window > 0 && hi - window + 1 > 0) ? hi - window + 1 : 0, (chunk > 0 && hi > 0) ? (hi / chunk) * chunk : 0);
         // m_ref: the maximum the exponentials are taken against.  It follows the row's running
@@ -387,7 +409,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                         l_run *= f;
                     }
 #pragma unroll 1
-                    for (int c0 = 0; c0 < HD; c0 += 32) {
+                    for (int c0 = 0; c0 < HDV; c0 += 32) {
                         uint32_t o[32];
                         tmem_ld32(tO + c0, o);
                         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -437,9 +459,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
             const size_t prow = (((size_t)tile * PT_BM + r) * nq + head_a + h) * nsplit + split;
             part_ml[prow * 2] = m_ref;
             part_ml[prow * 2 + 1] = l_run;
-            float* dstf = part_o + prow * HD;
+            float* dstf = part_o + prow * HDV;
 #pragma unroll 1
-            for (int c0 = 0; c0 < HD; c0 += 32) {
+            for (int c0 = 0; c0 < HDV; c0 += 32) {
                 uint32_t o[32];
                 tmem_ld32(tO + c0, o);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -452,15 +474,24 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
         if (sinks != nullptr && m_ref != -INFINITY) l_run += ex2_approx(sinks[head_a + h] * 1.4426950408889634f - m_ref);
         float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
         if (ht.gate != nullptr && r < rows) inv *= 1.0f / (1.0f + expf(-__ldcg(ht.gate + (size_t)(qs + q0 + r) * ht.ldg + head_a + h)));
-        __nv_bfloat16* dst = out + (size_t)(qs + q0 + (r < rows ? r : 0)) * out_stride + (size_t)(head_a + h) * HD;
+        const size_t at = (size_t)(qs + q0 + (r < rows ? r : 0)) * out_stride + (size_t)(head_a + h) * sz.hdv;
+        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out_v) + at;
+        float* dst32 = reinterpret_cast<float*>(out_v) + at;
 #pragma unroll 1
-        for (int c0 = 0; c0 < HD; c0 += 32) {
+        for (int c0 = 0; c0 < HDV; c0 += 32) {
             uint32_t o[32];
             tmem_ld32(tO + c0, o);
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-            if (r < rows) {
+            if (r < rows && sz.out_f32) {
+#pragma unroll
+                for (int d = 0; d < 32; d += 4)
+                    if (c0 + d < sz.hdv)
+                        *reinterpret_cast<float4*>(dst32 + c0 + d) = make_float4(__uint_as_float(o[d]) * inv, __uint_as_float(o[d + 1]) * inv,
+                                                                                 __uint_as_float(o[d + 2]) * inv, __uint_as_float(o[d + 3]) * inv);
+            } else if (r < rows) {
 #pragma unroll
                 for (int d = 0; d < 32; d += 8) {
+                    if (c0 + d >= sz.hdv) break;
                     __nv_bfloat162 a = __floats2bfloat162_rn(__uint_as_float(o[d]) * inv, __uint_as_float(o[d + 1]) * inv);
                     __nv_bfloat162 b = __floats2bfloat162_rn(__uint_as_float(o[d + 2]) * inv, __uint_as_float(o[d + 3]) * inv);
                     __nv_bfloat162 c = __floats2bfloat162_rn(__uint_as_float(o[d + 4]) * inv, __uint_as_float(o[d + 5]) * inv);
@@ -490,8 +521,8 @@ constexpr int PT_MAX_SPLITS = 8;
 template <int HD>
 __global__ void __launch_bounds__(256) prefill_merge_splits_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                                    const int* __restrict__ q_start, const int* __restrict__ tile_seq,
-                                                                   const int* __restrict__ tile_q0, __nv_bfloat16* __restrict__ out,
-                                                                   long out_stride, int nq, int nsplit) {
+                                                                   const int* __restrict__ tile_q0, void* __restrict__ out_v,
+                                                                   long out_stride, int nq, int nsplit, int hdv, int out_f32) {
     constexpr int PER = HD / 32;
     griddep_launch();
     const int lane = threadIdx.x & 31;
@@ -537,18 +568,26 @@ __global__ void __launch_bounds__(256) prefill_merge_splits_kernel(const float* 
         for (int i = 0; i < PER; ++i) acc[i] = fmaf(w, o[sp][i], acc[i]);
     }
     const float inv = L > 0.f ? 1.0f / L : 0.f;
-    __nv_bfloat16* dst = out + (size_t)(qs + q0 + r) * out_stride + (size_t)head * HD + lane * PER;
+    if (lane * PER >= hdv) return;                       // columns that only pad the tile
+    const size_t at = (size_t)(qs + q0 + r) * out_stride + (size_t)head * hdv + lane * PER;
+    if (out_f32) {
+        float* dst = reinterpret_cast<float*>(out_v) + at;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) dst[i] = acc[i] * inv;
+        return;
+    }
+    __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out_v) + at;
 #pragma unroll
     for (int i = 0; i < PER; i += 2) *reinterpret_cast<__nv_bfloat162*>(dst + i) = __floats2bfloat162_rn(acc[i] * inv, acc[i + 1] * inv);
 }
 
-template <int HD>
+template <int HD, int HDV>
 static int launch_prefill_tc(const CUtensorMap& mq, const PtMaps& mk, const PtMaps& mv, int big_boxes, const int* bt, int max_blocks,
                              const int* q_start, const int* ctx_len, const int* tile_seq, const int* tile_q0, int num_tiles,
                              void* out, long out_stride, int nq, int nkv, int page_size, int window, float scale, int cache_rows,
                              void* scratch, long scratch_bytes, int max_ctx, int force_splits, int chunk, const float* sinks,
-                             const HeadTerms& ht, cudaStream_t stream) {
-    auto kern = prefill_tc_kernel<HD>;
+                             const HeadTerms& ht, const PtSizes& sz, cudaStream_t stream) {
+    auto kern = prefill_tc_kernel<HD, HDV>;
     // a chunk bounds the keys of a tile, and the merge of key ranges knows neither a sink nor a gate
     if (chunk > 0 || sinks != nullptr || ht.head_scale != nullptr || ht.slopes != nullptr || ht.gate != nullptr) {
         if (force_splits > 1) return AIEN_E_SHAPE;
@@ -557,7 +596,7 @@ static int launch_prefill_tc(const CUtensorMap& mq, const PtMaps& mk, const PtMa
     }
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, PtShape<HD>::SMEM) != cudaSuccess) return AIEN_E_STATE;
+        if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, PtShape<HD, HDV>::SMEM) != cudaSuccess) return AIEN_E_STATE;
         configured = true;
     }
     const int group = nq / nkv;
@@ -581,7 +620,7 @@ static int launch_prefill_tc(const CUtensorMap& mq, const PtMaps& mk, const PtMa
     int heads_per_cta = (group >= 2 && 18 * waves(single) > 25 * waves(paired)) ? 2 : 1;
     int nsplit = 1;
     const long part_rows = (long)num_tiles * PT_BM * nq;
-    auto fits = [&](int n) { return scratch != nullptr && part_rows * n * (HD + 2) * 4 <= scratch_bytes; };
+    auto fits = [&](int n) { return scratch != nullptr && part_rows * n * (HDV + 2) * 4 <= scratch_bytes; };
     if (force_splits > 0) {
         nsplit = force_splits;
         if (!fits(nsplit)) return AIEN_E_SHAPE;
@@ -596,14 +635,14 @@ static int launch_prefill_tc(const CUtensorMap& mq, const PtMaps& mk, const PtMa
     const long ctas = (long)num_tiles * nkv * ((group + heads_per_cta - 1) / heads_per_cta) * nsplit;
     if (ctas > 2147483647L) return AIEN_E_SHAPE;
     float* part_o = nsplit > 1 ? (float*)scratch : nullptr;
-    float* part_ml = nsplit > 1 ? part_o + part_rows * nsplit * HD : nullptr;
-    launch_chain(kern, dim3((unsigned)ctas), dim3(PT_THREADS), (size_t)PtShape<HD>::SMEM, stream, mq, mk, mv, bt, max_blocks, q_start, ctx_len, tile_seq, tile_q0, num_tiles,
-                                                                     (__nv_bfloat16*)out, out_stride, nq, nkv, page_size, window,
-                                                                     scale * 1.4426950408889634f, cache_rows, heads_per_cta, big_boxes, nsplit, part_o, part_ml, chunk, sinks, ht);
+    float* part_ml = nsplit > 1 ? part_o + part_rows * nsplit * HDV : nullptr;
+    launch_chain(kern, dim3((unsigned)ctas), dim3(PT_THREADS), (size_t)PtShape<HD, HDV>::SMEM, stream, mq, mk, mv, bt, max_blocks, q_start, ctx_len, tile_seq, tile_q0, num_tiles,
+                                                                     out, out_stride, nq, nkv, page_size, window,
+                                                                     scale * 1.4426950408889634f, cache_rows, heads_per_cta, big_boxes, nsplit, part_o, part_ml, chunk, sinks, ht, sz);
     if (launch_status() != 0) return launch_status();
     if (nsplit > 1)
-        launch_chain(prefill_merge_splits_kernel<HD>, dim3((unsigned)(part_rows / 8)), dim3(256), (size_t)0, stream, (const float*)part_o, (const float*)part_ml,
-                     q_start, tile_seq, tile_q0, (__nv_bfloat16*)out, out_stride, nq, nsplit);
+        launch_chain(prefill_merge_splits_kernel<HDV>, dim3((unsigned)(part_rows / 8)), dim3(256), (size_t)0, stream, (const float*)part_o, (const float*)part_ml,
+                     q_start, tile_seq, tile_q0, out, out_stride, nq, nsplit, sz.hdv, sz.out_f32);
     return launch_status();
 }
 
@@ -617,6 +656,12 @@ AIEN_API int aien_paged_attention_prefill_tc_supports(int hd, int page_size) {
     return ((hd == 64 || hd == 128) && page_size >= 8 && page_size <= 128 && (page_size & 7) == 0 && 128 % page_size == 0) ? 1 : 0;
 }
 
+// The same for keys and values of their own sizes (aien_paged_attention_prefill_tc_values).
+AIEN_API int aien_paged_attention_prefill_tc_values_supports(int hd, int hdv, int page_size) {
+    return (hd > 0 && hd <= 128 && (hd & 7) == 0 && hdv > 0 && hdv <= 128 && (hdv & 7) == 0 && page_size >= 8 && page_size <= 128 &&
+            (page_size & 7) == 0 && 128 % page_size == 0) ? 1 : 0;
+}
+
 // q [q_rows, nq*hd] (leading dimension q_stride), k_cache/v_cache [cache_rows, nkv*hd] contiguous;
 // the other arguments as aien_paged_attention_prefill.
 // scratch (may be null), scratch_bytes: room for the partial results of key ranges, num_tiles * 128 * nq *
@@ -626,44 +671,70 @@ AIEN_API int aien_paged_attention_prefill_tc_supports(int hd, int page_size) {
 // one more term exp(sink) in every head's softmax denominator.  With either, every tile's keys stay in one range.
 // head_scale, slopes (float32 [nq]) and gate (float32 [tokens of the step, ldg]), each of which may be null, and softcap
 // (0: none): see HeadTerms.
+// hdv, v_share, out_f32: values of hdv numbers, one value head for every v_share neighbouring key heads (v_cache
+// [cache_rows, nkv / v_share * hdv], out [tokens, nq * hdv]), float32 results; hd and hdv are multiples of 8 up to 128.
+AIEN_API int aien_paged_attention_prefill_tc_values(
+    const void* q, long q_stride, int q_rows, const void* k_cache, const void* v_cache, int cache_rows, const int* block_table,
+    int max_blocks, const int* q_start, const int* ctx_len, const int* tile_seq, const int* tile_q0, int num_tiles, void* out,
+    long out_stride, int nq, int nkv, int hd, int page_size, int window, float scale, void* scratch, long scratch_bytes, int max_ctx,
+    int force_splits, int chunk, const float* sinks, const float* head_scale, const float* slopes, const float* gate, long ldg,
+    float softcap, int hdv, int v_share, int out_f32, cudaStream_t stream) {
+    const HeadTerms ht{head_scale, slopes, gate, ldg, softcap > 0.f ? softcap : 0.f};
+    if (num_tiles <= 0) return 0;
+    if (chunk < 0) return AIEN_E_SHAPE;
+    if (!aien_paged_attention_prefill_tc_values_supports(hd, hdv, page_size) || nkv <= 0 || nq % nkv != 0 || q_rows <= 0 || cache_rows <= 0 ||
+        v_share <= 0 || nkv % v_share != 0)
+        return AIEN_E_SHAPE;
+    if ((q_stride & 7) || (out_stride & 7) || ((uintptr_t)q & 15) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15) ||
+        ((uintptr_t)out & 15) || ((uintptr_t)scratch & 15))
+        return AIEN_E_ALIGN;
+    if (force_splits < 0 || force_splits > PT_MAX_SPLITS) return AIEN_E_SHAPE;
+    const PtSizes sz{hdv, ((hd & 63) ? 1 : 0) | ((hdv & 63) ? 2 : 0), v_share, out_f32 ? 1 : 0};
+    CUtensorMap mq;
+    static PtMaps mk, mv;                      // large: kept out of the stack; filled for every launch
+    static std::mutex mu;
+    std::lock_guard<std::mutex> lock(mu);
+    const int nv = nkv / v_share;
+    const uint64_t k_cols = (uint64_t)nkv * hd, v_cols = (uint64_t)nv * hdv;
+    auto rows_of = [&](CUtensorMap* m, const void* p, uint64_t rows, int heads, int size, uint64_t ld, bool by_head, uint32_t box_rows) {
+        return by_head ? make_map_heads(m, p, rows, (uint64_t)heads, (uint64_t)size, ld, box_rows)
+                       : make_map(m, p, rows, (uint64_t)heads * size, ld, 64, box_rows);
+    };
+    const bool kh = sz.by_head & 1, vh = sz.by_head & 2;
+    if (!rows_of(&mq, q, (uint64_t)q_rows, nq, hd, (uint64_t)q_stride, kh, PT_BM)) return AIEN_E_STATE;
+    for (int lv = 0; lv < 5; ++lv) {
+        const uint32_t rows = (uint32_t)page_size << lv;
+        if (rows > (uint32_t)PT_BN) { mk.m[lv] = mk.m[0]; mv.m[lv] = mv.m[0]; continue; }
+        if (!rows_of(&mk.m[lv], k_cache, (uint64_t)cache_rows, nkv, hd, k_cols, kh, rows) ||
+            !rows_of(&mv.m[lv], v_cache, (uint64_t)cache_rows, nv, hdv, v_cols, vh, rows))
+            return AIEN_E_STATE;
+    }
+    // one copy for a whole block of 128 keys, when the pool has that many rows at all and heads are whole chunks
+    int big_boxes = cache_rows >= PT_BN ? 1 : 0;
+    if (big_boxes && !kh) big_boxes = make_map_chunked(&mk.blk, k_cache, (uint64_t)cache_rows, k_cols, k_cols, PT_BN, (uint32_t)(hd / 64)) ? 1 : 0;
+    if (big_boxes && !vh) big_boxes = make_map_chunked(&mv.blk, v_cache, (uint64_t)cache_rows, v_cols, v_cols, PT_BN, (uint32_t)(hdv / 64)) ? 1 : 0;
+    if (!big_boxes || kh) mk.blk = mk.m[0];
+    if (!big_boxes || vh) mv.blk = mv.m[0];
+#define PT_CASE(HDV_, HVV_)                                                                                                        \
+    return launch_prefill_tc<HDV_, HVV_>(mq, mk, mv, big_boxes, block_table, max_blocks, q_start, ctx_len, tile_seq, tile_q0, num_tiles, out, \
+                                         out_stride, nq, nkv, page_size, window, scale, cache_rows, scratch, scratch_bytes, max_ctx,       \
+                                         force_splits, chunk, sinks, ht, sz, stream)
+    if (hd <= 64) { if (hdv <= 64) PT_CASE(64, 64); else PT_CASE(64, 128); }
+    if (hdv <= 64) PT_CASE(128, 64); else PT_CASE(128, 128);
+#undef PT_CASE
+}
+
 AIEN_API int aien_paged_attention_prefill_tc_terms(
     const void* q, long q_stride, int q_rows, const void* k_cache, const void* v_cache, int cache_rows, const int* block_table,
     int max_blocks, const int* q_start, const int* ctx_len, const int* tile_seq, const int* tile_q0, int num_tiles, void* out,
     long out_stride, int nq, int nkv, int hd, int page_size, int window, float scale, void* scratch, long scratch_bytes, int max_ctx,
     int force_splits, int chunk, const float* sinks, const float* head_scale, const float* slopes, const float* gate, long ldg,
     float softcap, cudaStream_t stream) {
-    const HeadTerms ht{head_scale, slopes, gate, ldg, softcap > 0.f ? softcap : 0.f};
-    if (num_tiles <= 0) return 0;
-    if (chunk < 0) return AIEN_E_SHAPE;
-    if (!aien_paged_attention_prefill_tc_supports(hd, page_size) || nkv <= 0 || nq % nkv != 0 || q_rows <= 0 || cache_rows <= 0)
-        return AIEN_E_SHAPE;
-    if ((q_stride & 7) || (out_stride & 7) || ((uintptr_t)q & 15) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15) ||
-        ((uintptr_t)out & 15) || ((uintptr_t)scratch & 15))
-        return AIEN_E_ALIGN;
-    if (force_splits < 0 || force_splits > PT_MAX_SPLITS) return AIEN_E_SHAPE;
-    CUtensorMap mq;
-    static PtMaps mk, mv;                      // large: kept out of the stack; filled for every launch
-    static std::mutex mu;
-    std::lock_guard<std::mutex> lock(mu);
-    const uint64_t kv_cols = (uint64_t)nkv * hd;
-    if (!make_map(&mq, q, (uint64_t)q_rows, (uint64_t)nq * hd, (uint64_t)q_stride, 64, PT_BM)) return AIEN_E_STATE;
-    for (int lv = 0; lv < 5; ++lv) {
-        const uint32_t rows = (uint32_t)page_size << lv;
-        if (rows > (uint32_t)PT_BN) { mk.m[lv] = mk.m[0]; mv.m[lv] = mv.m[0]; continue; }
-        if (!make_map(&mk.m[lv], k_cache, (uint64_t)cache_rows, kv_cols, kv_cols, 64, rows) ||
-            !make_map(&mv.m[lv], v_cache, (uint64_t)cache_rows, kv_cols, kv_cols, 64, rows))
-            return AIEN_E_STATE;
-    }
-    // one copy for a whole block of 128 keys, when the pool has that many rows at all
-    const int big_boxes = cache_rows >= PT_BN &&
-                          make_map_chunked(&mk.blk, k_cache, (uint64_t)cache_rows, kv_cols, kv_cols, PT_BN, (uint32_t)(hd / 64)) &&
-                          make_map_chunked(&mv.blk, v_cache, (uint64_t)cache_rows, kv_cols, kv_cols, PT_BN, (uint32_t)(hd / 64)) ? 1 : 0;
-    if (!big_boxes) { mk.blk = mk.m[0]; mv.blk = mv.m[0]; }
-    if (hd == 64)
-        return launch_prefill_tc<64>(mq, mk, mv, big_boxes, block_table, max_blocks, q_start, ctx_len, tile_seq, tile_q0, num_tiles, out, out_stride,
-                                     nq, nkv, page_size, window, scale, cache_rows, scratch, scratch_bytes, max_ctx, force_splits, chunk, sinks, ht, stream);
-    return launch_prefill_tc<128>(mq, mk, mv, big_boxes, block_table, max_blocks, q_start, ctx_len, tile_seq, tile_q0, num_tiles, out, out_stride,
-                                  nq, nkv, page_size, window, scale, cache_rows, scratch, scratch_bytes, max_ctx, force_splits, chunk, sinks, ht, stream);
+    if (num_tiles > 0 && !aien_paged_attention_prefill_tc_supports(hd, page_size)) return AIEN_E_SHAPE;
+    return aien_paged_attention_prefill_tc_values(q, q_stride, q_rows, k_cache, v_cache, cache_rows, block_table, max_blocks, q_start, ctx_len,
+                                                  tile_seq, tile_q0, num_tiles, out, out_stride, nq, nkv, hd, page_size, window, scale,
+                                                  scratch, scratch_bytes, max_ctx, force_splits, chunk, sinks, head_scale, slopes, gate, ldg,
+                                                  softcap, hd, 1, 0, stream);
 }
 
 AIEN_API int aien_paged_attention_prefill_tc_masked(

@@ -129,23 +129,29 @@ branch_norm_add_vec_kernel(float* __restrict__ x, const TA* __restrict__ a, int 
     }
 }
 
-// x[t] = x[t] / sqrt(mean(x[t]^2) + eps) * w in place (the norm of the embedding row), h as above.
+// x[t] = x[t] / sqrt(mean(x[t]^2) + eps) * w in place (the norm of the embedding row), h as above; center != 0: the layer
+// norm, whose mean is taken off first.
 template <typename TH>
 __global__ void __launch_bounds__(BN_THREADS)
-stream_norm_inplace_kernel(float* __restrict__ x, const void* __restrict__ w, int wdt, float eps, TH* __restrict__ h, int H) {
+stream_norm_inplace_kernel(float* __restrict__ x, const void* __restrict__ w, int wdt, float eps, TH* __restrict__ h, int H, int center) {
     __shared__ float red[32];
     griddep_launch();
     griddep_wait();
     const size_t base = (size_t)blockIdx.x * H;
-    float ss = 0.f;
+    float ss = 0.f, mean = 0.f;
+    if (center) {
+        float sm = 0.f;
+        for (int i = threadIdx.x; i < H; i += BN_THREADS) sm += __ldcg(x + base + i);
+        mean = block_sum(sm, red) / (float)H;
+    }
     for (int i = threadIdx.x; i < H; i += BN_THREADS) {
-        const float v = __ldcg(x + base + i);
+        const float v = __ldcg(x + base + i) - mean;
         ss += v * v;
     }
     const float total = block_sum(ss, red);
     const float scale = 1.0f / sqrtf(total / (float)H + eps);
     for (int i = threadIdx.x; i < H; i += BN_THREADS) {
-        const float r = __ldcg(x + base + i) * scale * load_dyn(w, wdt, i);
+        const float r = (__ldcg(x + base + i) - mean) * scale * load_dyn(w, wdt, i);
         x[base + i] = r;
         if (h != nullptr) h[base + i] = from_f<TH>(r);
     }
@@ -187,10 +193,10 @@ AIEN_API int aien_branch_norm_add(float* x, const void* a, int a_dt, int a_parts
 }
 
 AIEN_API int aien_stream_norm_inplace(float* x, const void* w, int w_dt, float eps, void* h, int h_dt, int T, int H,
-                                      cudaStream_t stream) {
+                                      int center, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (H <= 0) return AIEN_E_SHAPE;
     AIEN_DISPATCH_DTYPE(h_dt, TH,
-        (launch_chain(stream_norm_inplace_kernel<TH>, dim3(T), dim3(BN_THREADS), 0, stream, x, w, w_dt, eps, (TH*)h, H)));
+        (launch_chain(stream_norm_inplace_kernel<TH>, dim3(T), dim3(BN_THREADS), 0, stream, x, w, w_dt, eps, (TH*)h, H, center)));
     return launch_status();
 }

@@ -1,4 +1,4 @@
-// Row-wise kernels of the decoder: embedding gather, fused residual-add + RMSNorm, SwiGLU,
+// Row-wise kernels of the decoder: embedding gather, fused residual-add + RMSNorm or layer norm, gated activations,
 // rotary table, fused per-head q/k RMSNorm + rotation + cache write, row gather.
 //
 // The residual stream is float32 in both engine precisions; norms and rotation are computed
@@ -34,7 +34,9 @@ __device__ __forceinline__ float delta_sum(const TD* __restrict__ delta, int npa
     return d;
 }
 
-template <typename TD, typename TO>
+// CENTER: the layer norm, h[t] = (x[t] - mean) * (1/sqrt(mean((x - mean)^2) + eps)) * w; the deviations are taken from the
+// finished mean, in a pass of their own.
+template <typename TD, typename TO, bool CENTER>
 __global__ void add_rmsnorm_kernel(float* __restrict__ x, const TD* __restrict__ delta, int nparts, size_t part_stride,
                                    const void* __restrict__ w, int wdt, float eps,
                                    TO* __restrict__ h, int H) {
@@ -49,12 +51,21 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ x, const TD* __restrict__
             v += delta_sum(delta, nparts, part_stride, base + i);
             x[base + i] = v;
         }
-        ss += v * v;
+        ss += CENTER ? v : v * v;
     }
-    const float total = block_sum(ss, red);
+    float total = block_sum(ss, red), mean = 0.f;
+    if (CENTER) {
+        mean = total / (float)H;
+        ss = 0.f;
+        for (int i = threadIdx.x; i < H; i += blockDim.x) {
+            const float d = x[base + i] - mean;
+            ss += d * d;
+        }
+        total = block_sum(ss, red);
+    }
     const float scale = 1.0f / sqrtf(total / (float)H + eps);
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        h[base + i] = from_f<TO>(x[base + i] * scale * load_dyn(w, wdt, i));
+        h[base + i] = from_f<TO>((x[base + i] - mean) * scale * load_dyn(w, wdt, i));
     }
 }
 
@@ -83,7 +94,7 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
 // PARTS: the pending sum comes in several parts (the register budget of that case is its own).
 // BS threads a row: 256, or 1,024 for steps of so few rows that the grid leaves most SMs empty; a
 // thread then holds one vector of the row and has every load it makes in flight at once.
-template <typename TD, typename TO, int NV, bool PARTS, int BS>
+template <typename TD, typename TO, int NV, bool PARTS, int BS, bool CENTER>
 __global__ void __launch_bounds__(BS)
 add_rmsnorm_vec_kernel(float* __restrict__ x, const TD* __restrict__ delta, int nparts, size_t part_stride,
                        const void* __restrict__ w, int wdt, float eps, TO* __restrict__ h, int H) {
@@ -138,6 +149,20 @@ add_rmsnorm_vec_kernel(float* __restrict__ x, const TD* __restrict__ delta, int 
             }
         }
     }
+    if (CENTER) {                                                    // the sum goes back first: v then holds the deviations
+        float sm = 0.f;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) sm += (v[j].x + v[j].y) + (v[j].z + v[j].w);
+        const float mean = block_sum(sm, red) / (float)H;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = (j * BS + threadIdx.x) * 4;
+            if (i < H) {
+                if (delta != nullptr) store4(x + base + i, v[j]);
+                v[j].x -= mean; v[j].y -= mean; v[j].z -= mean; v[j].w -= mean;
+            }
+        }
+    }
     float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < NV; ++j) ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
@@ -147,7 +172,7 @@ add_rmsnorm_vec_kernel(float* __restrict__ x, const TD* __restrict__ delta, int 
     for (int j = 0; j < NV; ++j) {
         const int i = (j * BS + threadIdx.x) * 4;
         if (i < H) {
-            if (delta != nullptr) store4(x + base + i, v[j]);
+            if (!CENTER && delta != nullptr) store4(x + base + i, v[j]);
             store4(h + base + i, make_float4(v[j].x * scale * wv[j].x, v[j].y * scale * wv[j].y,
                                              v[j].z * scale * wv[j].z, v[j].w * scale * wv[j].w));
         }
@@ -178,12 +203,12 @@ __global__ void add_residual_kernel(float* __restrict__ x, const TD* __restrict_
     for (; idx < total; idx += stride) x[idx] = ld_act(x + idx) + delta_sum(delta, nparts, part_stride, idx);
 }
 
-// ---------------------------------------------------------------- SwiGLU
-// a = silu(g) * u, silu(g) = g / (1 + exp(-g))     (backend.rs:572-579).  gu = [T, 2I]:
+// ---------------------------------------------------------------- gated activations
+// a = f(g) * u, f = silu: g / (1 + exp(-g)) (backend.rs:572-579), or (gelu != 0) the tanh form of the gelu.  gu = [T, 2I]:
 // group == 0: gate columns [0, I), up columns [I, 2I);  group > 0: columns interleaved in runs of
 // `group` (gate run, then the matching up run), the layout the fused decode product wants.
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int I, int group, size_t total) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int I, int group, int gelu, size_t total) {
     griddep_launch();
     griddep_wait();
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -195,20 +220,21 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
         else { gi = (i / group) * 2 * group + (i % group); ui = gi + group; }
         const float g = ld_act(gu + t * 2 * I + gi);
         const float u = ld_act(gu + t * 2 * I + ui);
-        out[idx] = from_f<T>(g / (1.0f + expf(-g)) * u);
+        const float f = gelu ? 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : g / (1.0f + expf(-g));
+        out[idx] = from_f<T>(f * u);
     }
 }
 
 // ---------------------------------------------------------------- rotary table
 __global__ void rope_table_kernel(const int* __restrict__ positions, const double* __restrict__ inv_freq,
-                                  float* __restrict__ cos_t, float* __restrict__ sin_t, int T, int half) {
+                                  float* __restrict__ cos_t, float* __restrict__ sin_t, int T, int half, double mult) {
     const int idx = blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= T * half) return;
     const int t = idx / half, i = idx - t * half;
     double s, c;
     sincos((double)positions[t] * inv_freq[i], &s, &c);
-    cos_t[idx] = (float)c;
-    sin_t[idx] = (float)s;
+    cos_t[idx] = (float)(c * mult);                   // mult: 1, or the factor that some frequency scalings put on both
+    sin_t[idx] = (float)(s * mult);
 }
 
 // ---------------------------------------------------------------- q/k norm + rotation + cache write
@@ -685,7 +711,7 @@ AIEN_API int aien_embed_gather(const void* table, int table_dt, const int* ids, 
     return launch_status();
 }
 
-template <typename TD, typename TO>
+template <typename TD, typename TO, bool CENTER>
 static void launch_add_rmsnorm(float* x, const TD* delta, int nparts, size_t part_stride, const void* w, int w_dt,
                                float eps, TO* h, int T, int H, cudaStream_t stream) {
     const bool vec = (H % 4 == 0) && (((uintptr_t)x & 15) == 0) && (((uintptr_t)delta & 15) == 0) && (((uintptr_t)h & 15) == 0) &&
@@ -693,9 +719,9 @@ static void launch_add_rmsnorm(float* x, const TD* delta, int nparts, size_t par
 #define VEC_CASE(NV, BS)                                                                                                          \
     do {                                                                                                                          \
         if (delta != nullptr && nparts > 1)                                                                                       \
-            launch_chain(add_rmsnorm_vec_kernel<TD, TO, NV, true, BS>, dim3(T), dim3(BS), 0, stream, x, delta, nparts, part_stride, w, w_dt, eps, h, H); \
+            launch_chain(add_rmsnorm_vec_kernel<TD, TO, NV, true, BS, CENTER>, dim3(T), dim3(BS), 0, stream, x, delta, nparts, part_stride, w, w_dt, eps, h, H); \
         else                                                                                                                      \
-            launch_chain(add_rmsnorm_vec_kernel<TD, TO, NV, false, BS>, dim3(T), dim3(BS), 0, stream, x, delta, nparts, part_stride, w, w_dt, eps, h, H); \
+            launch_chain(add_rmsnorm_vec_kernel<TD, TO, NV, false, BS, CENTER>, dim3(T), dim3(BS), 0, stream, x, delta, nparts, part_stride, w, w_dt, eps, h, H); \
     } while (0)
     // fewer rows than SMs: the rows' latency is the kernel's time, so more threads share a row
     const bool few_rows = T <= 148 && H > 256 * 4;
@@ -710,7 +736,7 @@ static void launch_add_rmsnorm(float* x, const TD* delta, int nparts, size_t par
     else if (vec && H <= 256 * 4 * 8)
         VEC_CASE(8, 256);
     else
-        launch_chain(add_rmsnorm_kernel<TD, TO>, dim3(T), dim3(row_threads(H)), 0, stream, x, delta, nparts, part_stride, w, w_dt, eps, h, H);
+        launch_chain(add_rmsnorm_kernel<TD, TO, CENTER>, dim3(T), dim3(row_threads(H)), 0, stream, x, delta, nparts, part_stride, w, w_dt, eps, h, H);
 #undef VEC_CASE
 }
 
@@ -720,7 +746,17 @@ AIEN_API int aien_add_rmsnorm(float* x, const void* delta, int delta_dt, int npa
     if (T <= 0) return 0;
     if (delta != nullptr && nparts < 1) return AIEN_E_SHAPE;
     AIEN_DISPATCH_DTYPE(delta_dt, TD, AIEN_DISPATCH_DTYPE(h_dt, TO,
-        (launch_add_rmsnorm<TD, TO>(x, (const TD*)delta, nparts, part_stride, w, w_dt, eps, (TO*)h, T, H, stream))));
+        (launch_add_rmsnorm<TD, TO, false>(x, (const TD*)delta, nparts, part_stride, w, w_dt, eps, (TO*)h, T, H, stream))));
+    return launch_status();
+}
+
+// The same with the layer norm (weight, no bias) in the RMS norm's place.
+AIEN_API int aien_add_layernorm(float* x, const void* delta, int delta_dt, int nparts, size_t part_stride,
+                                const void* w, int w_dt, float eps, void* h, int h_dt, int T, int H, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (delta != nullptr && nparts < 1) return AIEN_E_SHAPE;
+    AIEN_DISPATCH_DTYPE(delta_dt, TD, AIEN_DISPATCH_DTYPE(h_dt, TO,
+        (launch_add_rmsnorm<TD, TO, true>(x, (const TD*)delta, nparts, part_stride, w, w_dt, eps, (TO*)h, T, H, stream))));
     return launch_status();
 }
 
@@ -833,20 +869,20 @@ AIEN_API int aien_add_residual(float* x, const void* delta, int delta_dt, int np
     return launch_status();
 }
 
-AIEN_API int aien_swiglu(const void* gu, void* out, int dt, int T, int I, int group, cudaStream_t stream) {
+AIEN_API int aien_swiglu(const void* gu, void* out, int dt, int T, int I, int group, int gelu, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (group < 0 || (group > 0 && I % group != 0)) return AIEN_E_SHAPE;
     const size_t total = (size_t)T * I;
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
-    AIEN_DISPATCH_DTYPE(dt, TT, (launch_chain(swiglu_kernel<TT>, dim3(blocks), dim3(256), 0, stream, (const TT*)gu, (TT*)out, I, group, total)));
+    AIEN_DISPATCH_DTYPE(dt, TT, (launch_chain(swiglu_kernel<TT>, dim3(blocks), dim3(256), 0, stream, (const TT*)gu, (TT*)out, I, group, gelu, total)));
     return launch_status();
 }
 
 AIEN_API int aien_rope_table(const int* positions, const double* inv_freq, float* cos_t, float* sin_t,
-                             int T, int half, cudaStream_t stream) {
+                             int T, int half, double mult, cudaStream_t stream) {
     if (T <= 0 || half <= 0) return 0;
     const int n = T * half;
-    rope_table_kernel<<<(n + 127) / 128, 128, 0, stream>>>(positions, inv_freq, cos_t, sin_t, T, half);
+    rope_table_kernel<<<(n + 127) / 128, 128, 0, stream>>>(positions, inv_freq, cos_t, sin_t, T, half, mult);
     return launch_status();
 }
 

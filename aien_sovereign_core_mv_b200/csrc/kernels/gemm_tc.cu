@@ -47,7 +47,8 @@ __device__ __forceinline__ float tc_gelu_tanh(float z) { return 0.5f * z * (1.0f
 
 // Stores 32 consecutive accumulator columns of one row: r holds columns n0+c0 .. +31 of row `row`.
 // EPI 0: as they are; EPI 1: silu(gate)*up over columns interleaved in runs of 8 (out has N/2 columns);
-// EPI 2 / 3: the gelu in its erf / tanh form of every value; EPI 4: the square of relu.
+// EPI 2 / 3: the gelu in its erf / tanh form of every value; EPI 4: the square of relu; EPI 6: EPI 1 with the tanh form of the
+// gelu in silu's place.
 template <int EPI, typename TC>
 __device__ __forceinline__ void tc_store_chunk(const uint32_t r_in[32], TC* __restrict__ out, long ldc, int row, int n0, int c0, int N) {
                 uint32_t r[32];
@@ -56,7 +57,7 @@ __device__ __forceinline__ void tc_store_chunk(const uint32_t r_in[32], TC* __re
                     r[j] = EPI == 2 ? __float_as_uint(tc_gelu_erf(__uint_as_float(r_in[j])))
                                     : (EPI == 3 ? __float_as_uint(tc_gelu_tanh(__uint_as_float(r_in[j])))
                                                 : (EPI == 4 ? __float_as_uint(tc_relu2(__uint_as_float(r_in[j]))) : r_in[j]));
-                if (EPI != 1) {
+                if (EPI != 1 && EPI != 6) {
                     TC* dst = out + (size_t)row * ldc + n0 + c0;
                     const int valid = N - (n0 + c0);
                     if (valid >= 32 && (((uintptr_t)dst & 15) == 0)) {
@@ -94,7 +95,8 @@ __device__ __forceinline__ void tc_store_chunk(const uint32_t r_in[32], TC* __re
 #pragma unroll
                         for (int j = 0; j < 8; ++j) {
                             const float g = __uint_as_float(r[run * 16 + j]), u = __uint_as_float(r[run * 16 + 8 + j]);
-                            y[run * 8 + j] = __fdividef(g, 1.0f + __expf(-g)) * u;
+                            if (EPI == 6) y[run * 8 + j] = 0.5f * g * (1.0f + tanh_ex2(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+                            else y[run * 8 + j] = __fdividef(g, 1.0f + __expf(-g)) * u;
                         }
                     if (valid >= 16 && sizeof(TC) == 2 && (((uintptr_t)dst & 15) == 0)) {
                         uint4* d4 = reinterpret_cast<uint4*>(dst);
@@ -813,7 +815,8 @@ static int launch_tc(const void* A, long lda, const void* W, long ldw, void* out
 
 using namespace aien;
 
-// epilogue 0: out[M,N]; 1: out[M,N/2] = silu(gate)*up with gate/up rows of W interleaved in runs of 8;
+// epilogue 0: out[M,N]; 1: out[M,N/2] = silu(gate)*up with gate/up rows of W interleaved in runs of 8 (6: the same with the
+// tanh form of the gelu in silu's place, bfloat16);
 // 2 / 3: out[M,N] = gelu (erf / tanh form) of the product, bfloat16.
 // splits > 1 (epilogue 0, float32 out): K is cut into ranges of whole 64-value blocks and out is
 // [ranges][M][ldc] partial products, part_stride elements apart; aien_gemm_tc_ranges says how many
@@ -838,9 +841,9 @@ AIEN_API int aien_gemm_tc(const void* A, long lda, const void* W, long ldw, void
     if (K <= 0 || (K & 7) || splits < 1 || splits > 64) return AIEN_E_SHAPE;
     if (splits > 1 && (epilogue != 0 || c_dt != AIEN_DT_F32)) return AIEN_E_SHAPE;
     if ((lda & 7) || (ldw & 7) || ((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return AIEN_E_ALIGN;
-    if (epilogue == 1 && (N & 15)) return AIEN_E_SHAPE;
+    if ((epilogue == 1 || epilogue == 6) && (N & 15)) return AIEN_E_SHAPE;
     if ((M + TC_BM - 1) / TC_BM > 2147483647 / 1 || (N + 95) / 96 > 65535) return AIEN_E_SHAPE;
-    if (epilogue == 2 || epilogue == 3 || epilogue == 4) {   // gelu (erf / tanh form) or relu squared of every value, bfloat16 out, K in one range
+    if (epilogue == 2 || epilogue == 3 || epilogue == 4 || epilogue == 6) {   // gelu (erf / tanh form) or relu squared of every value, bfloat16 out, K in one range
         if (c_dt != AIEN_DT_BF16 || splits != 1) return AIEN_E_SHAPE;
         const int plan = tc_plan(M, N, 1);
         const int wide = plan == 256 ? tc_m256_cols(M, N, K, 1) : 0;
@@ -848,6 +851,11 @@ AIEN_API int aien_gemm_tc(const void* A, long lda, const void* W, long ldw, void
             if (wide > 0) return launch_tc_persistent_m256<2, __nv_bfloat16>(wide, A, lda, W, ldw, out, ldc, M, N, K, stream);
             if (plan == 256) return launch_tc_persistent<256, 2, __nv_bfloat16>(A, lda, W, ldw, out, ldc, M, N, K, 1, 0, stream);
             return launch_tc<2, __nv_bfloat16>(A, lda, W, ldw, out, ldc, 1, 0, M, N, K, stream);
+        }
+        if (epilogue == 6) {
+            if (wide > 0) return launch_tc_persistent_m256<6, __nv_bfloat16>(wide, A, lda, W, ldw, out, ldc, M, N, K, stream);
+            if (plan == 256) return launch_tc_persistent<256, 6, __nv_bfloat16>(A, lda, W, ldw, out, ldc, M, N, K, 1, 0, stream);
+            return launch_tc<6, __nv_bfloat16>(A, lda, W, ldw, out, ldc, 1, 0, M, N, K, stream);
         }
         if (epilogue == 4) {
             if (wide > 0) return launch_tc_persistent_m256<4, __nv_bfloat16>(wide, A, lda, W, ldw, out, ldc, M, N, K, stream);

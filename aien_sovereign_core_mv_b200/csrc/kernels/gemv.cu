@@ -139,8 +139,14 @@ gemv_mma_kernel(const __nv_bfloat16* __restrict__ a, long lda, const __nv_bfloat
         } else {
             const int col = blockIdx.x * 8 + g;                 // output column of this gate/up pair
             if (v1) {
-                const float y0 = sum[0] / (1.0f + expf(-sum[0])) * sum[2];
-                const float y1 = sum[1] / (1.0f + expf(-sum[1])) * sum[3];
+                float y0, y1;
+                if (EPI == 6) {                                  // the tanh form of the gelu in silu's place
+                    y0 = 0.5f * sum[0] * (1.0f + tanhf(0.7978845608028654f * (sum[0] + 0.044715f * sum[0] * sum[0] * sum[0]))) * sum[2];
+                    y1 = 0.5f * sum[1] * (1.0f + tanhf(0.7978845608028654f * (sum[1] + 0.044715f * sum[1] * sum[1] * sum[1]))) * sum[3];
+                } else {
+                    y0 = sum[0] / (1.0f + expf(-sum[0])) * sum[2];
+                    y1 = sum[1] / (1.0f + expf(-sum[1])) * sum[3];
+                }
                 if (t0 < M) out[(size_t)t0 * ldc + col] = from_f<TC>(y0);
                 if (t0 + 1 < M) out[(size_t)(t0 + 1) * ldc + col] = from_f<TC>(y1);
             }
@@ -171,7 +177,8 @@ static int launch_gemv(const void* a, long lda, const void* W, long ldw, void* o
 
 using namespace aien;
 
-// epilogue: 0 plain, 1 silu(gate)*up over rows interleaved in groups of 8 (N counts both).
+// epilogue: 0 plain, 1 silu(gate)*up over rows interleaved in groups of 8 (N counts both), 6 the same with the tanh form of
+// the gelu in silu's place.
 // splits > 1: K is cut into `splits` ranges, out is float32 [splits][M][ldc] partial products
 // (part_stride elements apart) for the consumer to add; only with epilogue 0.
 AIEN_API int aien_gemv_bf16(const void* a, long lda, const void* W, long ldw, void* out, int c_dt, long ldc,
@@ -180,7 +187,7 @@ AIEN_API int aien_gemv_bf16(const void* a, long lda, const void* W, long ldw, vo
     if (M > 16 || K <= 0 || (K & 7) || splits < 1 || splits > 64) return AIEN_E_SHAPE;
     if (splits > 1 && epilogue != 0) return AIEN_E_SHAPE;
     if ((lda & 7) || (ldw & 7) || ((uintptr_t)a & 15) || ((uintptr_t)W & 15)) return AIEN_E_ALIGN;
-    if (epilogue == 1 && (N & 15)) return AIEN_E_SHAPE;
+    if ((epilogue == 1 || epilogue == 6) && (N & 15)) return AIEN_E_SHAPE;
     if (epilogue == 0) {
         return M <= 8 ? launch_gemv<1, 0>(a, lda, W, ldw, out, c_dt, ldc, splits, part_stride, M, N, K, stream)
                       : launch_gemv<2, 0>(a, lda, W, ldw, out, c_dt, ldc, splits, part_stride, M, N, K, stream);
@@ -188,6 +195,10 @@ AIEN_API int aien_gemv_bf16(const void* a, long lda, const void* W, long ldw, vo
     if (epilogue == 1) {
         return M <= 8 ? launch_gemv<1, 1>(a, lda, W, ldw, out, c_dt, ldc, 1, 0, M, N, K, stream)
                       : launch_gemv<2, 1>(a, lda, W, ldw, out, c_dt, ldc, 1, 0, M, N, K, stream);
+    }
+    if (epilogue == 6) {
+        return M <= 8 ? launch_gemv<1, 6>(a, lda, W, ldw, out, c_dt, ldc, 1, 0, M, N, K, stream)
+                      : launch_gemv<2, 6>(a, lda, W, ldw, out, c_dt, ldc, 1, 0, M, N, K, stream);
     }
     return AIEN_E_SHAPE;
 }

@@ -59,7 +59,8 @@ struct GsFuse {
     float* ssq_out;            // [gridDim.x][16]
 };
 
-// MT token tiles of 8; EPI 0 store / 1 swiglu / 2 residual / 3, 4 gelu (erf, tanh form) then store; STAGES ring depth
+// MT token tiles of 8; EPI 0 store / 1 swiglu / 2 residual / 3, 4 gelu (erf, tanh form) then store / 6 swiglu with the tanh form
+// of the gelu in silu's place; STAGES ring depth
 template <int MT, int EPI, typename TC, int STAGES>
 __global__ void __launch_bounds__(GS_THREADS, 1)
 gemv_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_a,
@@ -232,7 +233,7 @@ gemv_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
                             ss[mt][i & 1] += xn * xn;
                         }
                     }
-                } else if (EPI == 0 || EPI >= 3) {
+                } else if (EPI == 0 || (EPI >= 3 && EPI <= 5)) {
                     if (EPI == 3) {
 #pragma unroll
                         for (int i = 0; i < 4; ++i) sum[i] = 0.5f * sum[i] * (1.0f + erff(sum[i] * 0.7071067811865476f));
@@ -253,8 +254,14 @@ gemv_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
                     }
                 } else if (r1 < N) {
                     const int col = tile * 8 + g;
-                    const float y0 = sum[0] / (1.0f + expf(-sum[0])) * sum[2];
-                    const float y1 = sum[1] / (1.0f + expf(-sum[1])) * sum[3];
+                    float y0, y1;
+                    if (EPI == 6) {
+                        y0 = 0.5f * sum[0] * (1.0f + tanhf(0.7978845608028654f * (sum[0] + 0.044715f * sum[0] * sum[0] * sum[0]))) * sum[2];
+                        y1 = 0.5f * sum[1] * (1.0f + tanhf(0.7978845608028654f * (sum[1] + 0.044715f * sum[1] * sum[1] * sum[1]))) * sum[3];
+                    } else {
+                        y0 = sum[0] / (1.0f + expf(-sum[0])) * sum[2];
+                        y1 = sum[1] / (1.0f + expf(-sum[1])) * sum[3];
+                    }
                     if (t0 < M) o[(size_t)t0 * ldc + col] = from_f<TC>(y0);
                     if (t0 + 1 < M) o[(size_t)(t0 + 1) * ldc + col] = from_f<TC>(y1);
                 }
@@ -318,7 +325,7 @@ static int gemv_stream_dispatch(const void* a, long lda, const void* W, long ldw
     if (M > 16 || K <= 0 || (K & 63) || splits < 1 || splits > 64) return AIEN_E_SHAPE;
     if (splits > 1 && (epilogue != 0 || c_dt != AIEN_DT_F32)) return AIEN_E_SHAPE;
     if ((lda & 7) || (ldw & 7) || ((uintptr_t)a & 15) || ((uintptr_t)W & 15)) return AIEN_E_ALIGN;
-    if (epilogue == 1 && (N & 15)) return AIEN_E_SHAPE;
+    if ((epilogue == 1 || epilogue == 6) && (N & 15)) return AIEN_E_SHAPE;
     if (epilogue == 2 && (splits != 1 || !fz.resid || !fz.norm_w || !fz.xw || !fz.ssq_out || fz.ssq_in)) return AIEN_E_SHAPE;
     if (fz.ssq_in && (splits != 1 || fz.ssq_parts <= 0)) return AIEN_E_SHAPE;
     CUtensorMap mw, ma;
@@ -341,6 +348,7 @@ static int gemv_stream_dispatch(const void* a, long lda, const void* W, long ldw
     if (epilogue == 3 && c_dt == AIEN_DT_BF16 && splits == 1) { if (M <= 8) GS_CASE(1, 3, __nv_bfloat16); else GS_CASE(2, 3, __nv_bfloat16); }
     if (epilogue == 4 && c_dt == AIEN_DT_BF16 && splits == 1) { if (M <= 8) GS_CASE(1, 4, __nv_bfloat16); else GS_CASE(2, 4, __nv_bfloat16); }
     if (epilogue == 5 && c_dt == AIEN_DT_BF16 && splits == 1) { if (M <= 8) GS_CASE(1, 5, __nv_bfloat16); else GS_CASE(2, 5, __nv_bfloat16); }
+    if (epilogue == 6 && c_dt == AIEN_DT_BF16 && splits == 1) { if (M <= 8) GS_CASE(1, 6, __nv_bfloat16); else GS_CASE(2, 6, __nv_bfloat16); }
 #undef GS_CASE
     return AIEN_E_SHAPE;
 }
@@ -350,7 +358,7 @@ static int gemv_stream_dispatch(const void* a, long lda, const void* W, long ldw
 // partial products are written as zeros.
 AIEN_API int aien_gemv_stream_bf16(const void* a, long lda, const void* W, long ldw, void* out, int c_dt, long ldc,
                                    int M, int N, int K, int epilogue, int splits, size_t part_stride, cudaStream_t stream) {
-    if (epilogue != 0 && epilogue != 1 && epilogue != 3 && epilogue != 4 && epilogue != 5) return AIEN_E_SHAPE;    // 3 / 4: gelu (erf / tanh form), 5: relu squared; bfloat16 out
+    if (epilogue != 0 && epilogue != 1 && (epilogue < 3 || epilogue > 6)) return AIEN_E_SHAPE;    // 6: gelu (tanh form) of gate, times up; 3 / 4: gelu (erf / tanh form), 5: relu squared; bfloat16 out
     GsFuse none = {};
     return gemv_stream_dispatch(a, lda, W, ldw, out, c_dt, ldc, M, N, K, epilogue, splits, part_stride, none, stream);
 }

@@ -87,13 +87,14 @@ __global__ void rotate_pairs_rows_kernel(const TQ* __restrict__ q, long ldq, lon
 // C[t, h, n] = sum_k A[t, h, k] * W[h, n, k]: every head multiplies its own slice of the rows by its own
 // matrix (stored [out, in] like every weight).  Float32 sums on the CUDA cores, k in order, so a row's
 // result depends on that row alone.  a_head / c_head: distance between heads inside a row.  gate (or null): the result
-// of head h is multiplied by sigmoid(gate[t, h]) (rows ldg apart).
+// of head h is multiplied by sigmoid(gate[t, h]) (rows ldg apart), or with gate_n > 0 element n of it by sigmoid(gate[t, h *
+// gate_n + n]).
 constexpr int HP_BM = 64, HP_BN = 64, HP_BK = 16;
 
 template <typename TA, typename TW, typename TC>
 __global__ void __launch_bounds__(256)
 head_project_kernel(const TA* __restrict__ A, long lda, long a_head, const TW* __restrict__ W, long ldw, long w_head,
-                    TC* __restrict__ C, long ldc, long c_head, int M, int N, int K, const float* __restrict__ gate, long ldg) {
+                    TC* __restrict__ C, long ldc, long c_head, int M, int N, int K, const void* __restrict__ gate, int gdt, long ldg, int gate_n) {
     __shared__ float As[HP_BK][HP_BM + 4];
     __shared__ float Ws[HP_BK][HP_BN + 4];
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
@@ -134,11 +135,13 @@ head_project_kernel(const TA* __restrict__ A, long lda, long a_head, const TW* _
     for (int i = 0; i < 4; ++i) {
         const int gm = m0 + ty * 4 + i;
         if (gm >= M) continue;
-        const float gs = gate != nullptr ? 1.0f / (1.0f + expf(-gate[(size_t)gm * ldg + h])) : 1.0f;
+        const float gs = (gate != nullptr && gate_n == 0) ? 1.0f / (1.0f + expf(-load_dyn(gate, gdt, (size_t)gm * ldg + h))) : 1.0f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int gn = n0 + tx * 4 + j;
-            if (gn < N) C[(size_t)gm * ldc + gn] = from_f<TC>(acc[i][j] * gs);
+            if (gn >= N) continue;
+            const float ge = gate_n > 0 ? 1.0f / (1.0f + expf(-load_dyn(gate, gdt, (size_t)gm * ldg + (size_t)h * gate_n + gn))) : gs;
+            C[(size_t)gm * ldc + gn] = from_f<TC>(acc[i][j] * ge);
         }
     }
 }
@@ -332,15 +335,15 @@ AIEN_API int aien_rotate_pairs_rows(const void* q, int q_dt, long ldq, long q_he
 }
 
 AIEN_API int aien_head_project(const void* A, int a_dt, long lda, long a_head, const void* W, int w_dt, long ldw, long w_head,
-                               void* C, int c_dt, long ldc, long c_head, int M, int N, int K, int heads, const float* gate, long ldg,
-                               cudaStream_t stream) {
+                               void* C, int c_dt, long ldc, long c_head, int M, int N, int K, int heads, const void* gate, int gate_dt, long ldg,
+                               int gate_n, cudaStream_t stream) {
     if (M <= 0 || N <= 0 || heads <= 0) return 0;
-    if (K <= 0 || heads > 65535) return AIEN_E_SHAPE;
+    if (K <= 0 || heads > 65535 || gate_n < 0 || (gate_n > 0 && (gate == nullptr || gate_n != N))) return AIEN_E_SHAPE;
     dim3 grid((N + HP_BN - 1) / HP_BN, (M + HP_BM - 1) / HP_BM, heads);
     if (grid.y > 65535) return AIEN_E_SHAPE;
     AIEN_DISPATCH_DTYPE(a_dt, TA, AIEN_DISPATCH_DTYPE(w_dt, TW, AIEN_DISPATCH_DTYPE(c_dt, TC,
         (head_project_kernel<TA, TW, TC><<<grid, 256, 0, stream>>>((const TA*)A, lda, a_head, (const TW*)W, ldw, w_head, (TC*)C, ldc,
-                                                                  c_head, M, N, K, gate, ldg)))));
+                                                                  c_head, M, N, K, gate, gate_dt, ldg, gate_n)))));
     return launch_status();
 }
 

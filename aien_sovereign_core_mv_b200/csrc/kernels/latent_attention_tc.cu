@@ -347,7 +347,7 @@ constexpr int HT_BM = 64, HT_BN = 64, HT_BK = 64, HT_STR = HT_BK + 8;
 template <typename TC>
 __global__ void __launch_bounds__(128)
 head_project_tc_kernel(const __nv_bfloat16* __restrict__ A, long lda, long a_head, const __nv_bfloat16* __restrict__ W, long w_head,
-                       TC* __restrict__ C, long ldc, long c_head, int M, int N, int K, const float* __restrict__ gate, long ldg) {
+                       TC* __restrict__ C, long ldc, long c_head, int M, int N, int K, const void* __restrict__ gate, int gdt, long ldg, int gate_n) {
     __shared__ __align__(16) __nv_bfloat16 As[HT_BM * HT_STR];
     __shared__ __align__(16) __nv_bfloat16 Ws[HT_BN * HT_STR];
     const uint32_t As_u = (uint32_t)__cvta_generic_to_shared(As), Ws_u = (uint32_t)__cvta_generic_to_shared(Ws);
@@ -400,7 +400,7 @@ head_project_tc_kernel(const __nv_bfloat16* __restrict__ A, long lda, long a_hea
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
             const int m = m0 + mh * 32 + mt * 16 + g + r * 8;
-            gs[mt][r] = (gate != nullptr && m < M) ? 1.0f / (1.0f + expf(-gate[(size_t)m * ldg + h])) : 1.0f;
+            gs[mt][r] = (gate != nullptr && gate_n == 0 && m < M) ? 1.0f / (1.0f + expf(-load_dyn(gate, gdt, (size_t)m * ldg + h))) : 1.0f;
         }
 #pragma unroll
     for (int mt = 0; mt < 2; ++mt)
@@ -409,7 +409,9 @@ head_project_tc_kernel(const __nv_bfloat16* __restrict__ A, long lda, long a_hea
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int m = m0 + mh * 32 + mt * 16 + g + (e >> 1) * 8, n = n0 + nh * 32 + j * 8 + 2 * c + (e & 1);
-                if (m < M && n < N) C[(size_t)m * ldc + n] = from_f<TC>(acc[mt][j][e] * gs[mt][e >> 1]);
+                if (m >= M || n >= N) continue;
+                const float ge = gate_n > 0 ? __fdividef(1.0f, 1.0f + __expf(-load_dyn(gate, gdt, (size_t)m * ldg + (size_t)h * gate_n + n))) : gs[mt][e >> 1];
+                C[(size_t)m * ldc + n] = from_f<TC>(acc[mt][j][e] * ge);
             }
 }
 
@@ -454,13 +456,13 @@ AIEN_API int aien_latent_attention_tc(const void* q, const void* cache, const in
 // A bfloat16 [M, lda] (head h at column h * a_head), W bfloat16 [heads, N, K], C [M, ldc] (head h at column h * c_head).
 // K, lda and a_head multiples of 8, A and W 16-byte aligned.
 AIEN_API int aien_head_project_tc(const void* A, long lda, long a_head, const void* W, void* C, int c_dt, long ldc, long c_head,
-                                  int M, int N, int K, int heads, const float* gate, long ldg, cudaStream_t stream) {
+                                  int M, int N, int K, int heads, const void* gate, int gate_dt, long ldg, int gate_n, cudaStream_t stream) {
     if (M <= 0 || N <= 0 || heads <= 0) return 0;
-    if (K <= 0 || heads > 65535) return AIEN_E_SHAPE;
+    if (K <= 0 || heads > 65535 || gate_n < 0 || (gate_n > 0 && (gate == nullptr || gate_n != N))) return AIEN_E_SHAPE;
     if ((K & 7) || (lda & 7) || (a_head & 7) || ((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return AIEN_E_ALIGN;
     dim3 grid((N + HT_BN - 1) / HT_BN, (M + HT_BM - 1) / HT_BM, heads);
     if (grid.y > 65535) return AIEN_E_SHAPE;
     AIEN_DISPATCH_DTYPE(c_dt, TC, (head_project_tc_kernel<TC><<<grid, 128, 0, stream>>>((const __nv_bfloat16*)A, lda, a_head, (const __nv_bfloat16*)W,
-                                                                                     (long)N * K, (TC*)C, ldc, c_head, M, N, K, gate, ldg)));
+                                                                                     (long)N * K, (TC*)C, ldc, c_head, M, N, K, gate, gate_dt, ldg, gate_n)));
     return launch_status();
 }

@@ -149,9 +149,9 @@ __global__ void gelu_times_table_kernel(const TZ* __restrict__ z, long ldz, cons
     }
 }
 
-__global__ void softcap_kernel(float* __restrict__ v, size_t n, float cap) {
+__global__ void softcap_kernel(float* __restrict__ v, size_t n, float cap, float mult) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) v[i] = cap * tanhf(v[i] / cap);
+    if (i < n) v[i] = cap > 0.f ? cap * tanhf(v[i] * mult / cap) : v[i] * mult;
 }
 
 }  // namespace aien
@@ -214,9 +214,10 @@ AIEN_API int aien_gelu_times_table(const void* z, int z_dt, long ldz, const void
     return launch_status();
 }
 
-AIEN_API int aien_softcap(float* v, size_t n, float cap, cudaStream_t stream) {
+// v = cap * tanh(v * mult / cap) in place; cap 0: v * mult.
+AIEN_API int aien_softcap(float* v, size_t n, float cap, float mult, cudaStream_t stream) {
     if (n == 0) return 0;
-    if (!(cap > 0.f)) return AIEN_E_SHAPE;
-    softcap_kernel<<<(unsigned)((n + 255) / 256), 256, 0, stream>>>(v, n, cap);
+    if (!(cap >= 0.f)) return AIEN_E_SHAPE;
+    softcap_kernel<<<(unsigned)((n + 255) / 256), 256, 0, stream>>>(v, n, cap, mult);
     return launch_status();
 }

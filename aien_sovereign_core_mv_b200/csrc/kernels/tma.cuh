@@ -126,4 +126,29 @@ inline bool make_map_chunked(CUtensorMap* map, const void* ptr, uint64_t rows, u
     return true;
 }
 
+// A bfloat16 matrix [rows, heads * size] (leading dimension ld) seen as [rows][heads][size]: boxes of box_rows rows x one
+// head x 64 of its columns, laid out and swizzled like make_map's; columns beyond the head's size are filled with zeros,
+// so that tiles are padded to whole 64-column chunks.  Needs size % 8 == 0.
+inline bool make_map_heads(CUtensorMap* map, const void* ptr, uint64_t rows, uint64_t heads, uint64_t size, uint64_t ld, uint32_t box_rows) {
+    static std::map<std::tuple<const void*, uint64_t, uint64_t, uint64_t, uint64_t, uint32_t>, CUtensorMap> cache;
+    static std::mutex mu;
+    std::lock_guard<std::mutex> lock(mu);
+    auto key = std::make_tuple(ptr, rows, heads, size, ld, box_rows);
+    auto it = cache.find(key);
+    if (it != cache.end()) { *map = it->second; return true; }
+    EncodeTiledFn fn = encode_fn();
+    if (!fn || (size & 7) || (ld & 7)) return false;
+    cuuint64_t dims[3] = {size, heads, rows};
+    cuuint64_t strides[2] = {size * 2, ld * 2};
+    cuuint32_t box[3] = {64, 1, box_rows};
+    cuuint32_t estr[3] = {1, 1, 1};
+    if (fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, estr,
+           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
+        return false;
+    if (cache.size() > 4096) cache.clear();
+    cache[key] = *map;
+    return true;
+}
+
 }  // namespace aien

@@ -110,16 +110,17 @@ def _declare(l: ctypes.CDLL) -> None:
     sigs = {
         "aien_embed_gather": [P, I, P, P, I, I, I, P],
         "aien_add_rmsnorm": [P, P, I, I, c_size_t, P, I, F, P, I, I, I, P],
+        "aien_add_layernorm": [P, P, I, I, c_size_t, P, I, F, P, I, I, I, P],
         "aien_gather_add_rows": [P, P, I, I, c_size_t, P, P, I, I, P],
-        "aien_swiglu": [P, P, I, I, I, I, P],
+        "aien_swiglu": [P, P, I, I, I, I, I, P],
         "aien_add_residual": [P, P, I, I, c_size_t, I, I, P],
-        "aien_rope_table": [P, P, P, P, I, I, P],
+        "aien_rope_table": [P, P, P, P, I, I, c_double, P],
         "aien_qk_norm_rope_kv_write": [P, L, I, P, L, P, L, I, I, I, c_size_t, P, L, I, P, P, I, F, P, P, I, P, P, P, I, I, I, P],
         "aien_convert": [P, I, P, I, c_size_t, P],
         "aien_gemm_simple": [P, I, L, P, I, L, P, I, L, I, I, I, P],
-        "aien_paged_attention_generic": [P, L, P, P, P, I, P, P, P, L, I, I, I, I, I, F, I, I, I, I, P, I, P, P, P, P, L, F, P],
+        "aien_paged_attention_generic": [P, L, P, P, P, I, P, P, P, L, I, I, I, I, I, F, I, I, I, I, P, I, P, P, P, P, L, F, I, I, P],
         "aien_branch_norm_add": [P, P, I, I, c_size_t, P, I, I, c_size_t, P, I, F, P, I, I, I, P],
-        "aien_stream_norm_inplace": [P, P, I, F, P, I, I, I, P],
+        "aien_stream_norm_inplace": [P, P, I, F, P, I, I, I, I, P],
         "aien_qk_rope_pairs_unit_kv_write": [P, L, I, P, L, P, L, I, I, I, c_size_t, P, L, I, I, I, F, P, P, I, P, P, P, I, I, I, P],
         "aien_moe_route": [P, I, I, I, I, I, I, P, P, P, P],
         "aien_moe_expert_up": [P, I, L, P, I, P, P, P, I, I, I, I, I, I, I, I, P],
@@ -167,14 +168,14 @@ def _declare(l: ctypes.CDLL) -> None:
         "aien_latent_prepare": [P, I, L, I, P, P, I, F, P, I, L, I, I, I, I, P, P, P, P, I, I, P],
         "aien_rotate_pairs_rows": [P, I, L, L, P, I, L, L, I, I, I, I, P, P, P],
         "aien_latent_attention_tc": [P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, P, I, P, P, I, P],
-        "aien_head_project_tc": [P, L, L, P, P, I, L, L, I, I, I, I, P, L, P],
+        "aien_head_project_tc": [P, L, L, P, P, I, L, L, I, I, I, I, P, I, L, I, P],
         "aien_latent_attention_tc_supports": [I, I],
-        "aien_head_project": [P, I, L, L, P, I, L, L, P, I, L, L, I, I, I, I, P, L, P],
+        "aien_head_project": [P, I, L, L, P, I, L, L, P, I, L, L, I, I, I, I, P, I, L, I, P],
         "aien_latent_attention": [P, L, P, I, P, I, P, P, P, P, I, L, I, I, I, I, I, I, F, P, P],
         "aien_post_norm_add": [P, P, I, I, c_size_t, P, I, F, F, P, I, F, P, I, I, I, P],
         "aien_embed_gather_scaled": [P, I, P, P, I, I, I, F, P],
         "aien_gelu_times_table": [P, I, L, P, I, L, I, P, I, P, I, L, I, I, P],
-        "aien_softcap": [P, c_size_t, F, P],
+        "aien_softcap": [P, c_size_t, F, F, P],
         "aien_replicate_streams": [P, c_size_t, I, P],
         "aien_hc_norm": [P, I, P, I, I, c_size_t, P, P, P, I, F, P, I, I, I, P, I, P, P, P, P],
         "aien_token_shift": [P, P, I, P, P, P, P, P, P, I, I, I, P],
@@ -205,7 +206,11 @@ def _declare(l: ctypes.CDLL) -> None:
         "aien_matrix_memory_chunks_supports": [I, I],
         "aien_matrix_memory_chunked": [P, L, I, I, I, I, F, P, P, c_size_t, P, P, P, P, I, F, F, P, L, P, I, I, I, I, I, P],
         "aien_matrix_memory_token": [P, I, L, I, I, I, I, F, P, L, I, I, P, P, F, P, c_size_t, P, P, P, P, I, F, F, P, I, L, I, I, I, I, P],
-        "aien_rope_halves_value_write": [P, L, I, I, I, I, I, I, I, P, P, I, P, P, I, L, P, P, I, I, P],
+        "aien_rope_halves_value_write": [P, I, L, I, c_size_t, P, I, I, I, I, I, I, I, I, P, P, I, P, P, I, L, P, P, I, I, P],
+        "aien_map_difference_norm": [P, L, P, I, L, I, I, I, I, F, F, F, P],
+        "aien_paged_attention_decode_values": [P, L, P, P, P, I, P, P, P, P, L, P, P, P, I, I, I, I, I, F, I, I, I, F, I, I, I, I, P],
+        "aien_paged_attention_prefill_tc_values": [P, L, I, P, P, I, P, I, P, P, P, P, I, P, L, I, I, I, I, I, F, P, L, I, I, I, P, P, P, P, L, F, I, I, I, P],
+        "aien_paged_attention_prefill_tc_values_supports": [I, I, I],
     }
     for name, args in sigs.items():
         fn = getattr(l, name)
@@ -321,6 +326,17 @@ def add_rmsnorm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Te
                                   _p(weight), dt(weight), float(eps), _p(out), dt(out), T, H, _stream()), "add_rmsnorm")
 
 
+def add_layernorm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float, out: torch.Tensor) -> None:
+    """x += delta (when given); out = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight.  x float32 [T,H] updated in place."""
+    _dev(x, delta, weight, out)
+    T, H = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and out.shape == x.shape
+    assert weight.numel() == H and weight.is_contiguous()
+    nparts, stride = _parts_of(delta, x.shape)
+    _check(lib().aien_add_layernorm(_p(x), _p(delta), dt(delta) if delta is not None else F32, nparts, stride,
+                                    _p(weight), dt(weight), float(eps), _p(out), dt(out), T, H, _stream()), "add_layernorm")
+
+
 def gather_add_rows(x: torch.Tensor, delta: Optional[torch.Tensor], rows: torch.Tensor, out: torch.Tensor) -> None:
     """out[r] = x[rows[r]] + delta[rows[r]] in float32."""
     _dev(x, delta, rows, out)
@@ -341,22 +357,25 @@ def add_residual(x: torch.Tensor, delta: torch.Tensor) -> None:
     _check(lib().aien_add_residual(_p(x), _p(delta), dt(delta), nparts, stride, T, H, _stream()), "add_residual")
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, group: int = 0) -> None:
-    """out = silu(gate) * up for gate_up = [T, 2I]: gate columns first (group 0), or gate and up
-    columns interleaved in runs of ``group``."""
+GATED_ACTS = {"silu": 1, "gelu_tanh": 6}        # act(gate) * up: the products' epilogue that computes it
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, group: int = 0, act: str = "silu") -> None:
+    """out = act(gate) * up for gate_up = [T, 2I]: gate columns first (group 0), or gate and up
+    columns interleaved in runs of ``group``.  ``act``: a key of GATED_ACTS."""
     _dev(gate_up, out)
     T, I = out.shape
     assert gate_up.shape == (T, 2 * I) and gate_up.is_contiguous() and out.is_contiguous() and gate_up.dtype == out.dtype
-    _check(lib().aien_swiglu(_p(gate_up), _p(out), dt(out), T, I, int(group), _stream()), "swiglu")
+    _check(lib().aien_swiglu(_p(gate_up), _p(out), dt(out), T, I, int(group), 1 if act == "gelu_tanh" else 0, _stream()), "swiglu")
 
 
-def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> None:
-    """cos/sin [T, half] float32 of positions[t] * inv_freq[i], the angle taken in float64."""
+def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, mult: float = 1.0) -> None:
+    """cos/sin [T, half] float32 of positions[t] * inv_freq[i], the angle taken in float64, both times ``mult``."""
     _dev(positions, inv_freq, cos, sin)
     T, half = cos.shape
     assert positions.dtype == torch.int32 and inv_freq.dtype == torch.float64 and inv_freq.numel() == half
     assert cos.dtype == torch.float32 and sin.dtype == torch.float32 and cos.is_contiguous() and sin.is_contiguous()
-    _check(lib().aien_rope_table(_p(positions), _p(inv_freq), _p(cos), _p(sin), T, half, _stream()), "rope_table")
+    _check(lib().aien_rope_table(_p(positions), _p(inv_freq), _p(cos), _p(sin), T, half, float(mult), _stream()), "rope_table")
 
 
 def qk_norm_rope_kv_write(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tensor], head_dim: int,
@@ -431,15 +450,15 @@ def branch_norm_add(x: torch.Tensor, a: torch.Tensor, weight: torch.Tensor, eps:
                                       _p(h), dt(h) if h is not None else F32, T, H, _stream()), "branch_norm_add")
 
 
-def stream_norm_inplace(x: torch.Tensor, weight: torch.Tensor, eps: float, h: Optional[torch.Tensor] = None) -> None:
-    """x = x / sqrt(mean(x^2) + eps) * weight in place (float32 rows); ``h`` as in branch_norm_add."""
+def stream_norm_inplace(x: torch.Tensor, weight: torch.Tensor, eps: float, h: Optional[torch.Tensor] = None, center: bool = False) -> None:
+    """x = x / sqrt(mean(x^2) + eps) * weight in place (float32 rows), with ``center`` the layer norm; ``h`` as in branch_norm_add."""
     _dev(x, weight, h)
     T, H = x.shape
     assert x.dtype == torch.float32 and x.is_contiguous() and weight.numel() == H and weight.is_contiguous()
     if h is not None:
         assert h.is_contiguous() and tuple(h.shape) == (T, H)
     _check(lib().aien_stream_norm_inplace(_p(x), _p(weight), dt(weight), float(eps), _p(h), dt(h) if h is not None else F32,
-                                          T, H, _stream()), "stream_norm_inplace")
+                                          T, H, 1 if center else 0, _stream()), "stream_norm_inplace")
 
 
 def qk_rope_pairs_unit_kv_write(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tensor], head_dim: int,
@@ -641,7 +660,7 @@ def paged_attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: tor
                             scale: float, chunk: int = 0, sinks: Optional[torch.Tensor] = None, value_dim: int = 0,
                             token_list: Optional[torch.Tensor] = None, num_tokens: Optional[int] = None,
                             head_scale: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
-                            gate: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
+                            gate: Optional[torch.Tensor] = None, softcap: float = 0.0, v_share: int = 1) -> None:
     """Causal attention of T query tokens over their requests' pages.  q [T, nq*hd] (row stride
     free), caches [slots, nkv, hd], block_table int32 [S, max_blocks], out [T, nq*hd].
     ``chunk`` > 0: a token sees only the keys of its own chunk of that many positions.  ``sinks``
@@ -650,7 +669,8 @@ def paged_attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: tor
     ``token_list`` (int32) with ``num_tokens``: only these tokens of the step are served.  Per head (float32 [nq]):
     ``head_scale`` multiplies the scaled score, ``slopes`` takes slope * (query position - key position) off it;
     ``gate`` (float32 [T, >= nq], row stride free): the head's output is multiplied by sigmoid(gate[t, h]).
-    ``softcap`` c > 0: the scaled score s becomes c * tanh(s / c)."""
+    ``softcap`` c > 0: the scaled score s becomes c * tanh(s / c).  ``v_share``: so many neighbouring key heads share one
+    value head (v_cache [slots, nkv / v_share, value_dim])."""
     _dev(q, k_cache, v_cache, block_table, seq_of_token, positions, out, sinks, token_list, head_scale, slopes, gate)
     for v in (head_scale, slopes):
         assert v is None or (v.dtype == torch.float32 and v.is_contiguous() and v.numel() == num_q_heads)
@@ -658,7 +678,7 @@ def paged_attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: tor
     if sinks is not None:
         assert sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == num_q_heads
     T = q.shape[0] if token_list is None else int(num_tokens)
-    assert q.stride(1) == 1 and out.stride(1) == 1 and q.dtype == out.dtype
+    assert q.stride(1) == 1 and out.stride(1) == 1
     assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == v_cache.dtype
     assert block_table.dtype == torch.int32 and seq_of_token.dtype == torch.int32 and positions.dtype == torch.int32
     assert token_list is None or (token_list.dtype == torch.int32 and token_list.numel() >= T)
@@ -666,7 +686,7 @@ def paged_attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: tor
         _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(block_table), max_blocks, _p(seq_of_token), _p(positions),
         _p(out), out.stride(0), num_q_heads, num_kv_heads, head_dim, page_size, window, float(scale),
         dt(q), dt(k_cache), T, int(chunk), _p(sinks), int(value_dim), _p(token_list), _p(head_scale), _p(slopes), _p(gate),
-        gate.stride(0) if gate is not None else 0, float(softcap or 0.0), _stream()), "paged_attention_generic")
+        gate.stride(0) if gate is not None else 0, float(softcap or 0.0), int(v_share), dt(out), _stream()), "paged_attention_generic")
 
 
 # ---------------------------------------------------------------------------- sampling
@@ -727,6 +747,7 @@ def gemv(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = 0)
     """out = a . w^T for up to 16 rows of a (bfloat16, float32 accumulation).  ``epilogue=1``:
     w holds gate|up rows interleaved in groups of 8 and out = silu(gate)*up with N/2 columns.
     ``epilogue=3`` / ``4`` / ``5`` (the streamed kernel, bfloat16 out): the gelu in its erf / tanh form, the square of relu.
+    ``epilogue=6`` (bfloat16 out): as 1 with the tanh form of the gelu in silu's place.
     ``out`` of shape [P, M, N] float32 receives P partial products over P ranges of K."""
     _dev(a, w, out)
     M, K_ = a.shape
@@ -736,8 +757,8 @@ def gemv(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = 0)
         assert epilogue == 0 and out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape[1:]) == (M, N)
         splits, part_stride = out.shape[0], M * N
     else:
-        assert w.shape[1] == K_ and out.shape == (M, N // 2 if epilogue == 1 else N)
-    assert epilogue in (0, 1) or gemv_takes_activation(K_)
+        assert w.shape[1] == K_ and out.shape == (M, N // 2 if epilogue in (1, 6) else N)
+    assert epilogue in (0, 1, 6) or gemv_takes_activation(K_)
     fn = lib().aien_gemv_stream_bf16 if (GEMV_IMPL == "stream" and K_ % 64 == 0) else lib().aien_gemv_bf16
     _check(fn(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), dt(out), out.stride(-2), M, N, K_,
               epilogue, splits, part_stride, _stream()), "gemv_bf16")
@@ -764,7 +785,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int =
     """out = a . w^T on the tcgen05 tensor cores (bfloat16 operands, float32 accumulation in
     tensor memory).  ``epilogue=1``: w holds gate|up rows interleaved in runs of 8 and
     out = silu(gate)*up with N/2 columns.  ``epilogue=2`` / ``3`` / ``4`` (bfloat16 out): the gelu in its erf / tanh
-    form, the square of relu."""
+    form, the square of relu.  ``epilogue=6`` (bfloat16 out): as 1 with the tanh form of the gelu in silu's place."""
     _dev(a, w, out)
     M, K_ = a.shape
     N = w.shape[0]
@@ -774,7 +795,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int =
         assert out.shape[0] == gemm_tc_ranges(K_, out.shape[0])
         splits, part_stride = out.shape[0], M * N
     else:
-        assert w.shape[1] == K_ and out.shape == (M, N // 2 if epilogue == 1 else N)
+        assert w.shape[1] == K_ and out.shape == (M, N // 2 if epilogue in (1, 6) else N)
     _check(lib().aien_gemm_tc(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), dt(out), out.stride(-2), M, N, K_,
                               epilogue, splits, part_stride, _stream()), "gemm_tc")
 
@@ -1100,15 +1121,17 @@ def decode_splits(max_ctx: int, chunk: int) -> int:
     return min(splits, (chunk + DECODE_CHUNK - 1) // DECODE_CHUNK + 1) if chunk > 0 else splits
 
 
-def decode_masked_takes(num_q_heads: int, num_kv_heads: int, head_dim: int, splits: int) -> bool:
+def decode_masked_takes(num_q_heads: int, num_kv_heads: int, head_dim: int, splits: int, value_dim: int = 0) -> bool:
     """Whether the split-key kernel's shared memory (a block of keys and values, scores, and the merge's
     scratch, which grows with the number of blocks) stays within what a CTA can have; else the plain kernel runs."""
     G = num_q_heads // num_kv_heads
     nh = 8 * ((G + 7) // 8)
     loop = (DECODE_CHUNK * nh + 2 * nh) * 4 + nh * DECODE_CHUNK * 2
     r4 = lambda n: (n + 3) & ~3
-    merge = (r4(G) + r4(splits * G) + max(r4(splits * G), 8 * head_dim)) * 4
-    kv = DECODE_CHUNK * (head_dim * 2 + 16) * 2
+    value_dim = value_dim or head_dim
+    merge = (r4(G) + r4(splits * G) + max(r4(splits * G), 8 * value_dim)) * 4
+    pieces = head_dim // 8
+    kv = DECODE_CHUNK * (max(head_dim * 2 + 16, (pieces + (4 - pieces % 8) % 8) * 16 if pieces % 8 else head_dim * 2) + value_dim * 2 + 16)
     return ((max(loop, merge) + 127) & ~127) + kv <= 200 * 1024 - 1024
 
 
@@ -1303,11 +1326,11 @@ def gelu_times_table(z: torch.Tensor, table: torch.Tensor, col0: int, ids: torch
                                        table.shape[0], _p(out), dt(out), out.stride(0), T, n, _stream()), "gelu_times_table")
 
 
-def softcap(v: torch.Tensor, cap: float) -> None:
-    """v = cap * tanh(v / cap) in place (float32)."""
+def softcap(v: torch.Tensor, cap: float, mult: float = 1.0) -> None:
+    """v = cap * tanh(v * mult / cap) in place (float32); cap 0: v = v * mult."""
     _dev(v)
     assert v.dtype == torch.float32 and v.is_contiguous()
-    _check(lib().aien_softcap(_p(v), v.numel(), float(cap), _stream()), "softcap")
+    _check(lib().aien_softcap(_p(v), v.numel(), float(cap), float(mult), _stream()), "softcap")
 
 
 # ---------------------------------------------------------------------------- mixers with a state of fixed size
@@ -1431,7 +1454,8 @@ def rotate_pairs_rows(q: torch.Tensor, q_head: int, col0: int, out: torch.Tensor
 def head_project(a: torch.Tensor, a_head: int, a_col0: int, w: torch.Tensor, out: torch.Tensor, o_head: int, o_col0: int,
                  gate: Optional[torch.Tensor] = None) -> None:
     """out[t, h*o_head + o_col0 + n] = sum_k a[t, h*a_head + a_col0 + k] * w[h, n, k]: one product per head, w [heads, N, K].
-    ``gate`` float32 [T, heads] (row stride free): the result of head h is multiplied by sigmoid(gate[t, h]).
+    ``gate`` (row stride free): [T, heads], the result of head h is multiplied by sigmoid(gate[t, h]); or [T, heads*N],
+    element n of head h by sigmoid(gate[t, h*N + n]).
     bfloat16 operands whose rows are whole aligned 16-byte pieces run on the tensor cores, everything else on the CUDA cores;
     both sum in float32."""
     _dev(a, w, out)
@@ -1439,17 +1463,18 @@ def head_project(a: torch.Tensor, a_head: int, a_col0: int, w: torch.Tensor, out
     M = a.shape[0]
     assert a.stride(1) == 1 and out.stride(1) == 1 and w.is_contiguous() and out.shape[0] == M
     assert (heads - 1) * a_head + a_col0 + K_ <= a.shape[1] and (heads - 1) * o_head + o_col0 + N <= out.shape[1]
-    assert gate is None or (gate.dtype == torch.float32 and tuple(gate.shape) == (M, heads) and gate.stride(1) == 1)
+    assert gate is None or (tuple(gate.shape) in ((M, heads), (M, heads * N)) and gate.stride(1) == 1)
     _dev(gate)
-    gp, ldg = _p(gate), gate.stride(0) if gate is not None else 0
+    gate_n = N if gate is not None and gate.shape[1] == heads * N and N > 1 else 0
+    gp, gdt, ldg = _p(gate), dt(gate) if gate is not None else F32, gate.stride(0) if gate is not None else 0
     av, ov = a[:, a_col0:], out[:, o_col0:]
     if (_LATENT_IMPL != "plain" and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and K_ % 8 == 0 and a.stride(0) % 8 == 0
             and a_head % 8 == 0 and av.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
         _check(lib().aien_head_project_tc(_p(av), a.stride(0), int(a_head), _p(w), _p(ov), dt(out), out.stride(0), int(o_head), M, N, K_,
-                                          heads, gp, ldg, _stream()), "head_project_tc")
+                                          heads, gp, gdt, ldg, gate_n, _stream()), "head_project_tc")
         return
     _check(lib().aien_head_project(_p(av), dt(a), a.stride(0), int(a_head), _p(w), dt(w), K_, N * K_, _p(ov), dt(out), out.stride(0),
-                                   int(o_head), M, N, K_, heads, gp, ldg, _stream()), "head_project")
+                                   int(o_head), M, N, K_, heads, gp, gdt, ldg, gate_n, _stream()), "head_project")
 
 
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, max_blocks: int, seq_of_token: torch.Tensor,
@@ -1906,52 +1931,84 @@ def scale_rows(o: torch.Tensor, mult: float, out: torch.Tensor) -> None:
     sigmoid_gate(o, None, mult, out)
 
 
-# ---------------------------------------------------------------------------- attention with a capped score
-def capped_attention_workspace_bytes(lim, num_heads: int, value_dim: int) -> int:
+# ---------------------------------------------------------------------------- attention with values of their own size
+def _tile_cols(n: int) -> int:
+    """Columns of a key or value tile of the tcgen05 kernel for a head of n numbers."""
+    return 64 if n <= 64 else 128
+
+
+def _span_splits(max_ctx: int, window: int, chunk: int) -> int:
+    """Key blocks of 128 that the split-key kernel runs per token: those a chunk or a window can touch, or all."""
+    sizes = [n for n in (window, chunk) if n > 0]
+    return decode_splits(max_ctx, min(sizes) if sizes else 0)
+
+
+def capped_attention_workspace_bytes(lim, num_heads: int, value_dim: int, window: int = 0, chunk: int = 0) -> int:
     """Scratch of :func:`capped_attention` for the largest step: the partial results of the split-key kernel and of the
     key ranges of the tcgen05 kernel."""
-    return biased_attention_workspace_bytes(lim, num_heads, value_dim, 0) + attention_workspace_bytes(lim, num_heads, value_dim)
+    n = lim.max_seqs * num_heads * _span_splits(lim.max_context, window, chunk) * (value_dim + 2) * 4 + 8192
+    if not chunk:
+        n += prefill_split_scratch_bytes(PREFILL_SPLIT_MAX_TILES, num_heads, _tile_cols(value_dim), lim.max_context)
+    return n
 
 
 def capped_attention(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, group, out: torch.Tensor, num_q_heads: int,
-                     num_kv_heads: int, head_dim: int, value_dim: int, window: int, scale: float, softcap: float) -> None:
-    """Causal attention of the step's tokens over one cache group with the scaled score s turned into softcap * tanh(s /
-    softcap) (softcap 0: left as it is), an optional window, values of size ``value_dim``.  Picks the kernel for the step:
-    in bfloat16 with values as large as keys, portions of prompts go through the tcgen05 kernel and tokens that come alone
-    through the split-key kernel; all else through the plain one."""
+                     num_kv_heads: int, head_dim: int, value_dim: int, window: int, scale: float, softcap: float = 0.0, chunk: int = 0,
+                     v_share: int = 1) -> None:
+    """Causal attention of the step's tokens over one cache group, values of size ``value_dim``: an optional window
+    (``window`` keys back, the token itself included), an optional chunk mask (a token sees the keys of its own chunk of
+    ``chunk`` positions), optionally the scaled score s turned into softcap * tanh(s / softcap).  ``v_share`` neighbouring
+    key heads share one value head.  ``out`` [T, num_q_heads * value_dim] in the compute dtype or float32.  Picks the kernel
+    for the step: in bfloat16, portions of prompts go through the tcgen05 kernel (head sizes that are multiples of 8 up to
+    128) and tokens that come alone through the split-key kernel (keys in multiples of 8, values of 16, up to 256); all
+    else through the plain one."""
+    num_v_heads = num_kv_heads // v_share
     k2 = k_cache.view(-1, num_kv_heads, head_dim)
-    v2 = v_cache.view(-1, num_kv_heads, value_dim)
-    fast = (_FORCE_ATTN != "generic" and value_dim == head_dim and out.dtype == torch.bfloat16
-            and decode_attention_supports(q, k2, num_q_heads, num_kv_heads, head_dim))
-    splits = max(1, (ctx.max_ctx_len + DECODE_CHUNK - 1) // DECODE_CHUNK)
+    v2 = v_cache.view(-1, num_v_heads, value_dim)
+    fast = (_FORCE_ATTN != "generic" and q.dtype == torch.bfloat16 and k2.dtype == torch.bfloat16 and q.stride(0) % 8 == 0
+            and q.data_ptr() % 16 == 0 and k2.data_ptr() % 16 == 0 and v2.data_ptr() % 16 == 0)
+    splits = _span_splits(ctx.max_ctx_len, window, chunk)
+    splits_ok = (fast and head_dim % 8 == 0 and head_dim <= 256 and value_dim % 16 == 0 and value_dim <= 256
+                 and num_q_heads // num_kv_heads <= 16 and decode_masked_takes(num_q_heads, num_kv_heads, head_dim, splits, value_dim))
 
     def single_tokens(tokens, n):
-        part_out = ctx.workspace.take((n * num_q_heads * splits * head_dim,), torch.float32)
+        global _ticket_counters
+        if _ticket_counters is None:
+            _ticket_counters = torch.zeros(1 << 16, dtype=torch.int32, device=q.device)
+        assert n * num_kv_heads <= _ticket_counters.numel()
+        part_out = ctx.workspace.take((n * num_q_heads * splits * value_dim,), torch.float32)
         part_ml = ctx.workspace.take((n * num_q_heads * splits * 2,), torch.float32)
-        paged_attention_decode(q, k2, v2, group.block_table, group.max_blocks, None if tokens is None else ctx.seq_of_token,
-                               ctx.positions, out, part_out, part_ml, num_q_heads, num_kv_heads, head_dim, group.page_size, window, scale,
-                               splits, token_list=tokens, num_tokens=n, impl="direct", softcap=softcap)
+        _check(lib().aien_paged_attention_decode_values(
+            _p(q), q.stride(0), _p(k2), _p(v2), _p(group.block_table), group.max_blocks, None if tokens is None else _p(ctx.seq_of_token),
+            _p(ctx.positions), _p(tokens), _p(out), out.stride(0), _p(part_out), _p(part_ml), _p(_ticket_counters), num_q_heads,
+            num_kv_heads, head_dim, group.page_size, window, float(scale), splits, n, int(chunk), float(softcap or 0.0), value_dim,
+            int(v_share), 1 if out.dtype == torch.float32 else 0, 1 if window > 0 or chunk > 0 else 0, _stream()),
+            "paged_attention_decode_values")
 
     def plain(tokens=None, n=None):
         paged_attention_generic(q, k2, v2, group.block_table, group.max_blocks, ctx.seq_of_token, ctx.positions, out, num_q_heads,
                                 num_kv_heads, head_dim, group.page_size, window, scale, value_dim=value_dim, softcap=softcap,
-                                token_list=tokens, num_tokens=n)
+                                token_list=tokens, num_tokens=n, chunk=chunk, v_share=v_share)
 
-    splits_ok = fast and decode_masked_takes(num_q_heads, num_kv_heads, head_dim, splits)
+    _dev(q, k_cache, v_cache, group.block_table, ctx.positions, out)
+    assert q.stride(1) == 1 and out.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
     if ctx.decode_only and splits_ok:
         single_tokens(None, q.shape[0])
         return
-    if (not ctx.decode_only and fast and ctx.prefill_tiles is not None and _PREFILL_IMPL == "tc"
-            and prefill_tc_supports(q, out, head_dim, group.page_size)):
+    if (not ctx.decode_only and fast and ctx.prefill_tiles is not None and _PREFILL_IMPL == "tc" and out.stride(0) % 8 == 0
+            and out.data_ptr() % 16 == 0 and lib().aien_paged_attention_prefill_tc_values_supports(head_dim, value_dim, group.page_size)):
         tile_seq, tile_q0, n = ctx.prefill_tiles
         if n > 0:
             scratch = None
-            if n <= PREFILL_SPLIT_MAX_TILES:
-                nbytes = prefill_split_scratch_bytes(n, num_q_heads, head_dim, ctx.max_ctx_len)
+            if n <= PREFILL_SPLIT_MAX_TILES and not chunk:
+                nbytes = prefill_split_scratch_bytes(n, num_q_heads, _tile_cols(value_dim), ctx.max_ctx_len)
                 scratch = ctx.workspace.take((nbytes // 4,), torch.float32) if nbytes else None
-            paged_attention_prefill(q, k2, v2, group.block_table, group.max_blocks, ctx.q_start, ctx.ctx_len, tile_seq, tile_q0, n,
-                                    out, num_q_heads, num_kv_heads, head_dim, group.page_size, window, scale, impl="tc",
-                                    scratch=scratch, max_ctx=ctx.max_ctx_len, softcap=softcap)
+            _check(lib().aien_paged_attention_prefill_tc_values(
+                _p(q), q.stride(0), q.shape[0], _p(k2), _p(v2), k2.shape[0], _p(group.block_table), group.max_blocks, _p(ctx.q_start),
+                _p(ctx.ctx_len), _p(tile_seq), _p(tile_q0), n, _p(out), out.stride(0), num_q_heads, num_kv_heads, head_dim,
+                group.page_size, window, float(scale), _p(scratch), scratch.numel() * 4 if scratch is not None else 0,
+                int(ctx.max_ctx_len), 0, int(chunk), None, None, None, None, 0, float(softcap or 0.0), value_dim, int(v_share),
+                1 if out.dtype == torch.float32 else 0, _stream()), "paged_attention_prefill_tc_values")
         tokens, nd = ctx.single_tokens if ctx.single_tokens is not None else (None, 0)
         if nd > 0 and splits_ok:
             single_tokens(tokens, nd)
@@ -1959,7 +2016,6 @@ def capped_attention(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
             plain(tokens, nd)
         return
     plain()
-
 
 
 def routed_combine(parts: torch.Tensor, h: Optional[torch.Tensor], w_same: Optional[torch.Tensor], shared: Optional[torch.Tensor],
@@ -2000,22 +2056,42 @@ def moe_route_biased(z: torch.Tensor, num_experts: int, real: int, top: int, ren
 
 def rope_halves_value_write(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, nq: int, nkv: int, hd: int, hdv: int,
                             cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rot: int, slot_map: torch.Tensor,
-                            q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor) -> None:
-    """q, k (heads of ``hd``) and v (heads of ``hdv``) are column blocks of the float32 rows ``proj``; the first ``rot``
-    dimensions of every q and k head turn (i with i + rot/2) by cos/sin float32 [T, rot/2]; q goes to ``q_out`` [T, nq*hd],
-    k and v to the token's cache slot (k_cache [slots, nkv, hd], v_cache [slots, nkv, hdv])."""
-    _dev(proj, cos, sin, slot_map, q_out, k_cache, v_cache)
-    T = proj.shape[0]
-    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and q_out.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
+                            q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, bias: Optional[torch.Tensor] = None,
+                            nv: Optional[int] = None) -> None:
+    """q, k (heads of ``hd``) and v (``nv`` heads of ``hdv``, default ``nkv``) are column blocks of the rows ``proj`` [T, *]
+    (either dtype) or of float32 partial products [P, T, *]; ``bias`` (float32, a number per column) is added first; the
+    first ``rot`` dimensions of every q and k head turn (i with i + rot/2) by cos/sin float32 [T, rot/2]; q goes to
+    ``q_out`` [T, nq*hd], k and v to the token's cache slot (k_cache [slots, nkv, hd], v_cache [slots, nv, hdv])."""
+    _dev(proj, cos, sin, slot_map, q_out, k_cache, v_cache, bias)
+    nparts, stride = 1, 0
+    if proj.dim() == 3:
+        assert proj.dtype == torch.float32 and proj.is_contiguous()
+        nparts, stride = proj.shape[0], proj.shape[1] * proj.shape[2]
+    T, cols = proj.shape[-2:]
+    nv = nkv if nv is None else int(nv)
+    assert proj.stride(-1) == 1 and q_out.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert q_off + nq * hd <= cols and k_off + nkv * hd <= cols and v_off + nv * hdv <= cols
     assert k_cache.dtype == v_cache.dtype and slot_map.dtype == torch.int32
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() >= max(q_off + nq * hd, k_off + nkv * hd, v_off + nv * hdv))
     if rot:
         assert cos is not None and tuple(cos.shape) == (T, rot // 2) and cos.is_contiguous() and sin.is_contiguous()
-    _check(lib().aien_rope_halves_value_write(_p(proj), proj.stride(0), int(q_off), int(k_off), int(v_off), int(nq), int(nkv), int(hd), int(hdv),
-                                              _p(cos), _p(sin), int(rot), _p(slot_map), _p(q_out), dt(q_out), q_out.stride(0), _p(k_cache),
-                                              _p(v_cache), dt(k_cache), T, _stream()), "rope_halves_value_write")
+    _check(lib().aien_rope_halves_value_write(_p(proj), dt(proj), proj.stride(-2), nparts, stride, _p(bias), int(q_off), int(k_off), int(v_off),
+                                              int(nq), int(nkv), int(hd), nv, int(hdv), _p(cos), _p(sin), int(rot), _p(slot_map), _p(q_out),
+                                              dt(q_out), q_out.stride(0), _p(k_cache), _p(v_cache), dt(k_cache), T, _stream()),
+           "rope_halves_value_write")
 
 
-# ---------------------------------------------------------------------------- several branches pending at once
+def map_difference_norm(a: torch.Tensor, out: torch.Tensor, heads: int, per_group: int, value_dim: int, lam: float, eps: float, mult: float) -> None:
+    """a float32 [T, 2 * heads * value_dim]: per group the first map's outputs of its ``per_group`` heads, then the second
+    map's.  out [T, heads * value_dim] = o / sqrt(mean(o^2) + eps) * mult per head with o = a1 - lam * a2."""
+    _dev(a, out)
+    T = a.shape[0]
+    assert a.dtype == torch.float32 and a.stride(1) == 1 and out.stride(1) == 1
+    assert a.shape[1] == 2 * heads * value_dim and tuple(out.shape) == (T, heads * value_dim)
+    _check(lib().aien_map_difference_norm(_p(a), a.stride(0), _p(out), dt(out), out.stride(0), T, int(heads), int(per_group), int(value_dim),
+                                          float(lam), float(eps), float(mult), _stream()), "map_difference_norm")
+
+
 MAX_SUM_TERMS = 3
 
 

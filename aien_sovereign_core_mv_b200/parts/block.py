@@ -46,6 +46,28 @@ class PreNormBlock(Block):
         return self.feed_forward.forward(ctx, h2, sink=sink) if sink is not None else self.feed_forward.forward(ctx, h2)
 
 
+@register_block("prenorm_mixer")
+class PreNormMixerBlock(PreNormBlock):
+    """The pre-norm block of a layer that has no feed-forward: x -> norm -> mixer -> +x."""
+
+    norm_slots = ("norm_in",)
+
+    def __init__(self, mixer: Mixer, feed_forward: Optional[FeedForward], norm_in: Norm):
+        if feed_forward is not None:
+            raise ValueError("the block kind 'prenorm_mixer' takes no feed-forward")
+        super().__init__(mixer, None, norm_in, None)
+
+    def parts(self):
+        return {"norm_in": self.norm_in, "mixer": self.mixer}
+
+    def forward(self, ctx: StepContext, x: torch.Tensor, delta, run: RunBinding, next_norm: Optional[Norm] = None):
+        h = self.norm_in.forward(ctx, x, delta)
+        if isinstance(h, Prenormed) and not self.mixer.takes_prenormed:
+            h = h.materialise(ctx)
+        sink = next_norm.sink(ctx, x) if (next_norm is not None and self.mixer.feeds_residual) else None
+        return self.mixer.forward(ctx, h, run, sink=sink) if sink is not None else self.mixer.forward(ctx, h, run)
+
+
 @register_block("branchnorm")
 class BranchNormBlock(Block):
     """x -> x + norm_mixer(mixer(x)) -> x + norm_ff(feed_forward(x)): the sublayers read the

@@ -97,11 +97,12 @@ class NormedTableEmbedding(TableEmbedding):
 class LinearHead(Head):
     """logits = rows . W^T with W = ``weight`` [vocab, hidden], or the embedding's table when
     tied: the same buffer, no copy (crates/aien-inference-abi/src/weights.rs:131-136,
-    src/transformer_backend.rs:1370-1386).  ``softcap`` c > 0: logits = c * tanh(logits / c), in float32."""
+    src/transformer_backend.rs:1370-1386).  ``scale``: the logits are multiplied by it; then, ``softcap`` c > 0:
+    logits = c * tanh(logits / c); both in float32."""
 
-    def __init__(self, vocab_size: int, hidden_size: int, tied: bool = False, softcap: float = 0.0):
+    def __init__(self, vocab_size: int, hidden_size: int, tied: bool = False, softcap: float = 0.0, scale: float = 1.0):
         self.vocab_size, self.hidden_size, self.tied = int(vocab_size), int(hidden_size), bool(tied)
-        self.softcap = float(softcap or 0.0)
+        self.softcap, self.scale = float(softcap or 0.0), float(scale)
         self.weight: Optional[torch.Tensor] = None
 
     def param_shapes(self):
@@ -118,8 +119,8 @@ class LinearHead(Head):
 
     def forward(self, ctx: StepContext, rows: torch.Tensor, logits: torch.Tensor) -> None:
         linear(ctx, rows, self.weight, out=logits)
-        if self.softcap > 0.0:
-            K.softcap(logits, self.softcap)
+        if self.softcap > 0.0 or self.scale != 1.0:
+            K.softcap(logits, self.softcap, self.scale)
 
 
 @register_pass_input("step_vector")

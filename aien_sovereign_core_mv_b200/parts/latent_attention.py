@@ -14,12 +14,12 @@ from .linear import linear, stack_rows
 @register_mixer("latent_attention")
 class LatentAttention(Mixer):
     """Queries through a latent: c_q = RMSnorm(W_dq h) (weight ``dq_norm``), q = W_uq c_q, per head ``head_dim``
-    unrotated then ``rot_dim`` rotated numbers.  Keys and values through a latent: W_dkv h has ``kv_rank`` + ``rot_dim``
+    unrotated then ``rot_dim`` rotated numbers; without a ``q_rank`` (0) q = W_q h.  Keys and values through a latent: W_dkv h has ``kv_rank`` + ``rot_dim``
     rows; the first kv_rank, RMS-normed (weight ``dkv_norm``), are the latent c, the rest one rotated key part shared by
     all heads.  Per head the unrotated key is W_uk c and the value W_uv c; score = (q_unrot . k_unrot + q_rot . k_rot) *
     ``scale``; causal, optionally only the last ``window`` positions (the token itself included); optionally a learned
-    sink per head in the softmax denominator; optionally (``head_gate``) head h's output times sigmoid(W_g h)_h; W_o on the
-    heads.  The rotation turns neighbouring pairs of the first
+    sink per head in the softmax denominator; optionally (``head_gate``) head h's output times sigmoid(W_g h)_h, or (``out_gate``) the concatenated
+    heads element by element times sigmoid(W_g h); W_o on the heads.  The rotation turns neighbouring pairs of the first
     ``rotary_dim`` numbers of the rotated part (the position part's table).
 
     The cache keeps one row [c | k_rot] per token and nothing per head.  The kernels never build a head's keys or
@@ -30,11 +30,12 @@ class LatentAttention(Mixer):
 
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, value_dim: int, kv_rank: int, q_rank: int,
                  position: Position, scale: Optional[float] = None, window: int = 0, cache_window: Optional[int] = None,
-                 sink: bool = False, norm_eps: float = 1e-6, own_cache: bool = True, head_gate: bool = False):
+                 sink: bool = False, norm_eps: float = 1e-6, own_cache: bool = True, head_gate: bool = False,
+                 out_gate: bool = False):
         self.hidden_size, self.num_heads, self.head_dim, self.rot_dim = int(hidden_size), int(num_heads), int(head_dim), int(rot_dim)
-        self.value_dim, self.kv_rank, self.q_rank = int(value_dim), int(kv_rank), int(q_rank)
-        if min(self.num_heads, self.head_dim, self.value_dim, self.kv_rank, self.q_rank) <= 0 or self.rot_dim < 0:
-            raise ValueError("latent attention: heads, head_dim, value_dim, kv_rank and q_rank must be positive")
+        self.value_dim, self.kv_rank, self.q_rank = int(value_dim), int(kv_rank), int(q_rank or 0)
+        if min(self.num_heads, self.head_dim, self.value_dim, self.kv_rank) <= 0 or min(self.q_rank, self.rot_dim) < 0:
+            raise ValueError("latent attention: heads, head_dim, value_dim and kv_rank must be positive")
         if self.rot_dim and getattr(position, "pairing", "interleaved") != "interleaved":
             raise ValueError("this mixer rotates neighbouring pairs (2i with 2i+1): give it a position part with pairing='interleaved'")
         self.position = position
@@ -47,9 +48,13 @@ class LatentAttention(Mixer):
         if self.window < 0 or (self.window == 0) != (self.cache_window == 0) or self.cache_window < self.window:
             raise ValueError("cache_window must cover window (0 for both: every earlier position is seen)")
         self.sink, self.norm_eps, self.own_cache = bool(sink), float(norm_eps), bool(own_cache)
-        self.head_gate = bool(head_gate)
-        self.side_rows, self.riders = (self.num_heads if self.head_gate else 0), 0     # rows of the first product behind the query latent
+        self.head_gate, self.out_gate = bool(head_gate), bool(out_gate)
+        if self.head_gate and self.out_gate:
+            raise ValueError("latent attention: a gate per head or one per element, not both")
         self.q_head = self.head_dim + self.rot_dim
+        self.gate_rows = self.num_heads if self.head_gate else (self.num_heads * self.value_dim if self.out_gate else 0)
+        self.q_cols = self.q_rank or self.num_heads * self.q_head        # rows of the first product that belong to the query
+        self.side_rows, self.riders = self.gate_rows, 0                  # and those behind them: gates, riders
         self.row = self.kv_rank + self.rot_dim
         self.w_down = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = self.dq_norm = self.dkv_norm = self.sinks = None
 
@@ -57,14 +62,15 @@ class LatentAttention(Mixer):
     def param_shapes(self):
         H, n = self.hidden_size, self.num_heads
         shapes = {"dq_proj": ((self.q_rank, H), "matrix"), "dq_norm": ((self.q_rank,), "norm"),
-                  "uq_proj": ((n * self.q_head, self.q_rank), "matrix"), "uk_proj": ((n * self.head_dim, self.kv_rank), "matrix"),
+                  "uq_proj": ((n * self.q_head, self.q_rank), "matrix")} if self.q_rank else {"q_proj": ((n * self.q_head, H), "matrix")}
+        shapes = {**shapes, "uk_proj": ((n * self.head_dim, self.kv_rank), "matrix"),
                   "uv_proj": ((n * self.value_dim, self.kv_rank), "matrix"), "o_proj": ((H, n * self.value_dim), "matrix")}
         if self.own_cache:
             shapes.update({"dkv_proj": ((self.row, H), "matrix"), "dkv_norm": ((self.kv_rank,), "norm")})
         if self.sink:
             shapes["sink"] = ((n,), "vector")
-        if self.head_gate:
-            shapes["g_proj"] = ((n, H), "matrix")
+        if self.gate_rows:
+            shapes["g_proj"] = ((self.gate_rows, H), "matrix")
         return shapes
 
     takes_riders = True
@@ -72,26 +78,30 @@ class LatentAttention(Mixer):
     def _stack(self, dq, side, dkv):
         """Rows query latent | head gates and riders, filled up to whole vectors | key/value latent | shared key part."""
         head = stack_rows([dq] + side, 8) if side else dq
-        self.side_rows = head.shape[0] - self.q_rank
+        self.side_rows = head.shape[0] - self.q_cols
         self.w_down = stack_rows([head] + ([dkv] if dkv is not None else []))
 
     def set_riders(self, weight):
         w = self.w_down
-        gates = [w[self.q_rank:self.q_rank + self.num_heads]] if self.head_gate else []
-        dkv = w[self.q_rank + self.side_rows:] if self.own_cache else None
+        gates = [w[self.q_cols:self.q_cols + self.gate_rows]] if self.gate_rows else []
+        dkv = w[self.q_cols + self.side_rows:] if self.own_cache else None
         self.riders = weight.shape[0]
-        self._stack(w[:self.q_rank], gates + [weight], dkv)
+        self._stack(w[:self.q_cols], gates + [weight], dkv)
 
     def bind(self, tensors):
-        self._stack(tensors["dq_proj"], [tensors["g_proj"]] if self.head_gate else [], tensors["dkv_proj"] if self.own_cache else None)
-        self.w_uq, self.w_o = tensors["uq_proj"].contiguous(), tensors["o_proj"].contiguous()
+        self._stack(tensors["dq_proj" if self.q_rank else "q_proj"], [tensors["g_proj"]] if self.gate_rows else [],
+                    tensors["dkv_proj"] if self.own_cache else None)
+        self.w_uq = tensors["uq_proj"].contiguous() if self.q_rank else None
+        self.w_o = tensors["o_proj"].contiguous()
         n = self.num_heads
         # per head [kv_rank, head_dim]: the matrix that takes a head's unrotated query to the latent
         self.w_uk_t = tensors["uk_proj"].view(n, self.head_dim, self.kv_rank).transpose(1, 2).contiguous()
         self.w_uv = tensors["uv_proj"].view(n, self.value_dim, self.kv_rank).contiguous()
-        self.dq_norm = tensors["dq_norm"].contiguous()
+        self.dq_norm = tensors["dq_norm"].contiguous() if self.q_rank else None
         if self.own_cache:
-            self.dkv_norm = tensors["dkv_norm"].to(self.dq_norm.dtype).contiguous()
+            self.dkv_norm = tensors["dkv_norm"].contiguous()
+            if self.dq_norm is not None:
+                self.dkv_norm = self.dkv_norm.to(self.dq_norm.dtype)
         if self.sink:
             self.sinks = tensors["sink"].float().contiguous()           # the softmax is float32
 
@@ -101,7 +111,7 @@ class LatentAttention(Mixer):
 
     def workspace_bytes(self, lim):
         n = self.num_heads
-        per_token = (self.q_rank + self.side_rows + self.row) * 4 + self.q_rank * lim.itemsize + n * self.q_head * 4 + n * self.row * 4 \
+        per_token = (self.q_cols + self.side_rows + self.row) * 4 + self.q_rank * lim.itemsize + n * self.q_head * 4 + n * self.row * 4 \
             + n * self.kv_rank * lim.itemsize + n * self.value_dim * lim.itemsize + self.hidden_size * 4
         # the partial results of a step with few tiles: tokens * heads * ksplit rows, which latent_attention_tc_ksplit keeps
         # below 296 tiles' worth of 64 rows
@@ -116,17 +126,18 @@ class LatentAttention(Mixer):
         writes = run.writes and self.own_cache
         if run.writes and not self.own_cache:
             raise RuntimeError("a latent-attention layer without its own key/value projection was bound to write a cache")
-        kv_off = self.q_rank + self.side_rows
+        kv_off = self.q_cols + self.side_rows
         w_down = self.w_down if writes else self.w_down[:kv_off]
-        d = linear(ctx, h, w_down, out_dtype=torch.float32)
+        tc = K.latent_attention_tc_supports(cache.dtype, self.kv_rank, self.rot_dim) and ctx.dtype == torch.bfloat16
+        # a query latent is normed in float32; without one the rows are an operand of the next product as they are
+        d = linear(ctx, h, w_down, out_dtype=torch.float32 if self.q_rank or self.riders or not tc else torch.bfloat16)
         rot = self.position.rotary(ctx) if self.rotary_dim else None
         cos, sin, rdims = rot if rot is not None else (None, None, 0)
-        cq = ws.take((T, self.q_rank), ctx.dtype)
+        cq = ws.take((T, self.q_rank), ctx.dtype) if self.q_rank else None
         K.latent_prepare(d, self.q_rank, self.dq_norm, self.norm_eps, cq, kv_off, self.kv_rank, self.rot_dim, rdims,
                          self.dkv_norm, cos, sin, group.slot_map if writes else None, cache if writes else None)
-        tc = K.latent_attention_tc_supports(cache.dtype, self.kv_rank, self.rot_dim) and ctx.dtype == torch.bfloat16
         # per head: unrotated | rotated part, before rotation; an operand of the tensor-core products where those run
-        q = linear(ctx, cq, self.w_uq, out_dtype=torch.bfloat16 if tc else torch.float32)
+        q = linear(ctx, cq, self.w_uq, out_dtype=torch.bfloat16 if tc else torch.float32) if self.q_rank else d
         qf = ws.take((T, n * self.row), torch.bfloat16 if tc else torch.float32)    # per head: the query in the latent | rotated part
         K.head_project(q, self.q_head, 0, self.w_uk_t, qf, self.row, 0)
         if self.rot_dim:
@@ -143,9 +154,9 @@ class LatentAttention(Mixer):
                                self.rot_dim, group.page_size, self.window, self.scale, self.sinks)
         o = ws.take((T, n * self.value_dim), ctx.dtype)
         K.head_project(mixed, self.kv_rank, 0, self.w_uv, o, self.value_dim, 0,
-                       gate=d[:, self.q_rank:self.q_rank + n] if self.head_gate else None)
+                       gate=d[:, self.q_cols:self.q_cols + self.gate_rows] if self.gate_rows else None)
         y = linear(ctx, o, self.w_o, out_dtype=torch.float32, may_defer_sum=True)        # the consumer's norm adds partial products
         if not self.riders:
             return y
-        r0 = self.q_rank + (n if self.head_gate else 0)
+        r0 = self.q_cols + self.gate_rows
         return y, d[:, r0:r0 + self.riders]

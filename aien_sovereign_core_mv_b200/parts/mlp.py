@@ -13,12 +13,15 @@ from .linear import linear, linear_into_residual, linear_prenormed, _FORCE
 
 @register_feed_forward("swiglu")
 class SwiGLU(FeedForward):
-    """y = (silu(h Wg^T) * (h Wu^T)) Wd^T, no bias (crates/aien-inference-abi/src/
+    """y = (act(h Wg^T) * (h Wu^T)) Wd^T with ``act`` "silu" (or "gelu_tanh", the tanh form of the gelu), no bias (crates/aien-inference-abi/src/
     transformer_backend.rs:1322-1362, silu in src/backend.rs:572-579).  gate and up are one
     product over the stacked rows gate | up (src/resident.rs:284-288)."""
 
-    def __init__(self, hidden_size: int, intermediate_size: int):
+    def __init__(self, hidden_size: int, intermediate_size: int, act: str = "silu"):
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
+        if act not in K.GATED_ACTS:
+            raise ValueError(f"activation {act!r}: known are {sorted(K.GATED_ACTS)}")
+        self.act, self.epilogue = act, K.GATED_ACTS[act]
         self.w_gate_up = self.w_down = None
 
     def param_shapes(self):
@@ -48,20 +51,20 @@ class SwiGLU(FeedForward):
     feeds_residual = True
 
     def hidden(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
-        """silu(h Wg^T) * (h Wu^T)."""
+        """act(h Wg^T) * (h Wu^T)."""
         act = ctx.workspace.take((ctx.num_tokens, self.intermediate_size), ctx.dtype)
         if self.group == 8 and h.shape[0] <= K.GEMV_ROUTE_ROWS and K.gemv_supports(h, self.w_gate_up, act):
-            K.gemv(h, self.w_gate_up, act, epilogue=1)          # silu(gate)*up inside the product
+            K.gemv(h, self.w_gate_up, act, epilogue=self.epilogue)      # act(gate)*up inside the product
         elif self.group == 8 and K.gemm_tc_supports(h, self.w_gate_up, act) and not _FORCE:
-            K.gemm_tc(h, self.w_gate_up, act, epilogue=1)       # the same, in the tensor-core epilogue
+            K.gemm_tc(h, self.w_gate_up, act, epilogue=self.epilogue)   # the same, in the tensor-core epilogue
         else:
             gu = linear(ctx, h, self.w_gate_up)
-            K.swiglu(gu, act, self.group)
+            K.swiglu(gu, act, self.group, self.act)
         return act
 
     def forward(self, ctx: StepContext, h, sink: Optional[ResidualSink] = None):
         if isinstance(h, Prenormed):
-            act = linear_prenormed(ctx, h, self.w_gate_up, epilogue=1) if self.group == 8 else None
+            act = linear_prenormed(ctx, h, self.w_gate_up, epilogue=1) if self.group == 8 and self.act == "silu" else None
             if act is not None:
                 return linear_into_residual(ctx, act, self.w_down, sink) or linear(ctx, act, self.w_down, may_defer_sum=True)
             h = h.materialise(ctx)

@@ -1,4 +1,4 @@
-"""RMSNorm with the residual sum fused in front of it."""
+"""RMSNorm and layer norm with the residual sum fused in front of them."""
 from __future__ import annotations
 
 from typing import Optional
@@ -94,4 +94,41 @@ class RMSNorm(Norm):
             delta = None
         out = ctx.workspace.take(tuple(x.shape), ctx.dtype)
         K.add_rmsnorm(x, delta, self.weight, self.eps, out)
+        return out
+
+
+@register_norm("layernorm")
+class LayerNorm(Norm):
+    """h = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w over the last axis, no bias.  All of it float32; x is the float32
+    residual stream and is updated in place when ``delta`` is given.  ``norm_stream`` norms the stream in place (the
+    embedding's norm)."""
+
+    def __init__(self, size: int, eps: float):
+        self.size, self.eps = int(size), float(eps)
+        self.weight: Optional[torch.Tensor] = None
+
+    def param_shapes(self):
+        return {"weight": ((self.size,), "norm")}
+
+    def bind(self, tensors):
+        self.weight = tensors["weight"].contiguous()
+
+    def workspace_bytes(self, lim):
+        return lim.max_tokens * self.size * lim.itemsize + 256
+
+    def norm_stream(self, ctx: StepContext, x: torch.Tensor, want_copy: bool = False):
+        h = ctx.workspace.take(tuple(x.shape), ctx.dtype) if (want_copy and ctx.dtype != torch.float32) else None
+        K.stream_norm_inplace(x, self.weight, self.eps, h=h, center=True)
+        return (h if h is not None else x) if want_copy else None
+
+    def forward(self, ctx: StepContext, x: torch.Tensor, delta):
+        if isinstance(delta, NormedStream) and delta.norm is self:
+            return delta.h
+        if isinstance(delta, (Prenormed, NormedStream, StreamCopy)):
+            delta = None                          # the stream is up to date
+        if isinstance(delta, (ScaledSum, SumTerms)):
+            add_to_residual(ctx, x, delta)
+            delta = None
+        out = ctx.workspace.take(tuple(x.shape), ctx.dtype)
+        K.add_layernorm(x, delta, self.weight, self.eps, out)
         return out

@@ -1,4 +1,4 @@
-"""Rotary position encoding: frequency table, optional llama3 smoothing, per-step cos/sin."""
+"""Rotary position encoding: frequency table, optional llama3 smoothing or YaRN ramp, per-step cos/sin."""
 from __future__ import annotations
 
 import math
@@ -39,16 +39,34 @@ def inverse_frequencies(head_dim: int, theta: float, scaling: Optional[dict] = N
     return inv
 
 
+def yarn_frequencies(dims: int, theta: float, factor: float, original: float, fast: float, slow: float):
+    """(frequencies, factor on cos and sin).  A pair that turns often within ``original`` positions keeps its frequency, one
+    that turns seldom takes it divided by ``factor``; between the pair indices that turn ``fast`` and ``slow`` times the two
+    are mixed linearly in the index.  Both tables are multiplied by 0.1 ln(factor) + 1."""
+    def pair_that_turns(times):
+        return dims * math.log(original / (2.0 * math.pi * times)) / (2.0 * math.log(theta))
+
+    lo, hi = max(math.floor(pair_that_turns(fast)), 0), min(math.ceil(pair_that_turns(slow)), dims - 1)
+    span = max(hi - lo, 0.001)
+    out = []
+    for i in range(dims // 2):
+        f, r = theta ** (-2.0 * i / dims), min(max((i - lo) / span, 0.0), 1.0)
+        out.append(f / factor * r + f * (1.0 - r))
+    return out, 0.1 * math.log(factor) + 1.0
+
+
 @register_position("rotary")
 class RotaryPosition(Position):
     """angle = position * inv_freq in float64, cos and sin rounded to float32
     (crates/aien-inference-abi/src/tensor.rs:150-188).  The table of a step is built once and
     shared by every layer that uses the same part.  ``pairing`` says which dimensions a mixer
     rotates together: "halves" (i with i + d/2, rotate_half) or "interleaved" (2i with 2i+1); the
-    table is the same, the mixer's kernel reads ``pairing``.  ``linear_factor`` f: every frequency is divided by f."""
+    table is the same, the mixer's kernel reads ``pairing``.  ``linear_factor`` f: every frequency is divided by f.
+    ``yarn`` {factor, original, fast, slow}: see :func:`yarn_frequencies`."""
 
     def __init__(self, head_dim: int, theta: float, scaling: Optional[dict] = None, rotary_dim: Optional[int] = None,
-                 pairing: str = "halves", theta_as_float32: bool = True, linear_factor: float = 1.0):
+                 pairing: str = "halves", theta_as_float32: bool = True, linear_factor: float = 1.0,
+                 yarn: Optional[dict] = None):
         if pairing not in ("halves", "interleaved"):
             raise ValueError(f"rotary pairing {pairing!r}: 'halves' or 'interleaved'")
         self.pairing = pairing
@@ -61,7 +79,13 @@ class RotaryPosition(Position):
         self.linear_factor = float(linear_factor or 1.0)
         if self.linear_factor <= 0.0:
             raise ValueError(f"linear_factor {linear_factor!r} must be positive")
+        if yarn and (scaling or self.linear_factor != 1.0):
+            raise ValueError("one frequency scaling at a time")
+        self.mult = 1.0
         self._inv_host = inverse_frequencies(self.head_dim, self.theta, self.scaling, self.rotary_dim, bool(theta_as_float32), self.linear_factor)
+        if yarn:
+            self._inv_host, self.mult = yarn_frequencies(self.rotary_dim, self.theta, float(yarn["factor"]), float(yarn["original"]),
+                                                         float(yarn["fast"]), float(yarn["slow"]))
         self._inv_dev: Optional[torch.Tensor] = None
 
     def step_workspace_bytes(self, max_tokens):
@@ -76,7 +100,7 @@ class RotaryPosition(Position):
             half = self.rotary_dim // 2
             cos = ctx.workspace.take_step((ctx.num_tokens, half), torch.float32)
             sin = ctx.workspace.take_step((ctx.num_tokens, half), torch.float32)
-            K.rope_table(ctx.positions, self._inv_dev, cos, sin)
+            K.rope_table(ctx.positions, self._inv_dev, cos, sin, self.mult)
             hit = (cos, sin, self.rotary_dim)
             ctx.shared[key] = hit
         return hit
