@@ -1,7 +1,7 @@
 #!/usr/bin/env python3
 """Headline measurement: decode tokens per second of the Qwen3-8B-shaped model on one B200.
 
-    python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch B] [--prompt-len L] [--prefill-tokens T] [--layers N] [--workload decode|llama3_8b|serving|mixed_step|dulisun|ripesun|botalorn|mumazen|kuvidra]
+    python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch B] [--prompt-len L] [--prefill-tokens T] [--layers N] [--workload decode|llama3_8b|serving|mixed_step|dulisun|ripesun|botalorn|mumazen|kuvidra|folavik]
 
 A step is one decode step of a batch of requests that each hold a 1,024-token prompt (context
 limit 4,096, pages of 16 tokens), random bfloat16 weights, synthetic uniform token ids.  One JSON
@@ -699,15 +699,62 @@ KUVIDRA_SHAPES = (
 )
 
 
+def _prefill_and_decode(cfg, V: int, P: int, CTX: int) -> dict:
+    """One model (random bfloat16 weights): a prompt of P tokens in one step, then decode steps of 8 and 64 requests at CTX tokens
+    of context (captured graphs), timed on the device with CUDA events after warm-up."""
+    import torch
+    from aien_sovereign_core_mv_b200 import Engine, EngineConfig
+    from aien_sovereign_core_mv_b200 import kernels as K
+    ec = EngineConfig(dtype="bfloat16", page_size=16, max_cache_tokens=64 * (CTX + 64) + P + 64, max_requests=64,
+                      max_batch_tokens=P, max_context=4096, max_batch_size=64)
+    eng = Engine.from_config(cfg, seed=5, engine_config=ec, init_std=0.02, device_init=True)
+    toks = lambda n, s: [(7 * i + 13 * s) % V for i in range(n)]
+
+    def timed(fn, warm, reps):
+        for i in range(warm):
+            fn(i)
+        torch.cuda.synchronize()
+        ms = []
+        for i in range(reps):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn(warm + i)
+            e1.record()
+            torch.cuda.synchronize()
+            ms.append(e0.elapsed_time(e1))
+        return sorted(ms)[len(ms) // 2]
+
+    def prefill(i):
+        eng.step([(9000 + i, toks(P, i), [P - 1])])
+        eng.end_request(9000 + i)
+
+    out = {}
+    torch.cuda.profiler.start()
+    t = timed(prefill, 3, 5)
+    out["prefill_2048"] = {"ms": round(t, 3), "tokens_per_s": round(P / t * 1e3, 1)}
+    for batch in (8, 64):
+        for r in range(0, batch, 2):
+            eng.step([(r, toks(CTX, r), []), (r + 1, toks(CTX, r + 1), [])])
+        t = timed(lambda i: eng.step([(r, [(i + r) % V], [0]) for r in range(batch)]), 4, 12)
+        out[f"decode_b{batch}"] = {"ms": round(t, 3), "tokens_per_s": round(batch / t * 1e3, 1)}
+        for r in range(batch):
+            eng.end_request(r)
+    torch.cuda.profiler.stop()
+    eng.check_waits()
+    out["wait_errors"] = sum(1 for w in K.read_wait_errors() if w != 0)
+    out["weight_bytes"] = int(sum(t.numel() * t.element_size() for p in eng.model.parts() for t in vars(p).values()
+                                  if isinstance(t, torch.Tensor) and t.dim() >= 2))
+    del eng
+    torch.cuda.empty_cache()
+    return out
+
+
 def kuvidra_workload(only: str = "") -> int:
     """Prefill and decode throughput of the Kuvidra design at a few sizes that resemble a real model's layers (random
     bfloat16 weights), each beside the Ripesun model and the dense Qwen3-style model of equal size.  Prefill: one prompt of 2,048
     tokens; decode: 8 and 64 requests at 1,024 tokens of context, captured graphs.  Timed on the device with CUDA events
     after warm-up; every step reads more weights than L2 holds.  The timed steps lie between cudaProfilerStart and
     cudaProfilerStop.  AIEN_BENCH_MODELS names the models to run (default: all)."""
-    import torch
-    from aien_sovereign_core_mv_b200 import Engine, EngineConfig
-    from aien_sovereign_core_mv_b200 import kernels as K
     results = []
     P, CTX = 2048, 1024
     which_only = os.environ.get("AIEN_BENCH_MODELS", "").split(",") if os.environ.get("AIEN_BENCH_MODELS") else None
@@ -730,51 +777,69 @@ def kuvidra_workload(only: str = "") -> int:
         for which, cfg in (("kuvidra", _kuvidra_config(**sz)), ("ripesun", ripesun), ("dense", dense)):
             if which_only and which not in which_only:
                 continue
-            ec = EngineConfig(dtype="bfloat16", page_size=16, max_cache_tokens=64 * (CTX + 64) + P + 64, max_requests=64,
-                              max_batch_tokens=P, max_context=4096, max_batch_size=64)
-            eng = Engine.from_config(cfg, seed=5, engine_config=ec, init_std=0.02, device_init=True)
-            V = sz["vocab"]
-            toks = lambda n, s: [(7 * i + 13 * s) % V for i in range(n)]
-
-            def timed(fn, warm, reps):
-                for i in range(warm):
-                    fn(i)
-                torch.cuda.synchronize()
-                ms = []
-                for i in range(reps):
-                    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-                    e0.record()
-                    fn(warm + i)
-                    e1.record()
-                    torch.cuda.synchronize()
-                    ms.append(e0.elapsed_time(e1))
-                return sorted(ms)[len(ms) // 2]
-
-            def prefill(i):
-                eng.step([(9000 + i, toks(P, i), [P - 1])])
-                eng.end_request(9000 + i)
-
-            out = {}
-            torch.cuda.profiler.start()
-            t = timed(prefill, 3, 5)
-            out["prefill_2048"] = {"ms": round(t, 3), "tokens_per_s": round(P / t * 1e3, 1)}
-            for batch in (8, 64):
-                for r in range(0, batch, 2):
-                    eng.step([(r, toks(CTX, r), []), (r + 1, toks(CTX, r + 1), [])])
-                t = timed(lambda i: eng.step([(r, [(i + r) % V], [0]) for r in range(batch)]), 4, 12)
-                out[f"decode_b{batch}"] = {"ms": round(t, 3), "tokens_per_s": round(batch / t * 1e3, 1)}
-                for r in range(batch):
-                    eng.end_request(r)
-            torch.cuda.profiler.stop()
-            eng.check_waits()
-            out["wait_errors"] = sum(1 for w in K.read_wait_errors() if w != 0)
-            out["weight_bytes"] = int(sum(t.numel() * t.element_size() for p in eng.model.parts() for t in vars(p).values()
-                                          if isinstance(t, torch.Tensor) and t.dim() >= 2))
-            row[which] = out
-            del eng
-            torch.cuda.empty_cache()
+            row[which] = _prefill_and_decode(cfg, sz["vocab"], P, CTX)
         results.append(row)
     print(json.dumps({"metric": "kuvidra_beside_ripesun_and_dense", "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True,
+                      "dtype": "bf16", "data": "synthetic", "impl": "ours", "shapes": results,
+                      "config": {"prefill_tokens": P, "decode_context": CTX, "page_size": 16, "seed": 5,
+                                 "l2": "weights read per step exceed L2"}}))
+    return 0
+
+
+def _folavik_config(width, heads, kv, diff_dim, diff_vdim, dim, vdim, lat_dim, lat_vdim, kv_rank, span, ff, layers, vocab):
+    mlp = {"kind": "dense", "ff": ff}
+    dif = {"type": "attention_2", "mlp": mlp, "mixer": {
+        "heads": heads, "kv_heads": kv, "dim": diff_dim, "vdim": diff_vdim, "scale": diff_dim ** -0.5, "softcap": 50.0, "diff": 0.8,
+        "mask": {"size": span}, "rot": {"base": 1000000.0, "dims": diff_dim // 2,
+                                        "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    lat = {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": lat_dim, "vdim": lat_vdim, "kv_rank": kv_rank, "scale": lat_dim ** -0.5}}
+    att = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": span},
+        "rot": {"base": 500000.0, "dims": dim, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    return {"architecture": "Folavik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.5, "logit_softcap": 30.0,
+            "layers": [(dif, lat, att)[i % 3] for i in range(layers)]}
+
+
+# (name, Folavik sizes); layers go round differential attention (window), latent attention and attention inside chunks.  Beside each:
+# the Kuvidra model of the same width, heads, latent, layers and vocabulary (a matrix memory and latent attention, dense
+# feed-forwards of equal arithmetic) and the dense Qwen3-style model with the same gated feed-forward.
+FOLAVIK_SHAPES = (
+    ("w2048_h16", dict(width=2048, heads=16, kv=4, diff_dim=64, diff_vdim=128, dim=128, vdim=128, lat_dim=128, lat_vdim=128, kv_rank=512,
+                       span=1024, ff=4096, layers=6, vocab=32768)),
+    ("w4096_h32", dict(width=4096, heads=32, kv=8, diff_dim=64, diff_vdim=128, dim=128, vdim=128, lat_dim=128, lat_vdim=128, kv_rank=512,
+                       span=1024, ff=8192, layers=3, vocab=32768)),
+    ("w1024_h16", dict(width=1024, heads=16, kv=4, diff_dim=32, diff_vdim=64, dim=64, vdim=64, lat_dim=64, lat_vdim=64, kv_rank=256,
+                       span=1024, ff=2048, layers=6, vocab=32768)),
+)
+
+
+def folavik_workload(only: str = "") -> int:
+    """Prefill and decode throughput of the Folavik design at a few sizes that resemble a real model's layers (random
+    bfloat16 weights), each beside the Kuvidra model and the dense Qwen3-style model of equal size (see
+    :func:`_prefill_and_decode`); every step reads more weights than L2 holds.  AIEN_BENCH_MODELS names the models to run
+    (default: all)."""
+    results = []
+    P, CTX = 2048, 1024
+    which_only = os.environ.get("AIEN_BENCH_MODELS", "").split(",") if os.environ.get("AIEN_BENCH_MODELS") else None
+    for name, sz in FOLAVIK_SHAPES:
+        if only and only != name:
+            continue
+        kuvidra = _kuvidra_config(width=sz["width"], heads=sz["heads"], dim=sz["lat_dim"], vdim=sz["lat_vdim"], kv_rank=sz["kv_rank"],
+                                  q_rank=3 * sz["kv_rank"], mem_heads=sz["heads"], mem_dim=sz["dim"], mem_vdim=sz["vdim"], ff=sz["ff"] * 3 // 2,
+                                  experts=8, top=2, expert_ff=512, shared_ff=512, layers=sz["layers"], vocab=sz["vocab"])
+        for layer in kuvidra["layers"]:
+            layer["mlp"] = {"kind": "dense", "ff": sz["ff"] * 3 // 2}
+        dense = dict(architectures=["Qwen3ForCausalLM"], model_type="qwen3", num_hidden_layers=sz["layers"], hidden_size=sz["width"],
+                     num_attention_heads=sz["heads"], num_key_value_heads=sz["kv"], head_dim=sz["dim"], intermediate_size=sz["ff"],
+                     vocab_size=sz["vocab"], rope_theta=10000.0, rms_norm_eps=1e-6, tie_word_embeddings=False,
+                     max_position_embeddings=8192, hidden_act="silu", attention_bias=False, eos_token_id=0)
+        row = {"shape": name, "sizes": dict(sz)}
+        for which, cfg in (("folavik", _folavik_config(**sz)), ("kuvidra", kuvidra), ("dense", dense)):
+            if which_only and which not in which_only:
+                continue
+            row[which] = _prefill_and_decode(cfg, sz["vocab"], P, CTX)
+        results.append(row)
+    print(json.dumps({"metric": "folavik_beside_kuvidra_and_dense", "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True,
                       "dtype": "bf16", "data": "synthetic", "impl": "ours", "shapes": results,
                       "config": {"prefill_tokens": P, "decode_context": CTX, "page_size": 16, "seed": 5,
                                  "l2": "weights read per step exceed L2"}}))
@@ -799,11 +864,11 @@ def main() -> int:
     ap.add_argument("--top-k", type=int, default=0, help="top-k of the end-to-end run")
     ap.add_argument("--align-step-tokens", type=int, default=0,
                     help="serving workload: the scheduler cuts portions so that a step's tokens fill whole tiles of this many rows")
-    ap.add_argument("--shape", default="", help="dulisun, ripesun, botalorn, mumazen and kuvidra workloads: only this shape (default: all)")
+    ap.add_argument("--shape", default="", help="dulisun, ripesun, botalorn, mumazen, kuvidra and folavik workloads: only this shape (default: all)")
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--skip-prefill", action="store_true")
     ap.add_argument("--skip-e2e", action="store_true")
-    ap.add_argument("--workload", default="decode", choices=["decode", "llama3_8b", "serving", "mixed_step", "dulisun", "ripesun", "botalorn", "mumazen", "kuvidra"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "llama3_8b", "serving", "mixed_step", "dulisun", "ripesun", "botalorn", "mumazen", "kuvidra", "folavik"],
                     help="decode: the headline decode-step measurement (Qwen3-8B shape, 1,024-token prompts); llama3_8b: the same "
                          "line for the Llama-3-8B shape, 16 requests at contexts ending at 8,192 tokens; serving: continuous batching "
                          "of 32 requests on the Qwen3-4B shape (prompts of 64..4096 tokens, portions of 512, 256 new tokens each); "
@@ -811,7 +876,8 @@ def main() -> int:
                          "dulisun: prefill and decode of the Dulisun design at a few sizes beside the dense model of equal size; "
                          "ripesun: the same for the Ripesun design; botalorn: the Botalorn design beside Ripesun and the dense model; "
                          "mumazen: the Mumazen design beside Botalorn and the dense model; "
-                         "kuvidra: the Kuvidra design beside Ripesun and the dense model")
+                         "kuvidra: the Kuvidra design beside Ripesun and the dense model; "
+                         "folavik: the Folavik design beside Kuvidra and the dense model")
     ap.add_argument("--fill", default="prefill", choices=["prefill", "cache"],
                     help="how requests get their prompt: real prefill, or (development only) cache pages "
                          "filled with random keys/values without running the model")
@@ -839,6 +905,8 @@ def main() -> int:
         return mumazen_workload(args.shape)
     if args.workload == "kuvidra":
         return kuvidra_workload(args.shape)
+    if args.workload == "folavik":
+        return folavik_workload(args.shape)
 
     import numpy as np
     import torch
