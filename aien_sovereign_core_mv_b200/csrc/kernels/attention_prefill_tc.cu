@@ -99,9 +99,26 @@ struct PtMaps {
 // Sizes that the tiles' padding hides: hd and hdv columns of a head are real.  by_head: the maps are
 // [rows][heads][head size] (boxes of one head's 64 columns), for head sizes that are not whole chunks; the bit 0
 // stands for q and k, bit 1 for v.  v_share neighbouring key heads share a value head.  out_f32: float32 results.
+// egate (or null): bfloat16 rows of the step's tokens, ldeg numbers apart; column h * hdv + i of the result is multiplied by
+// sigmoid(egate[t][h * hdv + i]).
 struct PtSizes {
     int hdv, by_head, v_share, out_f32;
+    const __nv_bfloat16* egate;
+    long ldeg;
 };
+
+__device__ __forceinline__ float pt_sigmoid(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
+// 8 neighbouring numbers of a gate row
+__device__ __forceinline__ void pt_gate8(const __nv_bfloat16* p, float* g) {
+    const uint4 r = __ldcg(reinterpret_cast<const uint4*>(p));
+    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i]));
+        g[2 * i] = pt_sigmoid(f.x);
+        g[2 * i + 1] = pt_sigmoid(f.y);
+    }
+}
 
 template <int HD, int HDV>
 __global__ void __launch_bounds__(PT_THREADS, 1)
@@ -492,6 +509,12 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
 #pragma unroll
                 for (int d = 0; d < 32; d += 8) {
                     if (c0 + d >= sz.hdv) break;
+                    if (sz.egate != nullptr) {
+                        float g8[8];
+                        pt_gate8(sz.egate + (size_t)(qs + q0 + r) * sz.ldeg + (size_t)(head_a + h) * sz.hdv + c0 + d, g8);
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) o[d + i] = __float_as_uint(__uint_as_float(o[d + i]) * g8[i]);
+                    }
                     __nv_bfloat162 a = __floats2bfloat162_rn(__uint_as_float(o[d]) * inv, __uint_as_float(o[d + 1]) * inv);
                     __nv_bfloat162 b = __floats2bfloat162_rn(__uint_as_float(o[d + 2]) * inv, __uint_as_float(o[d + 3]) * inv);
                     __nv_bfloat162 c = __floats2bfloat162_rn(__uint_as_float(o[d + 4]) * inv, __uint_as_float(o[d + 5]) * inv);
@@ -522,7 +545,7 @@ template <int HD>
 __global__ void __launch_bounds__(256) prefill_merge_splits_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                                    const int* __restrict__ q_start, const int* __restrict__ tile_seq,
                                                                    const int* __restrict__ tile_q0, void* __restrict__ out_v,
-                                                                   long out_stride, int nq, int nsplit, int hdv, int out_f32) {
+                                                                   long out_stride, int nq, int nsplit, PtSizes sz) {
     constexpr int PER = HD / 32;
     griddep_launch();
     const int lane = threadIdx.x & 31;
@@ -568,9 +591,14 @@ __global__ void __launch_bounds__(256) prefill_merge_splits_kernel(const float* 
         for (int i = 0; i < PER; ++i) acc[i] = fmaf(w, o[sp][i], acc[i]);
     }
     const float inv = L > 0.f ? 1.0f / L : 0.f;
-    if (lane * PER >= hdv) return;                       // columns that only pad the tile
-    const size_t at = (size_t)(qs + q0 + r) * out_stride + (size_t)head * hdv + lane * PER;
-    if (out_f32) {
+    if (lane * PER >= sz.hdv) return;                    // columns that only pad the tile
+    const size_t at = (size_t)(qs + q0 + r) * out_stride + (size_t)head * sz.hdv + lane * PER;
+    if (sz.egate != nullptr) {
+        const __nv_bfloat16* gr = sz.egate + (size_t)(qs + q0 + r) * sz.ldeg + (size_t)head * sz.hdv + lane * PER;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) acc[i] *= pt_sigmoid(ld_act(gr + i));
+    }
+    if (sz.out_f32) {
         float* dst = reinterpret_cast<float*>(out_v) + at;
 #pragma unroll
         for (int i = 0; i < PER; ++i) dst[i] = acc[i] * inv;
@@ -642,7 +670,7 @@ static int launch_prefill_tc(const CUtensorMap& mq, const PtMaps& mk, const PtMa
     if (launch_status() != 0) return launch_status();
     if (nsplit > 1)
         launch_chain(prefill_merge_splits_kernel<HDV>, dim3((unsigned)(part_rows / 8)), dim3(256), (size_t)0, stream, (const float*)part_o, (const float*)part_ml,
-                     q_start, tile_seq, tile_q0, out, out_stride, nq, nsplit, sz.hdv, sz.out_f32);
+                     q_start, tile_seq, tile_q0, out, out_stride, nq, nsplit, sz);
     return launch_status();
 }
 
@@ -671,6 +699,7 @@ AIEN_API int aien_paged_attention_prefill_tc_values_supports(int hd, int hdv, in
 // one more term exp(sink) in every head's softmax denominator.  With either, every tile's keys stay in one range.
 // head_scale, slopes (float32 [nq]) and gate (float32 [tokens of the step, ldg]), each of which may be null, and softcap
 // (0: none): see HeadTerms.
+// k_ld, v_ld: numbers between rows of the caches (0: the rows are contiguous); egate, ldeg: see PtSizes (bfloat16 results only).
 // hdv, v_share, out_f32: values of hdv numbers, one value head for every v_share neighbouring key heads (v_cache
 // [cache_rows, nkv / v_share * hdv], out [tokens, nq * hdv]), float32 results; hd and hdv are multiples of 8 up to 128.
 AIEN_API int aien_paged_attention_prefill_tc_values(
@@ -678,7 +707,7 @@ AIEN_API int aien_paged_attention_prefill_tc_values(
     int max_blocks, const int* q_start, const int* ctx_len, const int* tile_seq, const int* tile_q0, int num_tiles, void* out,
     long out_stride, int nq, int nkv, int hd, int page_size, int window, float scale, void* scratch, long scratch_bytes, int max_ctx,
     int force_splits, int chunk, const float* sinks, const float* head_scale, const float* slopes, const float* gate, long ldg,
-    float softcap, int hdv, int v_share, int out_f32, cudaStream_t stream) {
+    float softcap, int hdv, int v_share, int out_f32, long k_ld, long v_ld, const void* egate, long ldeg, cudaStream_t stream) {
     const HeadTerms ht{head_scale, slopes, gate, ldg, softcap > 0.f ? softcap : 0.f};
     if (num_tiles <= 0) return 0;
     if (chunk < 0) return AIEN_E_SHAPE;
@@ -686,16 +715,18 @@ AIEN_API int aien_paged_attention_prefill_tc_values(
         v_share <= 0 || nkv % v_share != 0)
         return AIEN_E_SHAPE;
     if ((q_stride & 7) || (out_stride & 7) || ((uintptr_t)q & 15) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15) ||
-        ((uintptr_t)out & 15) || ((uintptr_t)scratch & 15))
+        ((uintptr_t)out & 15) || ((uintptr_t)scratch & 15) || ((k_ld | v_ld | ldeg) & 7) || ((uintptr_t)egate & 15))
         return AIEN_E_ALIGN;
+    if (egate != nullptr && out_f32) return AIEN_E_SHAPE;
     if (force_splits < 0 || force_splits > PT_MAX_SPLITS) return AIEN_E_SHAPE;
-    const PtSizes sz{hdv, ((hd & 63) ? 1 : 0) | ((hdv & 63) ? 2 : 0), v_share, out_f32 ? 1 : 0};
+    const PtSizes sz{hdv, ((hd & 63) ? 1 : 0) | ((hdv & 63) ? 2 : 0), v_share, out_f32 ? 1 : 0, (const __nv_bfloat16*)egate, ldeg};
     CUtensorMap mq;
     static PtMaps mk, mv;                      // large: kept out of the stack; filled for every launch
     static std::mutex mu;
     std::lock_guard<std::mutex> lock(mu);
     const int nv = nkv / v_share;
     const uint64_t k_cols = (uint64_t)nkv * hd, v_cols = (uint64_t)nv * hdv;
+    const uint64_t kld = k_ld > 0 ? (uint64_t)k_ld : k_cols, vld = v_ld > 0 ? (uint64_t)v_ld : v_cols;
     auto rows_of = [&](CUtensorMap* m, const void* p, uint64_t rows, int heads, int size, uint64_t ld, bool by_head, uint32_t box_rows) {
         return by_head ? make_map_heads(m, p, rows, (uint64_t)heads, (uint64_t)size, ld, box_rows)
                        : make_map(m, p, rows, (uint64_t)heads * size, ld, 64, box_rows);
@@ -705,14 +736,14 @@ AIEN_API int aien_paged_attention_prefill_tc_values(
     for (int lv = 0; lv < 5; ++lv) {
         const uint32_t rows = (uint32_t)page_size << lv;
         if (rows > (uint32_t)PT_BN) { mk.m[lv] = mk.m[0]; mv.m[lv] = mv.m[0]; continue; }
-        if (!rows_of(&mk.m[lv], k_cache, (uint64_t)cache_rows, nkv, hd, k_cols, kh, rows) ||
-            !rows_of(&mv.m[lv], v_cache, (uint64_t)cache_rows, nv, hdv, v_cols, vh, rows))
+        if (!rows_of(&mk.m[lv], k_cache, (uint64_t)cache_rows, nkv, hd, kld, kh, rows) ||
+            !rows_of(&mv.m[lv], v_cache, (uint64_t)cache_rows, nv, hdv, vld, vh, rows))
             return AIEN_E_STATE;
     }
     // one copy for a whole block of 128 keys, when the pool has that many rows at all and heads are whole chunks
     int big_boxes = cache_rows >= PT_BN ? 1 : 0;
-    if (big_boxes && !kh) big_boxes = make_map_chunked(&mk.blk, k_cache, (uint64_t)cache_rows, k_cols, k_cols, PT_BN, (uint32_t)(hd / 64)) ? 1 : 0;
-    if (big_boxes && !vh) big_boxes = make_map_chunked(&mv.blk, v_cache, (uint64_t)cache_rows, v_cols, v_cols, PT_BN, (uint32_t)(hdv / 64)) ? 1 : 0;
+    if (big_boxes && !kh) big_boxes = make_map_chunked(&mk.blk, k_cache, (uint64_t)cache_rows, k_cols, kld, PT_BN, (uint32_t)(hd / 64)) ? 1 : 0;
+    if (big_boxes && !vh) big_boxes = make_map_chunked(&mv.blk, v_cache, (uint64_t)cache_rows, v_cols, vld, PT_BN, (uint32_t)(hdv / 64)) ? 1 : 0;
     if (!big_boxes || kh) mk.blk = mk.m[0];
     if (!big_boxes || vh) mv.blk = mv.m[0];
 #define PT_CASE(HDV_, HVV_)                                                                                                        \
@@ -734,7 +765,7 @@ AIEN_API int aien_paged_attention_prefill_tc_terms(
     return aien_paged_attention_prefill_tc_values(q, q_stride, q_rows, k_cache, v_cache, cache_rows, block_table, max_blocks, q_start, ctx_len,
                                                   tile_seq, tile_q0, num_tiles, out, out_stride, nq, nkv, hd, page_size, window, scale,
                                                   scratch, scratch_bytes, max_ctx, force_splits, chunk, sinks, head_scale, slopes, gate, ldg,
-                                                  softcap, hd, 1, 0, stream);
+                                                  softcap, hd, 1, 0, 0, 0, nullptr, 0, stream);
 }
 
 AIEN_API int aien_paged_attention_prefill_tc_masked(

@@ -56,7 +56,7 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
                            const int* __restrict__ block_table, int max_blocks, const int* __restrict__ q_start,
                            const int* __restrict__ positions, int S, __nv_bfloat16* __restrict__ out,
                            int H, int r_lat, int rd, int page_size, int window, float scale_log2e, const float* __restrict__ sinks,
-                           int ksplit, float* __restrict__ part_o, float* __restrict__ part_ml) {
+                           int ksplit, float* __restrict__ part_o, float* __restrict__ part_ml, int single_only) {
     constexpr int BM = SLABS * 16, PARTS = WARPS / SLABS, KP = LX_BN / PARTS, NJ = KP / 8, CHP = R / PARTS, THREADS = WARPS * 32;
     constexpr int DT = CHP / 8;                  // n8 tiles of this warp's share of the channels
     static_assert(DT >= 2 && DT % 2 == 0, "a warp's share of the latent must be whole pairs of n8 tiles");
@@ -72,12 +72,14 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
     const uint32_t Ps_u = (uint32_t)__cvta_generic_to_shared(Ps);
 
     // which request, which rows
-    int s = -1, row0 = 0, acc = 0;
+    int s = -1, row0 = 0, acc = 0, unit = 0;             // unit: how many served tokens come before a single one
     for (int i = 0; i < S; ++i) {
-        const int tiles = ((q_start[i + 1] - q_start[i]) * H + BM - 1) / BM;
+        const int n = q_start[i + 1] - q_start[i];
+        const int tiles = single_only && n != 1 ? 0 : (n * H + BM - 1) / BM;         // single_only: portions are served elsewhere
         if ((int)blockIdx.x < acc + tiles) {
             s = i;
             row0 = ((int)blockIdx.x - acc) * BM;
+            unit = acc / tiles;
             break;
         }
         acc += tiles;
@@ -251,7 +253,7 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
         for (int r = 0; r < 2; ++r) {
             const int row = r == 0 ? ra : rb;
             if (row >= nrows) continue;
-            const size_t slot = ((size_t)qs * H + row0 + row) * ksplit + blockIdx.y;
+            const size_t slot = ((size_t)(single_only ? unit : qs) * H + row0 + row) * ksplit + blockIdx.y;
             if (half == 0 && c == 0) {
                 part_ml[slot * 2] = m_run[r];
                 part_ml[slot * 2 + 1] = l_run[r];
@@ -296,45 +298,68 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
     }
 }
 
-// out[row] = sum_s 2^(m_s - M) o_s / (sum_s 2^(m_s - M) l_s + 2^(sink - M)), M = max over the row's parts and the sink
-__global__ void latent_attention_merge_kernel(int R, const float* __restrict__ part_o, const float* __restrict__ part_ml, int ksplit,
-                                              const float* __restrict__ sinks, int H, __nv_bfloat16* __restrict__ out) {
-    const size_t row = blockIdx.x;
-    const float sk = sinks != nullptr ? sinks[row % H] * 1.4426950408889634f : -INFINITY;
+// out[row] = sum_s 2^(m_s - M) o_s / (sum_s 2^(m_s - M) l_s + 2^(sink - M)), M = max over the row's parts and the sink.
+// One CTA per (token, head) row; tokens (may be null): the tokens served.  The weights of the parts are made once, in shared
+// memory; the sums run over the parts in order, eight requested at a time.
+constexpr int LX_MAX_SPLIT = 512;
+__global__ void __launch_bounds__(128)
+latent_attention_merge_kernel(int R, const float* __restrict__ part_o, const float* __restrict__ part_ml, int ksplit,
+                              const float* __restrict__ sinks, int H, __nv_bfloat16* __restrict__ out, const int* __restrict__ tokens) {
+    __shared__ float wt[LX_MAX_SPLIT];
+    __shared__ float red[32];
+    const int unit = blockIdx.x / H, h = blockIdx.x - unit * H;
+    const size_t row = blockIdx.x, to = (size_t)(tokens != nullptr ? tokens[unit] : unit) * H + h;
+    const float sk = sinks != nullptr ? sinks[h] * 1.4426950408889634f : -INFINITY;
     float M = sk;
-    for (int s = 0; s < ksplit; ++s) M = fmaxf(M, part_ml[(row * ksplit + s) * 2]);
-    float den = (sinks != nullptr && M != -INFINITY) ? exp2f(sk - M) : 0.f;
-    for (int s = 0; s < ksplit; ++s) {
+    for (int s = threadIdx.x; s < ksplit; s += 128) M = fmaxf(M, part_ml[(row * ksplit + s) * 2]);
+    M = block_max(M, red);
+    float den = 0.f;
+    for (int s = threadIdx.x; s < ksplit; s += 128) {
         const float m = part_ml[(row * ksplit + s) * 2];
-        if (m != -INFINITY) den += exp2f(m - M) * part_ml[(row * ksplit + s) * 2 + 1];
+        const float w = m != -INFINITY ? exp2f(m - M) : 0.f;
+        wt[s] = w;
+        den += w * part_ml[(row * ksplit + s) * 2 + 1];
     }
+    den = block_sum(den, red);                                             // its barriers also order the weights
+    if (sinks != nullptr && M != -INFINITY) den += exp2f(sk - M);
     const float inv = den > 0.f ? 1.0f / den : 0.f;
-    for (int ch = threadIdx.x; ch < R; ch += blockDim.x) {
-        float acc = 0.f;
-        for (int s = 0; s < ksplit; ++s) {
-            const float m = part_ml[(row * ksplit + s) * 2];
-            if (m != -INFINITY) acc += exp2f(m - M) * part_o[(row * ksplit + s) * R + ch];
+    for (int ch = threadIdx.x * 2; ch < R; ch += 256) {                    // R is a multiple of 8
+        const float* src = part_o + row * ksplit * R + ch;
+        float2 acc = make_float2(0.f, 0.f);
+        for (int s0 = 0; s0 < ksplit; s0 += 8) {
+            float2 v[8];
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+                v[u] = s0 + u < ksplit && wt[s0 + u] != 0.f ? *reinterpret_cast<const float2*>(src + (size_t)(s0 + u) * R) : make_float2(0.f, 0.f);
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                const float w = s0 + u < ksplit ? wt[s0 + u] : 0.f;
+                acc.x = fmaf(w, v[u].x, acc.x);
+                acc.y = fmaf(w, v[u].y, acc.y);
+            }
         }
-        out[row * R + ch] = __float2bfloat16_rn(acc * inv);
+        *reinterpret_cast<uint32_t*>(out + to * R + ch) = lx_pack(acc.x * inv, acc.y * inv);
     }
 }
 
 template <int R, int SLABS, int WARPS>
 static int launch_latent_tc(const void* q, const void* cache, const int* bt, int max_blocks, const int* q_start, const int* positions,
                             int T, int S, void* out, int H, int r_lat, int rd, int page_size, int window, float scale, const float* sinks,
-                            int ksplit, float* part_o, float* part_ml, cudaStream_t stream) {
+                            int ksplit, float* part_o, float* part_ml, const int* tokens, int num_tokens, cudaStream_t stream) {
     const int D = r_lat + rd;
     constexpr int BM = SLABS * 16;
     const size_t smem = (size_t)(BM + LX_BN) * (lx_row_width(R, D) + 8) * 2 + (size_t)BM * LX_PSTR * 2 + (size_t)WARPS * 16 * sizeof(float);
     if (smem > 227 * 1024) return AIEN_E_SHAPE;
     auto kern = latent_attention_tc_kernel<R, SLABS, WARPS>;
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return AIEN_E_STATE;
-    const long tiles = ((long)T * H) / BM + S;
+    // tokens: only these, each a request's one token of the step
+    const long tiles = tokens != nullptr ? (long)num_tokens * ((H + BM - 1) / BM) : ((long)T * H) / BM + S;
     kern<<<dim3((unsigned)tiles, ksplit), WARPS * 32, smem, stream>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, bt, max_blocks, q_start,
                                                                      positions, S, (__nv_bfloat16*)out, H, r_lat, rd, page_size, window,
-                                                                     scale * 1.4426950408889634f, sinks, ksplit, part_o, part_ml);
+                                                                     scale * 1.4426950408889634f, sinks, ksplit, part_o, part_ml, tokens != nullptr ? 1 : 0);
     if (ksplit > 1)
-        latent_attention_merge_kernel<<<dim3((unsigned)((long)T * H)), 128, 0, stream>>>(r_lat, part_o, part_ml, ksplit, sinks, H, (__nv_bfloat16*)out);
+        latent_attention_merge_kernel<<<dim3((unsigned)((long)(tokens != nullptr ? num_tokens : T) * H)), 128, 0, stream>>>(
+            r_lat, part_o, part_ml, ksplit, sinks, H, (__nv_bfloat16*)out, tokens);
     return launch_status();
 }
 
@@ -344,13 +369,15 @@ static int launch_latent_tc(const void* q, const void* cache, const int* bt, int
 // four warps, k in steps of 64 through shared memory (cp.async), mma.sync.m16n8k16 with float32 accumulation.
 constexpr int HT_BM = 64, HT_BN = 64, HT_BK = 64, HT_STR = HT_BK + 8;
 
+// Two stages of k-steps: the next one's pieces are requested before the products of this one.  rows (or null): A's and C's rows
+// are those that it lists, M of them.
 template <typename TC>
 __global__ void __launch_bounds__(128)
 head_project_tc_kernel(const __nv_bfloat16* __restrict__ A, long lda, long a_head, const __nv_bfloat16* __restrict__ W, long w_head,
-                       TC* __restrict__ C, long ldc, long c_head, int M, int N, int K, const void* __restrict__ gate, int gdt, long ldg, int gate_n) {
-    __shared__ __align__(16) __nv_bfloat16 As[HT_BM * HT_STR];
-    __shared__ __align__(16) __nv_bfloat16 Ws[HT_BN * HT_STR];
-    const uint32_t As_u = (uint32_t)__cvta_generic_to_shared(As), Ws_u = (uint32_t)__cvta_generic_to_shared(Ws);
+                       TC* __restrict__ C, long ldc, long c_head, int M, int N, int K, const void* __restrict__ gate, int gdt, long ldg, int gate_n,
+                       const int* __restrict__ rows) {
+    __shared__ __align__(16) __nv_bfloat16 As[2][HT_BM * HT_STR];
+    __shared__ __align__(16) __nv_bfloat16 Ws[2][HT_BN * HT_STR];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int mh = warp & 1, nh = warp >> 1, g = lane >> 2, c = lane & 3;
     const int m0 = blockIdx.y * HT_BM, n0 = blockIdx.x * HT_BN, h = blockIdx.z;
@@ -362,17 +389,28 @@ head_project_tc_kernel(const __nv_bfloat16* __restrict__ A, long lda, long a_hea
     for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
-    for (int k0 = 0; k0 < K; k0 += HT_BK) {
+    auto fetch = [&](int k0, int st) {
+        const uint32_t As_u = (uint32_t)__cvta_generic_to_shared(As[st]), Ws_u = (uint32_t)__cvta_generic_to_shared(Ws[st]);
         for (int idx = tid; idx < HT_BM * (HT_BK / 8); idx += 128) {
             const int r = idx >> 3, ch = idx & 7;
             const bool kin = k0 + ch * 8 < K;
             const bool va = kin && m0 + r < M, vw = kin && n0 + r < N;
-            lx_cp_async16(As_u + (uint32_t)(r * HT_STR + ch * 8) * 2, A + (size_t)(va ? m0 + r : 0) * lda + (va ? k0 + ch * 8 : 0), va);
+            const size_t ar = va ? (size_t)(rows != nullptr ? rows[m0 + r] : m0 + r) : 0;
+            lx_cp_async16(As_u + (uint32_t)(r * HT_STR + ch * 8) * 2, A + ar * lda + (va ? k0 + ch * 8 : 0), va);
             lx_cp_async16(Ws_u + (uint32_t)(r * HT_STR + ch * 8) * 2, W + (size_t)(vw ? n0 + r : 0) * K + (vw ? k0 + ch * 8 : 0), vw);
         }
         lx_cp_async_commit();
-        lx_cp_async_wait_all();
+    };
+    fetch(0, 0);
+    for (int k0 = 0, st = 0; k0 < K; k0 += HT_BK, st ^= 1) {
+        if (k0 + HT_BK < K) {
+            fetch(k0 + HT_BK, st ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            lx_cp_async_wait_all();
+        }
         __syncthreads();
+        const uint32_t As_u = (uint32_t)__cvta_generic_to_shared(As[st]), Ws_u = (uint32_t)__cvta_generic_to_shared(Ws[st]);
 #pragma unroll
         for (int kk = 0; kk < HT_BK / 16; ++kk) {
             uint32_t a[2][4];
@@ -394,25 +432,72 @@ head_project_tc_kernel(const __nv_bfloat16* __restrict__ A, long lda, long a_hea
         }
         __syncthreads();
     }
-    float gs[2][2];                                              // sigmoid of the head's gate, for this thread's four rows
+    const bool pairs = ((N | ldc | c_head) & 1) == 0 && ((uintptr_t)C & (2 * sizeof(TC) - 1)) == 0;     // two neighbouring columns at a time
 #pragma unroll
     for (int mt = 0; mt < 2; ++mt)
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
-            const int m = m0 + mh * 32 + mt * 16 + g + r * 8;
-            gs[mt][r] = (gate != nullptr && gate_n == 0 && m < M) ? 1.0f / (1.0f + expf(-load_dyn(gate, gdt, (size_t)m * ldg + h))) : 1.0f;
-        }
+            const int ml = m0 + mh * 32 + mt * 16 + g + r * 8;
+            if (ml >= M) continue;
+            const size_t m = (size_t)(rows != nullptr ? rows[ml] : ml);
+            const float gs = (gate != nullptr && gate_n == 0) ? 1.0f / (1.0f + expf(-load_dyn(gate, gdt, m * ldg + h))) : 1.0f;
 #pragma unroll
-    for (int mt = 0; mt < 2; ++mt)
+            for (int j = 0; j < 4; ++j) {
+                const int n = n0 + nh * 32 + j * 8 + 2 * c;
+                float v[2] = {acc[mt][j][2 * r] * gs, acc[mt][j][2 * r + 1] * gs};
+                if (gate_n > 0) {
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int m = m0 + mh * 32 + mt * 16 + g + (e >> 1) * 8, n = n0 + nh * 32 + j * 8 + 2 * c + (e & 1);
-                if (m >= M || n >= N) continue;
-                const float ge = gate_n > 0 ? __fdividef(1.0f, 1.0f + __expf(-load_dyn(gate, gdt, (size_t)m * ldg + (size_t)h * gate_n + n))) : gs[mt][e >> 1];
-                C[(size_t)m * ldc + n] = from_f<TC>(acc[mt][j][e] * ge);
+                    for (int e = 0; e < 2; ++e)
+                        if (n + e < N) v[e] *= __fdividef(1.0f, 1.0f + __expf(-load_dyn(gate, gdt, m * ldg + (size_t)h * gate_n + n + e)));
+                }
+                TC* dst = C + m * ldc + n;
+                if (pairs && n + 1 < N) {
+                    if constexpr (sizeof(TC) == 2) *reinterpret_cast<uint32_t*>(dst) = lx_pack(v[0], v[1]);
+                    else *reinterpret_cast<float2*>(dst) = make_float2(v[0], v[1]);
+                } else {
+                    if (n < N) dst[0] = from_f<TC>(v[0]);
+                    if (n + 1 < N) dst[1] = from_f<TC>(v[1]);
+                }
             }
+        }
+}
+
+// ---------------------------------------------------------------- the latents of portions, for keys and values per head
+// Portion p of the step (the p-th request that brings more than one token) gets rows p * len .. of `out`: its cached latents at
+// positions 0 .. ctx_len - 1, then zeros.  table [S, len / 128]: the 128-row pages of those rows, in order, for requests
+// with a portion.  One CTA per 32 rows; a warp finds the portion's request, then each of the eight copies rows.
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, int r_lat, const int* __restrict__ block_table, int max_blocks, int page_size,
+                     const int* __restrict__ q_start, const int* __restrict__ ctx_len, int S, int len, __nv_bfloat16* __restrict__ out,
+                     int* __restrict__ table) {
+    __shared__ int s_req;
+    const int p = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    if (tid == 0) s_req = -1;
+    __syncthreads();
+    if (warp == 0) {
+        int before = 0;
+        for (int base = 0; base < S; base += 32) {
+            const int i = base + lane;
+            const bool has = i < S && q_start[i + 1] - q_start[i] > 1;
+            const uint32_t mask = __ballot_sync(0xffffffffu, has);
+            if (has && before + __popc(mask & ((1u << lane) - 1u)) == p) s_req = i;
+            before += __popc(mask);
+        }
+    }
+    __syncthreads();
+    const int s = s_req, n = s >= 0 ? ctx_len[s] : 0;
+    if (s >= 0 && blockIdx.x == 0)
+        for (int b = tid; b < len / 128; b += 256) table[(size_t)s * (len / 128) + b] = p * (len / 128) + b;
+    const int* bt = s >= 0 ? block_table + (size_t)s * max_blocks : nullptr;
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+        const int key = blockIdx.x * 32 + warp * 4 + u;
+        if (key >= len) return;
+        const int page = key < n ? bt[key / page_size] : -1;
+        const uint4* src = reinterpret_cast<const uint4*>(cache + ((size_t)(page >= 0 ? page : 0) * page_size + key % page_size) * r_lat);
+        uint4* dst = reinterpret_cast<uint4*>(out + ((size_t)p * len + key) * r_lat);
+        for (int i = lane; i < r_lat / 8; i += 32) dst[i] = page >= 0 ? src[i] : make_uint4(0u, 0u, 0u, 0u);
+    }
 }
 
 }  // namespace aien
@@ -431,20 +516,21 @@ AIEN_API int aien_latent_attention_tc_supports(int kv_rank, int rot_dim) {
 // The step's T tokens are the portions q_start[s] .. q_start[s + 1] of S requests; positions[t] is token t's position.
 // ksplit > 1: the key blocks of every tile are dealt out to ksplit CTAs (for steps with few tiles); part_o (float32,
 // T * H * ksplit * kv_rank) and part_ml (float32, T * H * ksplit * 2) hold their partial results for the merging launch.
+// tokens (may be null), num_tokens: serve only these tokens, each the one token that its request brings (a mixed step's).
 // small_tiles != 0: tiles of 16 rows instead of 64 (steps in which every request brings one token), for latents of more than 64.
 AIEN_API int aien_latent_attention_tc(const void* q, const void* cache, const int* block_table, int max_blocks, const int* q_start,
                                       const int* positions, void* out, int T, int S, int H, int kv_rank, int rot_dim, int page_size,
                                       int window, float scale, const float* sinks, int ksplit, float* part_o, float* part_ml,
-                                      int small_tiles, cudaStream_t stream) {
+                                      int small_tiles, const int* tokens, int num_tokens, cudaStream_t stream) {
     if (T <= 0 || S <= 0) return 0;
     if (H <= 0 || page_size <= 0 || window < 0 || !aien_latent_attention_tc_supports(kv_rank, rot_dim)) return AIEN_E_SHAPE;
     if (((uintptr_t)q & 15) || ((uintptr_t)cache & 15) || ((uintptr_t)out & 3)) return AIEN_E_ALIGN;
-    if (ksplit < 1 || ksplit > 65535 || (ksplit > 1 && (part_o == nullptr || part_ml == nullptr || ((uintptr_t)part_o & 7)))) return AIEN_E_SHAPE;
+    if (ksplit < 1 || ksplit > LX_MAX_SPLIT || num_tokens < 0 || (tokens != nullptr && num_tokens == 0) || (ksplit > 1 && (part_o == nullptr || part_ml == nullptr || ((uintptr_t)part_o & 7)))) return AIEN_E_SHAPE;
     const int padded = lx_padded_rank(kv_rank);
 #define LX_CASE(RV, SL)                                                                                                          \
     if (padded == RV)                                                                                                            \
         return launch_latent_tc<RV, SL, (SL == 4 ? 16 : 8)>(q, cache, block_table, max_blocks, q_start, positions, T, S, out, H, kv_rank, rot_dim, page_size,  \
-                                        window, scale, sinks, ksplit, part_o, part_ml, stream);
+                                        window, scale, sinks, ksplit, part_o, part_ml, tokens, num_tokens, stream);
     if (small_tiles && padded >= 128) {                    // tiles of 16 rows: a latent of 64 would leave a warp half a pair of n8 tiles
         LX_CASE(128, 1) LX_CASE(256, 1) LX_CASE(512, 1)
     }
@@ -456,13 +542,26 @@ AIEN_API int aien_latent_attention_tc(const void* q, const void* cache, const in
 // A bfloat16 [M, lda] (head h at column h * a_head), W bfloat16 [heads, N, K], C [M, ldc] (head h at column h * c_head).
 // K, lda and a_head multiples of 8, A and W 16-byte aligned.
 AIEN_API int aien_head_project_tc(const void* A, long lda, long a_head, const void* W, void* C, int c_dt, long ldc, long c_head,
-                                  int M, int N, int K, int heads, const void* gate, int gate_dt, long ldg, int gate_n, cudaStream_t stream) {
+                                  int M, int N, int K, int heads, const void* gate, int gate_dt, long ldg, int gate_n, const int* rows,
+                                  cudaStream_t stream) {
     if (M <= 0 || N <= 0 || heads <= 0) return 0;
     if (K <= 0 || heads > 65535 || gate_n < 0 || (gate_n > 0 && (gate == nullptr || gate_n != N))) return AIEN_E_SHAPE;
     if ((K & 7) || (lda & 7) || (a_head & 7) || ((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return AIEN_E_ALIGN;
     dim3 grid((N + HT_BN - 1) / HT_BN, (M + HT_BM - 1) / HT_BM, heads);
     if (grid.y > 65535) return AIEN_E_SHAPE;
     AIEN_DISPATCH_DTYPE(c_dt, TC, (head_project_tc_kernel<TC><<<grid, 128, 0, stream>>>((const __nv_bfloat16*)A, lda, a_head, (const __nv_bfloat16*)W,
-                                                                                     (long)N * K, (TC*)C, ldc, c_head, M, N, K, gate, gate_dt, ldg, gate_n)));
+                                                                                     (long)N * K, (TC*)C, ldc, c_head, M, N, K, gate, gate_dt, ldg, gate_n, rows)));
+    return launch_status();
+}
+
+// cache bfloat16 [slots, r_lat]; out bfloat16 [portions * len, r_lat]; table int32 [S, len / 128]; len a multiple of 128 that
+// covers every portion's context; r_lat a multiple of 8.
+AIEN_API int aien_latent_gather(const void* cache, int r_lat, const int* block_table, int max_blocks, int page_size, const int* q_start,
+                                const int* ctx_len, int S, int portions, int len, void* out, int* table, cudaStream_t stream) {
+    if (portions <= 0 || S <= 0) return 0;
+    if (r_lat <= 0 || (r_lat & 7) || page_size <= 0 || len <= 0 || (len & 127) || portions > 65535) return AIEN_E_SHAPE;
+    if (((uintptr_t)cache & 15) || ((uintptr_t)out & 15)) return AIEN_E_ALIGN;
+    latent_gather_kernel<<<dim3(len / 32, portions), 256, 0, stream>>>((const __nv_bfloat16*)cache, r_lat, block_table, max_blocks, page_size, q_start,
+                                                                      ctx_len, S, len, (__nv_bfloat16*)out, table);
     return launch_status();
 }

@@ -167,8 +167,9 @@ def _declare(l: ctypes.CDLL) -> None:
         "aien_decay_linear_attention_chunked": [P, I, L, I, I, I, P, P, P, P, P, P, L, P, I, I, I, I, I, P],
         "aien_latent_prepare": [P, I, L, I, P, P, I, F, P, I, L, I, I, I, I, P, P, P, P, I, I, P],
         "aien_rotate_pairs_rows": [P, I, L, L, P, I, L, L, I, I, I, I, P, P, P],
-        "aien_latent_attention_tc": [P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, P, I, P, P, I, P],
-        "aien_head_project_tc": [P, L, L, P, P, I, L, L, I, I, I, I, P, I, L, I, P],
+        "aien_latent_attention_tc": [P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, P, I, P, P, I, P, I, P],
+        "aien_latent_gather": [P, I, P, I, I, P, P, I, I, I, P, P, P],
+        "aien_head_project_tc": [P, L, L, P, P, I, L, L, I, I, I, I, P, I, L, I, P, P],
         "aien_latent_attention_tc_supports": [I, I],
         "aien_head_project": [P, I, L, L, P, I, L, L, P, I, L, L, I, I, I, I, P, I, L, I, P],
         "aien_latent_attention": [P, L, P, I, P, I, P, P, P, P, I, L, I, I, I, I, I, I, F, P, P],
@@ -209,7 +210,7 @@ def _declare(l: ctypes.CDLL) -> None:
         "aien_rope_halves_value_write": [P, I, L, I, c_size_t, P, I, I, I, I, I, I, I, I, P, P, I, P, P, I, L, P, P, I, I, P],
         "aien_map_difference_norm": [P, L, P, I, L, I, I, I, I, F, F, F, P],
         "aien_paged_attention_decode_values": [P, L, P, P, P, I, P, P, P, P, L, P, P, P, I, I, I, I, I, F, I, I, I, F, I, I, I, I, P],
-        "aien_paged_attention_prefill_tc_values": [P, L, I, P, P, I, P, I, P, P, P, P, I, P, L, I, I, I, I, I, F, P, L, I, I, I, P, P, P, P, L, F, I, I, I, P],
+        "aien_paged_attention_prefill_tc_values": [P, L, I, P, P, I, P, I, P, P, P, P, I, P, L, I, I, I, I, I, F, P, L, I, I, I, P, P, P, P, L, F, I, I, I, L, L, P, L, P],
         "aien_paged_attention_prefill_tc_values_supports": [I, I, I],
     }
     for name, args in sigs.items():
@@ -1452,10 +1453,11 @@ def rotate_pairs_rows(q: torch.Tensor, q_head: int, col0: int, out: torch.Tensor
 
 
 def head_project(a: torch.Tensor, a_head: int, a_col0: int, w: torch.Tensor, out: torch.Tensor, o_head: int, o_col0: int,
-                 gate: Optional[torch.Tensor] = None) -> None:
+                 gate: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, num_rows: int = 0) -> None:
     """out[t, h*o_head + o_col0 + n] = sum_k a[t, h*a_head + a_col0 + k] * w[h, n, k]: one product per head, w [heads, N, K].
     ``gate`` (row stride free): [T, heads], the result of head h is multiplied by sigmoid(gate[t, h]); or [T, heads*N],
-    element n of head h by sigmoid(gate[t, h*N + n]).
+    element n of head h by sigmoid(gate[t, h*N + n]).  ``rows`` (int32) with ``num_rows``: only these rows t are served (the
+    tensor-core form only; the caller has seen to :func:`latent_attention_tc_supports`).
     bfloat16 operands whose rows are whole aligned 16-byte pieces run on the tensor cores, everything else on the CUDA cores;
     both sum in float32."""
     _dev(a, w, out)
@@ -1470,9 +1472,12 @@ def head_project(a: torch.Tensor, a_head: int, a_col0: int, w: torch.Tensor, out
     av, ov = a[:, a_col0:], out[:, o_col0:]
     if (_LATENT_IMPL != "plain" and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and K_ % 8 == 0 and a.stride(0) % 8 == 0
             and a_head % 8 == 0 and av.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
-        _check(lib().aien_head_project_tc(_p(av), a.stride(0), int(a_head), _p(w), _p(ov), dt(out), out.stride(0), int(o_head), M, N, K_,
-                                          heads, gp, gdt, ldg, gate_n, _stream()), "head_project_tc")
+        _check(lib().aien_head_project_tc(_p(av), a.stride(0), int(a_head), _p(w), _p(ov), dt(out), out.stride(0), int(o_head),
+                                          M if rows is None else int(num_rows), N, K_, heads, gp, gdt, ldg, gate_n, _p(rows), _stream()),
+               "head_project_tc")
         return
+    if rows is not None:
+        raise KernelError("head_project: only the tensor-core form takes a list of rows")
     _check(lib().aien_head_project(_p(av), dt(a), a.stride(0), int(a_head), _p(w), dt(w), K_, N * K_, _p(ov), dt(out), out.stride(0),
                                    int(o_head), M, N, K_, heads, gp, gdt, ldg, gate_n, _stream()), "head_project")
 
@@ -1505,13 +1510,15 @@ def latent_attention_tc_supports(dtype: torch.dtype, kv_rank: int, rot_dim: int)
 def latent_attention_tc(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, max_blocks: int, q_start: torch.Tensor,
                         positions: torch.Tensor, out: torch.Tensor, num_seqs: int, heads: int, kv_rank: int, rot_dim: int,
                         page_size: int, window: int, scale: float, sinks: Optional[torch.Tensor], ksplit: int = 1,
-                        scratch: Optional[torch.Tensor] = None, small_tiles: bool = False) -> None:
+                        scratch: Optional[torch.Tensor] = None, small_tiles: bool = False, tokens: Optional[torch.Tensor] = None,
+                        num_single: int = 0) -> None:
     """latent_attention on the tensor cores.  q bfloat16 [T, heads*(kv_rank + rot_dim)] and out bfloat16 [T, heads*kv_rank],
     both contiguous; the T tokens are the portions q_start[s]..q_start[s+1] of ``num_seqs`` requests (row s of the block
     table), each portion's positions counting up from positions[q_start[s]].  ``ksplit`` > 1 deals the key blocks of every
     tile out to that many CTAs and merges their results in a second launch (steps with few tiles); ``scratch`` is then
     float32 with ``latent_attention_tc_scratch(T, heads, kv_rank, ksplit)`` numbers.  ``small_tiles``: tiles of 16 rows
-    instead of 64, for steps in which every request brings one token (latents of more than 64)."""
+    instead of 64, for steps in which every request brings one token (latents of more than 64).  ``tokens`` (int32) with
+    ``num_single``: only these tokens are served, those that their requests bring alone."""
     _dev(q, cache, block_table, q_start, positions, out, sinks)
     T, D = q.shape[0], kv_rank + rot_dim
     assert q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
@@ -1522,14 +1529,15 @@ def latent_attention_tc(q: torch.Tensor, cache: torch.Tensor, block_table: torch
     part_o = part_ml = None
     if ksplit > 1:
         _dev(scratch)
-        n_o = T * heads * ksplit * kv_rank
+        count = T if tokens is None else int(num_single)
+        n_o = count * heads * ksplit * kv_rank
         assert scratch is not None and scratch.dtype == torch.float32 and scratch.is_contiguous()
-        assert scratch.numel() >= latent_attention_tc_scratch(T, heads, kv_rank, ksplit)
+        assert scratch.numel() >= latent_attention_tc_scratch(count, heads, kv_rank, ksplit)
         part_o, part_ml = scratch[:n_o], scratch[n_o:]
     _check(lib().aien_latent_attention_tc(_p(q), _p(cache), _p(block_table), int(max_blocks), _p(q_start), _p(positions), _p(out), T,
                                           int(num_seqs), int(heads), int(kv_rank), int(rot_dim), int(page_size), int(window),
-                                          float(scale), _p(sinks), int(ksplit), _p(part_o), _p(part_ml), 1 if small_tiles else 0, _stream()),
-           "latent_attention_tc")
+                                          float(scale), _p(sinks), int(ksplit), _p(part_o), _p(part_ml), 1 if small_tiles else 0, _p(tokens),
+                                          int(num_single), _stream()), "latent_attention_tc")
 
 
 LATENT_TC_TILE = 64          # (token, head) rows and keys per tile of the tensor-core kernel
@@ -1551,6 +1559,67 @@ def latent_attention_tc_ksplit(num_tokens: int, num_seqs: int, heads: int, max_c
     span = min(window, max_ctx) if window > 0 else max_ctx
     blocks = max(1, (span + LATENT_TC_TILE - 1) // LATENT_TC_TILE + 1)
     return max(1, min(blocks, 296 // tiles)) if tiles <= 148 else 1
+
+
+# Portions of prompts may leave the latent: their contexts' keys and values are made per head by one product and attended
+# over by the tcgen05 kernel.  "": by estimated time; "expand" / "absorb" pin the choice.
+LATENT_PORTIONS = __import__("os").environ.get("AIEN_B200_LATENT_PORTIONS", "").strip().lower()
+LATENT_EXPAND_MAX_BYTES = 256 << 20        # room for the keys and values of a step
+
+
+def latent_expand_rows(max_ctx: int, portions: int) -> int:
+    """Rows of keys and values of a step's portions: whole tiles of 128 positions of the longest context, for each."""
+    return portions * ((max_ctx + 127) // 128) * 128
+
+
+def latent_expand_takes(num_tokens: int, portions: int, max_ctx: int, heads: int, head_dim: int, value_dim: int, kv_rank: int) -> bool:
+    """Whether the portions of a step take the expanded form: where it is possible, where it fits, and where it is the
+    faster one.  The estimate counts flops at the rates the kernels reach on one B200 (TFLOP/s: products 900, tcgen05
+    attention 300, attention over the latent 115, products per head 80) and 15 us for the two more launches; the choice
+    depends on the step's sizes alone."""
+    rows = latent_expand_rows(max_ctx, portions)
+    if (LATENT_PORTIONS == "absorb" or portions <= 0 or _PREFILL_IMPL != "tc" or _FORCE_ATTN == "generic" or _LATENT_IMPL == "plain"
+            or rows * heads * (head_dim + value_dim) * 2 > LATENT_EXPAND_MAX_BYTES
+            or not lib().aien_paged_attention_prefill_tc_values_supports(head_dim, value_dim, 128)):
+        return False
+    if LATENT_PORTIONS == "expand":
+        return True
+    pairs = num_tokens * max_ctx * 0.75 * heads
+    both = 2 * (head_dim + value_dim)
+    expand = rows * heads * both * kv_rank / 900e6 + pairs * both / 300e6 + 15.0
+    absorb = pairs * 4 * kv_rank / 115e6 + num_tokens * heads * both * kv_rank / 80e6
+    return expand < absorb
+
+
+def latent_gather(cache: torch.Tensor, group, q_start: torch.Tensor, ctx_len: torch.Tensor, num_seqs: int, portions: int, length: int,
+                  out: torch.Tensor, table: torch.Tensor) -> None:
+    """The cached latents of the requests that bring several tokens, one after the other in ``out`` [portions * length,
+    kv_rank] (rows beyond a context are zeros); ``table`` int32 [num_seqs, length / 128]: the 128-row pages of a request's rows."""
+    _dev(cache, group.block_table, q_start, ctx_len, out, table)
+    assert cache.dtype == torch.bfloat16 and cache.is_contiguous() and out.is_contiguous() and tuple(out.shape) == (portions * length, cache.shape[-1])
+    assert length % 128 == 0 and table.dtype == torch.int32 and tuple(table.shape) == (num_seqs, length // 128)
+    _check(lib().aien_latent_gather(_p(cache), cache.shape[-1], _p(group.block_table), group.max_blocks, group.page_size, _p(q_start),
+                                    _p(ctx_len), int(num_seqs), int(portions), int(length), _p(out), _p(table), _stream()), "latent_gather")
+
+
+def portion_attention(ctx, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, table: torch.Tensor, out: torch.Tensor, heads: int,
+                      head_dim: int, value_dim: int, window: int, scale: float, sinks: Optional[torch.Tensor] = None,
+                      head_gate: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+    """Causal attention of the step's portions (not of its single tokens) over keys and values that lie in rows of their own:
+    k [rows, heads*head_dim] and v [rows, heads*value_dim] bfloat16 with free row strides, in 128-row pages named by ``table``
+    [S, pages].  q [T, heads*head_dim] (row stride free), out bfloat16 [T, heads*value_dim].  ``head_gate`` float32 [T, heads]:
+    head h's output times sigmoid(head_gate[t, h]); ``gate`` bfloat16 [T, heads*value_dim]: element by element."""
+    _dev(q, k, v, table, out, sinks, head_gate, gate)
+    tile_seq, tile_q0, n = ctx.prefill_tiles
+    assert q.dtype == k.dtype == v.dtype == out.dtype == torch.bfloat16 and q.stride(1) == k.stride(1) == v.stride(1) == out.stride(1) == 1
+    assert k.shape[0] == v.shape[0] and k.shape[1] == heads * head_dim and v.shape[1] == heads * value_dim
+    assert gate is None or (gate.dtype == torch.bfloat16 and gate.stride(1) == 1 and gate.shape[1] == heads * value_dim)
+    _check_head_terms(heads, None, None, head_gate)
+    _check(lib().aien_paged_attention_prefill_tc_values(
+        _p(q), q.stride(0), q.shape[0], _p(k), _p(v), k.shape[0], _p(table), table.shape[1], _p(ctx.q_start), _p(ctx.ctx_len), _p(tile_seq),
+        _p(tile_q0), n, _p(out), out.stride(0), heads, heads, head_dim, 128, window, float(scale), None, 0, int(ctx.max_ctx_len), 0, 0,
+        _p(sinks), None, None, _p(head_gate), head_gate.stride(0) if head_gate is not None else 0, 0.0, value_dim, 1, 0, k.stride(0),
+        v.stride(0), _p(gate), gate.stride(0) if gate is not None else 0, _stream()), "paged_attention_prefill_tc_values")
 
 
 # ---------------------------------------------------------------------------- several residual streams, token shift
@@ -2008,7 +2077,7 @@ def capped_attention(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
                 _p(ctx.ctx_len), _p(tile_seq), _p(tile_q0), n, _p(out), out.stride(0), num_q_heads, num_kv_heads, head_dim,
                 group.page_size, window, float(scale), _p(scratch), scratch.numel() * 4 if scratch is not None else 0,
                 int(ctx.max_ctx_len), 0, int(chunk), None, None, None, None, 0, float(softcap or 0.0), value_dim, int(v_share),
-                1 if out.dtype == torch.float32 else 0, _stream()), "paged_attention_prefill_tc_values")
+                1 if out.dtype == torch.float32 else 0, 0, 0, None, 0, _stream()), "paged_attention_prefill_tc_values")
         tokens, nd = ctx.single_tokens if ctx.single_tokens is not None else (None, 0)
         if nd > 0 and splits_ok:
             single_tokens(tokens, nd)

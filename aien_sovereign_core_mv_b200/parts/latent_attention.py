@@ -22,9 +22,12 @@ class LatentAttention(Mixer):
     heads element by element times sigmoid(W_g h); W_o on the heads.  The rotation turns neighbouring pairs of the first
     ``rotary_dim`` numbers of the rotated part (the position part's table).
 
-    The cache keeps one row [c | k_rot] per token and nothing per head.  The kernels never build a head's keys or
-    values: W_uk is applied to the query (q_lat = W_uk,h^T q_unrot) and W_uv to the weighted sum of latents, so a cached
-    row serves every head as key and as value.  ``own_cache`` False: the layer has no W_dkv and attends over the rows
+    The cache keeps one row [c | k_rot] per token and nothing per head.  Two forms of the same sums read it.  *Absorbed*:
+    no head's keys or values are built; W_uk is applied to the query (q_lat = W_uk,h^T q_unrot) and W_uv to the weighted
+    sum of latents, so a cached row serves every head as key and as value.  *Expanded* (portions of prompts in a bfloat16
+    engine, without a rotated part): the contexts' keys and values are made per head by one product for the length of the
+    step, which costs less than carrying every score and sum at the latent's size as soon as a portion has more than
+    a few dozen tokens (``kernels.latent_expand_takes``); single tokens beside them take the absorbed form.  ``own_cache`` False: the layer has no W_dkv and attends over the rows
     another layer wrote (its run binding names that layer's planes).  ``cache_window``: how many positions the cache
     must keep, when layers that share it have different windows (default: ``window``)."""
 
@@ -56,6 +59,10 @@ class LatentAttention(Mixer):
         self.q_cols = self.q_rank or self.num_heads * self.q_head        # rows of the first product that belong to the query
         self.side_rows, self.riders = self.gate_rows, 0                  # and those behind them: gates, riders
         self.row = self.kv_rank + self.rot_dim
+        # the expanded form of portions (a bfloat16 engine's)
+        self._expandable = self.rot_dim == 0 and self.kv_rank % 8 == 0 and self.head_dim % 8 == 0 and self.value_dim % 8 == 0 \
+            and max(self.head_dim, self.value_dim) <= 128
+        self.w_kv = None
         self.w_down = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = self.dq_norm = self.dkv_norm = self.sinks = None
 
     # ---- tensors
@@ -97,6 +104,8 @@ class LatentAttention(Mixer):
         # per head [kv_rank, head_dim]: the matrix that takes a head's unrotated query to the latent
         self.w_uk_t = tensors["uk_proj"].view(n, self.head_dim, self.kv_rank).transpose(1, 2).contiguous()
         self.w_uv = tensors["uv_proj"].view(n, self.value_dim, self.kv_rank).contiguous()
+        if self._expandable and tensors["uk_proj"].dtype == torch.bfloat16 == tensors["uv_proj"].dtype:
+            self.w_kv = torch.cat([tensors["uk_proj"], tensors["uv_proj"]], dim=0).contiguous()      # all heads' keys | all heads' values
         self.dq_norm = tensors["dq_norm"].contiguous() if self.q_rank else None
         if self.own_cache:
             self.dkv_norm = tensors["dkv_norm"].contiguous()
@@ -116,9 +125,51 @@ class LatentAttention(Mixer):
         # the partial results of a step with few tiles: tokens * heads * ksplit rows, which latent_attention_tc_ksplit keeps
         # below 296 tiles' worth of 64 rows
         split = 296 * K.LATENT_TC_TILE * (self.kv_rank + 2) * 4
-        return lim.max_tokens * per_token + 16384 + split + K.PARTIALS_MAX_BYTES
+        expand = 0
+        if self._expandable and lim.itemsize == 2:
+            rows = K.latent_expand_rows(lim.max_context, lim.max_seqs)
+            per_row = n * (self.head_dim + self.value_dim) * 2
+            rows = min(rows, K.LATENT_EXPAND_MAX_BYTES // per_row + 128)
+            expand = rows * (per_row + self.kv_rank * 2) + lim.max_seqs * (lim.max_context // 128 + 2) * 4 + 4096
+        return lim.max_tokens * per_token + 16384 + split + K.PARTIALS_MAX_BYTES + expand
 
     # ---- one step
+    def _expanded(self, ctx, q, cache, group, portions, gate, o):
+        """The portions' rows of ``o``: keys and values per head for the length of the step."""
+        n, ws = self.num_heads, ctx.workspace
+        length = K.latent_expand_rows(ctx.max_ctx_len, 1)
+        lat = ws.take((portions * length, self.kv_rank), torch.bfloat16)
+        table = ws.take((ctx.num_seqs, length // 128), torch.int32)
+        K.latent_gather(cache, group, ctx.q_start, ctx.ctx_len, ctx.num_seqs, portions, length, lat, table)
+        kv = linear(ctx, lat, self.w_kv)
+        k, v = kv[:, :n * self.head_dim], kv[:, n * self.head_dim:]
+        by_head = gate if self.head_gate else None
+        element = gate if self.out_gate else None
+        K.portion_attention(ctx, q, k, v, table, o, n, self.head_dim, self.value_dim, self.window, self.scale, self.sinks, by_head, element)
+
+    def _absorbed(self, ctx, q, cache, group, tc, gate, o, rot, singles, n_single):
+        """Rows of ``o`` over the latent itself: all of the step's, or those of ``singles`` (tokens that come alone)."""
+        T, n, ws = ctx.num_tokens, self.num_heads, ctx.workspace
+        cos, sin, rdims = rot if rot is not None else (None, None, 0)
+        qf = ws.take((T, n * self.row), torch.bfloat16 if tc else torch.float32)    # per head: the query in the latent | rotated part
+        K.head_project(q, self.q_head, 0, self.w_uk_t, qf, self.row, 0, rows=singles, num_rows=n_single)
+        if self.rot_dim:
+            K.rotate_pairs_rows(q, self.q_head, self.head_dim, qf, self.row, self.kv_rank, n, self.rot_dim, rdims, cos, sin)
+        mixed = ws.take((T, n * self.kv_rank), ctx.dtype)
+        if tc:
+            alone = ctx.decode_only or singles is not None
+            small = K.latent_attention_tc_small_tiles(alone, self.kv_rank)
+            count = n_single if singles is not None else T
+            ksplit = K.latent_attention_tc_ksplit(count, n_single if singles is not None else ctx.num_seqs, n, ctx.max_ctx_len, self.window, small)
+            scratch = ws.take((K.latent_attention_tc_scratch(count, n, self.kv_rank, ksplit),), torch.float32) if ksplit > 1 else None
+            K.latent_attention_tc(qf, cache, group.block_table, group.max_blocks, ctx.q_start, ctx.positions, mixed, ctx.num_seqs, n,
+                                  self.kv_rank, self.rot_dim, group.page_size, self.window, self.scale, self.sinks, ksplit, scratch, small,
+                                  singles, n_single)
+        else:
+            K.latent_attention(qf, cache, group.block_table, group.max_blocks, ctx.seq_of_token, ctx.positions, mixed, n, self.kv_rank,
+                               self.rot_dim, group.page_size, self.window, self.scale, self.sinks)
+        K.head_project(mixed, self.kv_rank, 0, self.w_uv, o, self.value_dim, 0, gate=gate, rows=singles, num_rows=n_single)
+
     def forward(self, ctx: StepContext, h: torch.Tensor, run: RunBinding):
         T, n, ws = ctx.num_tokens, self.num_heads, ctx.workspace
         group = ctx.groups[run.group]
@@ -138,23 +189,19 @@ class LatentAttention(Mixer):
                          self.dkv_norm, cos, sin, group.slot_map if writes else None, cache if writes else None)
         # per head: unrotated | rotated part, before rotation; an operand of the tensor-core products where those run
         q = linear(ctx, cq, self.w_uq, out_dtype=torch.bfloat16 if tc else torch.float32) if self.q_rank else d
-        qf = ws.take((T, n * self.row), torch.bfloat16 if tc else torch.float32)    # per head: the query in the latent | rotated part
-        K.head_project(q, self.q_head, 0, self.w_uk_t, qf, self.row, 0)
-        if self.rot_dim:
-            K.rotate_pairs_rows(q, self.q_head, self.head_dim, qf, self.row, self.kv_rank, n, self.rot_dim, rdims, cos, sin)
-        mixed = ws.take((T, n * self.kv_rank), ctx.dtype)
-        if tc:
-            small = K.latent_attention_tc_small_tiles(ctx.decode_only, self.kv_rank)
-            ksplit = K.latent_attention_tc_ksplit(T, ctx.num_seqs, n, ctx.max_ctx_len, self.window, small)
-            scratch = ws.take((K.latent_attention_tc_scratch(T, n, self.kv_rank, ksplit),), torch.float32) if ksplit > 1 else None
-            K.latent_attention_tc(qf, cache, group.block_table, group.max_blocks, ctx.q_start, ctx.positions, mixed, ctx.num_seqs, n,
-                                  self.kv_rank, self.rot_dim, group.page_size, self.window, self.scale, self.sinks, ksplit, scratch, small)
-        else:
-            K.latent_attention(qf, cache, group.block_table, group.max_blocks, ctx.seq_of_token, ctx.positions, mixed, n, self.kv_rank,
-                               self.rot_dim, group.page_size, self.window, self.scale, self.sinks)
+        gate = d[:, self.q_cols:self.q_cols + self.gate_rows] if self.gate_rows else None
         o = ws.take((T, n * self.value_dim), ctx.dtype)
-        K.head_project(mixed, self.kv_rank, 0, self.w_uv, o, self.value_dim, 0,
-                       gate=d[:, self.q_cols:self.q_cols + self.gate_rows] if self.gate_rows else None)
+        tiles = ctx.prefill_tiles[2] if ctx.prefill_tiles is not None and not ctx.decode_only else 0
+        singles, n_single = ctx.single_tokens if ctx.single_tokens is not None else (None, 0)
+        portions = ctx.num_seqs - n_single if tiles > 0 else 0
+        gate_suits = gate is None or (gate.dtype == torch.float32 if self.head_gate else
+                                      gate.dtype == torch.bfloat16 and gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)
+        expand = tc and self.w_kv is not None and q.dtype == torch.bfloat16 and q.stride(0) % 8 == 0 and gate_suits and \
+            K.latent_expand_takes(T - n_single, portions, ctx.max_ctx_len, n, self.head_dim, self.value_dim, self.kv_rank)
+        if expand:
+            self._expanded(ctx, q[:, :n * self.q_head], cache, group, portions, gate, o)
+        if not expand or n_single > 0:
+            self._absorbed(ctx, q, cache, group, tc, gate, o, rot, singles if expand else None, n_single if expand else 0)
         y = linear(ctx, o, self.w_o, out_dtype=torch.float32, may_defer_sum=True)        # the consumer's norm adds partial products
         if not self.riders:
             return y

@@ -786,15 +786,15 @@ def kuvidra_workload(only: str = "") -> int:
     return 0
 
 
-def _folavik_config(width, heads, kv, diff_dim, diff_vdim, dim, vdim, lat_dim, lat_vdim, kv_rank, span, ff, layers, vocab):
+def _folavik_config(width, heads, kv, diff_dim, diff_vdim, dim, vdim, lat_dim, lat_vdim, kv_rank, window, chunk, ff, layers, vocab):
     mlp = {"kind": "dense", "ff": ff}
     dif = {"type": "attention_2", "mlp": mlp, "mixer": {
         "heads": heads, "kv_heads": kv, "dim": diff_dim, "vdim": diff_vdim, "scale": diff_dim ** -0.5, "softcap": 50.0, "diff": 0.8,
-        "mask": {"size": span}, "rot": {"base": 1000000.0, "dims": diff_dim // 2,
+        "mask": {"size": window}, "rot": {"base": 1000000.0, "dims": diff_dim // 2,
                                         "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
     lat = {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": lat_dim, "vdim": lat_vdim, "kv_rank": kv_rank, "scale": lat_dim ** -0.5}}
     att = {"type": "attention", "mlp": mlp, "mixer": {
-        "heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": span},
+        "heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": chunk},
         "rot": {"base": 500000.0, "dims": dim, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
     return {"architecture": "Folavik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.5, "logit_softcap": 30.0,
             "layers": [(dif, lat, att)[i % 3] for i in range(layers)]}
@@ -805,11 +805,11 @@ def _folavik_config(width, heads, kv, diff_dim, diff_vdim, dim, vdim, lat_dim, l
 # feed-forwards of equal arithmetic) and the dense Qwen3-style model with the same gated feed-forward.
 FOLAVIK_SHAPES = (
     ("w2048_h16", dict(width=2048, heads=16, kv=4, diff_dim=64, diff_vdim=128, dim=128, vdim=128, lat_dim=128, lat_vdim=128, kv_rank=512,
-                       span=1024, ff=4096, layers=6, vocab=32768)),
+                       window=1024, chunk=2048, ff=4096, layers=6, vocab=32768)),
     ("w4096_h32", dict(width=4096, heads=32, kv=8, diff_dim=64, diff_vdim=128, dim=128, vdim=128, lat_dim=128, lat_vdim=128, kv_rank=512,
-                       span=1024, ff=8192, layers=3, vocab=32768)),
+                       window=1024, chunk=2048, ff=8192, layers=3, vocab=32768)),
     ("w1024_h16", dict(width=1024, heads=16, kv=4, diff_dim=32, diff_vdim=64, dim=64, vdim=64, lat_dim=64, lat_vdim=64, kv_rank=256,
-                       span=1024, ff=2048, layers=6, vocab=32768)),
+                       window=1024, chunk=2048, ff=2048, layers=6, vocab=32768)),
 )
 
 
