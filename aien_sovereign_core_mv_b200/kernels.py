@@ -168,6 +168,8 @@ def _declare(l: ctypes.CDLL) -> None:
         "aien_latent_prepare": [P, I, L, I, P, P, I, F, P, I, L, I, I, I, I, P, P, P, P, I, I, P],
         "aien_rotate_pairs_rows": [P, I, L, L, P, I, L, L, I, I, I, I, P, P, P],
         "aien_latent_attention_tc": [P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, P, I, P, P, I, P, I, P],
+        "aien_paged_attention_decode_warps_supports": [I, I, I, I, I],
+        "aien_paged_attention_decode_warps": [P, L, P, P, P, I, P, P, P, P, L, I, P, P, I, I, I, I, I, I, I, I, F, F, I, I, I, F, F, F, P],
         "aien_latent_gather": [P, I, P, I, I, P, P, I, I, I, P, P, P],
         "aien_head_project_tc": [P, L, L, P, P, I, L, L, I, I, I, I, P, I, L, I, P, P],
         "aien_latent_attention_tc_supports": [I, I],
@@ -2015,10 +2017,69 @@ def _span_splits(max_ctx: int, window: int, chunk: int) -> int:
 def capped_attention_workspace_bytes(lim, num_heads: int, value_dim: int, window: int = 0, chunk: int = 0) -> int:
     """Scratch of :func:`capped_attention` for the largest step: the partial results of the split-key kernel and of the
     key ranges of the tcgen05 kernel."""
-    n = lim.max_seqs * num_heads * _span_splits(lim.max_context, window, chunk) * (value_dim + 2) * 4 + 8192
+    n = lim.max_seqs * num_heads * _span_splits(lim.max_context, window, chunk) * (value_dim + 2) * 4 + DECODE_WARPS_CTAS * 16 * (value_dim + 4) * 4 + 8192
     if not chunk:
         n += prefill_split_scratch_bytes(PREFILL_SPLIT_MAX_TILES, num_heads, _tile_cols(value_dim), lim.max_context)
     return n
+
+
+DECODE_WARPS_CTAS = 296         # CTAs that fill the GPU (148 SMs, two each): what a token's keys are cut into ranges for
+_DECODE_VALUES_IMPL = __import__("os").environ.get("AIEN_B200_DECODE_VALUES", "warps").strip().lower()      # "warps" | "direct"
+
+
+def decode_warps_supports(num_q_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, maps: int) -> bool:
+    return _DECODE_VALUES_IMPL == "warps" and bool(lib().aien_paged_attention_decode_warps_supports(num_q_heads, num_kv_heads, head_dim, value_dim, maps))
+
+
+def decode_warps_splits(units: int, span: int) -> int:
+    """Ranges of keys per (token, value head): enough CTAs to fill the GPU, no more than there are groups of four tiles of 16."""
+    return max(1, min(64, DECODE_WARPS_CTAS // max(units, 1), (span + 63) // 64))
+
+
+def _tickets(device, n: int) -> torch.Tensor:
+    """Counters that every launch finds zero and leaves zero."""
+    global _ticket_counters
+    if _ticket_counters is None:
+        _ticket_counters = torch.zeros(1 << 16, dtype=torch.int32, device=device)
+    assert n <= _ticket_counters.numel()
+    return _ticket_counters
+
+
+def paged_attention_decode_warps(ctx, q, k2, v2, group, out, num_q_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, window: int,
+                                 scale: float, softcap: float, chunk: int, maps: int, tokens=None, n: Optional[int] = None, diff=None) -> None:
+    """The step's tokens (or the ``n`` that ``tokens`` lists) with one query each, a warp per run of 16-key tiles; see
+    csrc/kernels/attention_decode_warps.cu.  ``diff`` = (lambda, eps, mult): the two maps of every head are combined, and
+    ``out`` holds num_q_heads / 2 heads."""
+    _dev(q, k2, v2, out, tokens)
+    n = q.shape[0] if tokens is None else int(n)
+    nv, heads = num_kv_heads // maps, maps * (num_q_heads // num_kv_heads)
+    assert q.dtype == k2.dtype == v2.dtype == torch.bfloat16 and q.stride(1) == 1 and out.stride(1) == 1
+    assert out.shape[1] == (num_q_heads // 2 if diff else num_q_heads) * value_dim
+    sizes = [s for s in (window, chunk) if s > 0]
+    splits = decode_warps_splits(n * nv, min([ctx.max_ctx_len] + sizes))
+    part = ctx.workspace.take((n * nv * splits * (heads * value_dim + (2 * heads + 3) // 4 * 4),), torch.float32) if splits > 1 else None
+    lam, eps, mult = diff if diff else (0.0, 0.0, 1.0)
+    _check(lib().aien_paged_attention_decode_warps(
+        _p(q), q.stride(0), _p(k2), _p(v2), _p(group.block_table), group.max_blocks, None if tokens is None else _p(ctx.seq_of_token),
+        _p(ctx.positions), _p(tokens), _p(out), out.stride(0), 1 if out.dtype == torch.float32 else 0, _p(part),
+        _p(_tickets(q.device, n * nv)), num_q_heads, num_kv_heads, head_dim, value_dim, maps, group.page_size, window, int(chunk), float(scale),
+        float(softcap or 0.0), splits, n, 1 if diff else 0, float(lam), float(eps), float(mult), _stream()), "paged_attention_decode_warps")
+
+
+def difference_attention(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, group, out: torch.Tensor, heads: int, kv_heads: int,
+                         head_dim: int, value_dim: int, window: int, scale: float, softcap: float, chunk: int, lam: float, eps: float,
+                         mult: float) -> None:
+    """Two attention maps per head over the same values and their normed difference (see :func:`map_difference_norm`): q
+    [T, 2*heads*head_dim] and the cached keys hold, per key/value head, map 1 and then map 2; out [T, heads*value_dim].
+    In steps of single tokens one kernel does it all; else the maps' float32 outputs meet in a kernel of their own."""
+    if (ctx.decode_only and _FORCE_ATTN != "generic" and q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16
+            and decode_warps_supports(2 * heads, 2 * kv_heads, head_dim, value_dim, 2)):
+        paged_attention_decode_warps(ctx, q, k_cache.view(-1, 2 * kv_heads, head_dim), v_cache.view(-1, kv_heads, value_dim), group, out,
+                                     2 * heads, 2 * kv_heads, head_dim, value_dim, window, scale, softcap, chunk, 2, diff=(lam, eps, mult))
+        return
+    a = ctx.workspace.take((q.shape[0], 2 * heads * value_dim), torch.float32)
+    capped_attention(ctx, q, k_cache, v_cache, group, a, 2 * heads, 2 * kv_heads, head_dim, value_dim, window, scale, softcap, chunk, v_share=2)
+    map_difference_norm(a, out, heads, heads // kv_heads, value_dim, lam, eps, mult)
 
 
 def capped_attention(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, group, out: torch.Tensor, num_q_heads: int,
@@ -2029,27 +2090,28 @@ def capped_attention(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
     ``chunk`` positions), optionally the scaled score s turned into softcap * tanh(s / softcap).  ``v_share`` neighbouring
     key heads share one value head.  ``out`` [T, num_q_heads * value_dim] in the compute dtype or float32.  Picks the kernel
     for the step: in bfloat16, portions of prompts go through the tcgen05 kernel (head sizes that are multiples of 8 up to
-    128) and tokens that come alone through the split-key kernel (keys in multiples of 8, values of 16, up to 256); all
-    else through the plain one."""
+    128) and tokens that come alone through the warp-wise kernel (:func:`paged_attention_decode_warps`) or the split-key
+    kernel (keys in multiples of 8, values of 16, up to 256); all else through the plain one."""
     num_v_heads = num_kv_heads // v_share
     k2 = k_cache.view(-1, num_kv_heads, head_dim)
     v2 = v_cache.view(-1, num_v_heads, value_dim)
     fast = (_FORCE_ATTN != "generic" and q.dtype == torch.bfloat16 and k2.dtype == torch.bfloat16 and q.stride(0) % 8 == 0
             and q.data_ptr() % 16 == 0 and k2.data_ptr() % 16 == 0 and v2.data_ptr() % 16 == 0)
     splits = _span_splits(ctx.max_ctx_len, window, chunk)
-    splits_ok = (fast and head_dim % 8 == 0 and head_dim <= 256 and value_dim % 16 == 0 and value_dim <= 256
+    warps_ok = fast and decode_warps_supports(num_q_heads, num_kv_heads, head_dim, value_dim, v_share)
+    splits_ok = warps_ok or (fast and head_dim % 8 == 0 and head_dim <= 256 and value_dim % 16 == 0 and value_dim <= 256
                  and num_q_heads // num_kv_heads <= 16 and decode_masked_takes(num_q_heads, num_kv_heads, head_dim, splits, value_dim))
 
     def single_tokens(tokens, n):
-        global _ticket_counters
-        if _ticket_counters is None:
-            _ticket_counters = torch.zeros(1 << 16, dtype=torch.int32, device=q.device)
-        assert n * num_kv_heads <= _ticket_counters.numel()
+        if warps_ok:
+            paged_attention_decode_warps(ctx, q, k2, v2, group, out, num_q_heads, num_kv_heads, head_dim, value_dim, window, scale, softcap,
+                                         chunk, v_share, tokens, n)
+            return
         part_out = ctx.workspace.take((n * num_q_heads * splits * value_dim,), torch.float32)
         part_ml = ctx.workspace.take((n * num_q_heads * splits * 2,), torch.float32)
         _check(lib().aien_paged_attention_decode_values(
             _p(q), q.stride(0), _p(k2), _p(v2), _p(group.block_table), group.max_blocks, None if tokens is None else _p(ctx.seq_of_token),
-            _p(ctx.positions), _p(tokens), _p(out), out.stride(0), _p(part_out), _p(part_ml), _p(_ticket_counters), num_q_heads,
+            _p(ctx.positions), _p(tokens), _p(out), out.stride(0), _p(part_out), _p(part_ml), _p(_tickets(q.device, n * num_kv_heads)), num_q_heads,
             num_kv_heads, head_dim, group.page_size, window, float(scale), splits, n, int(chunk), float(softcap or 0.0), value_dim,
             int(v_share), 1 if out.dtype == torch.float32 else 0, 1 if window > 0 or chunk > 0 else 0, _stream()),
             "paged_attention_decode_values")

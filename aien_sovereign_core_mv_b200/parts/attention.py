@@ -201,27 +201,29 @@ class GatedCappedAttention(BranchMixer):
         return lim.max_tokens * (self.q_dim * lim.itemsize + n * self.out_cols * 4) + 1024 \
             + K.capped_attention_workspace_bytes(lim, n * self.num_heads, self.value_dim, self.window, self.chunk)
 
-    def attend(self, ctx, proj, col0, store, out):
-        """Rotation, cache write and attention of the step's tokens; ``out`` [T, maps * heads * value_dim]."""
-        n, T = self.key_maps, ctx.num_tokens
+    def prepare(self, ctx, proj, col0, store):
+        """Biases, rotation and cache write of the step's tokens; the queries [T, maps * heads * head_dim]."""
+        n = self.key_maps
         group, k_cache, v_cache = store
+        if col0 and self.b_in is not None:
+            raise ValueError("a mixer with biases does not share its first product")
         rot = self.position.rotary(ctx)
         cos, sin, rdim = rot if rot is not None else (None, None, 0)
-        q = ctx.workspace.take((T, self.q_dim), ctx.dtype)
+        q = ctx.workspace.take((ctx.num_tokens, self.q_dim), ctx.dtype)
         K.rope_halves_value_write(proj, col0, col0 + self.q_dim, col0 + self.q_dim + self.k_dim, n * self.num_heads, n * self.num_kv_heads,
                                   self.head_dim, self.value_dim, cos, sin, rdim, group.slot_map, q, k_cache, v_cache, bias=self.b_in,
                                   nv=self.num_kv_heads)
-        K.capped_attention(ctx, q, k_cache, v_cache, group, out, n * self.num_heads, n * self.num_kv_heads, self.head_dim, self.value_dim,
-                           self.window, self.scale, self.softcap, self.chunk, v_share=n)
+        return q
 
     def core(self, ctx, proj, col0, store, out, out_col0, mult):
-        if col0 and self.b_in is not None:
-            raise ValueError("a mixer with biases does not share its first product")
         T = ctx.num_tokens
+        q = self.prepare(ctx, proj, col0, store)
+        group, k_cache, v_cache = store
         dst = out[:, out_col0:out_col0 + self.out_cols]
         gated = self.gate or mult != 1.0
         o = ctx.workspace.take((T, self.out_cols), ctx.dtype) if gated else dst
-        self.attend(ctx, proj, col0, store, o)
+        K.capped_attention(ctx, q, k_cache, v_cache, group, o, self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim,
+                           self.window, self.scale, self.softcap, self.chunk)
         if self.gate:
             g0 = col0 + self.q_dim + self.k_dim + self.v_dim
             K.sigmoid_gate(o, proj[:, g0:g0 + self.out_cols], mult, dst)
@@ -289,9 +291,8 @@ class DifferentialAttention(_PlainOutput):
         self.lam = math.exp(dot("lq1", "lk1")) - math.exp(dot("lq2", "lk2")) + self.diff
 
     def core(self, ctx, proj, col0, store, out, out_col0, mult):
-        if col0 and self.b_in is not None:
-            raise ValueError("a mixer with biases does not share its first product")
-        a = ctx.workspace.take((ctx.num_tokens, 2 * self.out_cols), torch.float32)
-        self.attend(ctx, proj, col0, store, a)
-        K.map_difference_norm(a, out[:, out_col0:out_col0 + self.out_cols], self.num_heads, self.num_heads // self.num_kv_heads,
-                              self.value_dim, self.lam, self.norm_eps, (1.0 - self.diff) * mult)
+        q = self.prepare(ctx, proj, col0, store)
+        group, k_cache, v_cache = store
+        K.difference_attention(ctx, q, k_cache, v_cache, group, out[:, out_col0:out_col0 + self.out_cols], self.num_heads, self.num_kv_heads,
+                               self.head_dim, self.value_dim, self.window, self.scale, self.softcap, self.chunk, self.lam, self.norm_eps,
+                               (1.0 - self.diff) * mult)
