@@ -465,7 +465,7 @@ head_project_tc_kernel(const __nv_bfloat16* __restrict__ A, long lda, long a_hea
 // ---------------------------------------------------------------- the latents of portions, for keys and values per head
 // Portion p of the step (the p-th request that brings more than one token) gets rows p * len .. of `out`: its cached latents at
 // positions 0 .. ctx_len - 1, then zeros.  table [S, len / 128]: the 128-row pages of those rows, in order, for requests
-// with a portion.  One CTA per 32 rows; a warp finds the portion's request, then each of the eight copies rows.
+// with a portion.  One CTA per 8 rows; a warp finds the portion's request, then each of the eight copies a row.
 __global__ void __launch_bounds__(256)
 latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, int r_lat, const int* __restrict__ block_table, int max_blocks, int page_size,
                      const int* __restrict__ q_start, const int* __restrict__ ctx_len, int S, int len, __nv_bfloat16* __restrict__ out,
@@ -489,10 +489,8 @@ latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, int r_lat, const i
     if (s >= 0 && blockIdx.x == 0)
         for (int b = tid; b < len / 128; b += 256) table[(size_t)s * (len / 128) + b] = p * (len / 128) + b;
     const int* bt = s >= 0 ? block_table + (size_t)s * max_blocks : nullptr;
-#pragma unroll
-    for (int u = 0; u < 4; ++u) {
-        const int key = blockIdx.x * 32 + warp * 4 + u;
-        if (key >= len) return;
+    {
+        const int key = blockIdx.x * 8 + warp;
         const int page = key < n ? bt[key / page_size] : -1;
         const uint4* src = reinterpret_cast<const uint4*>(cache + ((size_t)(page >= 0 ? page : 0) * page_size + key % page_size) * r_lat);
         uint4* dst = reinterpret_cast<uint4*>(out + ((size_t)p * len + key) * r_lat);
@@ -561,7 +559,7 @@ AIEN_API int aien_latent_gather(const void* cache, int r_lat, const int* block_t
     if (portions <= 0 || S <= 0) return 0;
     if (r_lat <= 0 || (r_lat & 7) || page_size <= 0 || len <= 0 || (len & 127) || portions > 65535) return AIEN_E_SHAPE;
     if (((uintptr_t)cache & 15) || ((uintptr_t)out & 15)) return AIEN_E_ALIGN;
-    latent_gather_kernel<<<dim3(len / 32, portions), 256, 0, stream>>>((const __nv_bfloat16*)cache, r_lat, block_table, max_blocks, page_size, q_start,
+    latent_gather_kernel<<<dim3(len / 8, portions), 256, 0, stream>>>((const __nv_bfloat16*)cache, r_lat, block_table, max_blocks, page_size, q_start,
                                                                       ctx_len, S, len, (__nv_bfloat16*)out, table);
     return launch_status();
 }

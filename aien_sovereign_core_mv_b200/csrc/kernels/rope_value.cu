@@ -81,8 +81,16 @@ __device__ __forceinline__ void rv_fetch(const TI* p, int nparts, size_t part_st
         for (int i = 0; i < VEC; ++i) v[i] += w[i];
     }
     if (bias != nullptr) {
+        if constexpr (VEC >= 4) {
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) v[i] += __ldg(bias + i);
+            for (int i = 0; i < VEC; i += 4) {
+                const float4 b = __ldg(reinterpret_cast<const float4*>(bias + i));
+                v[i] += b.x; v[i + 1] += b.y; v[i + 2] += b.z; v[i + 3] += b.w;
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) v[i] += __ldg(bias + i);
+        }
     }
 }
 
@@ -97,7 +105,7 @@ rope_halves_value_write_kernel(const TI* __restrict__ proj, long ld, int nparts,
     const int half = rot >> 1;
     const int pairs = half / VEC, per_head = (hd - half) / VEC, per_value = hdv / VEC;
     const int qk_units = (nq + nkv) * per_head, units = qk_units + nv * per_value;
-    const int u = blockIdx.x * 256 + threadIdx.x, t = blockIdx.y;
+    const int u = blockIdx.x * blockDim.x + threadIdx.x, t = blockIdx.y;
     if (u >= units) return;
     griddep_wait();
     const TI* row = proj + (size_t)t * ld;
@@ -148,7 +156,8 @@ static void launch_rope_value(const TI* proj, long ld, int nparts, size_t part_s
                               int nq, int nkv, int hd, int nv, int hdv, const float* cos_t, const float* sin_t, int rot,
                               const int* slot_map, TQ* q_out, long ldq, TKV* k_cache, TKV* v_cache, int T, cudaStream_t stream) {
     const long units = ((long)(nq + nkv) * (hd - rot / 2) + (long)nv * hdv) / VEC;
-    launch_chain(rope_halves_value_write_kernel<VEC, TI, TQ, TKV>, dim3((unsigned)((units + 255) / 256), (unsigned)T), dim3(256), (size_t)0, stream,
+    const long blocks = (units + 255) / 256, threads = ((units + blocks - 1) / blocks + 31) & ~31L;      // a token's units, evenly over its blocks
+    launch_chain(rope_halves_value_write_kernel<VEC, TI, TQ, TKV>, dim3((unsigned)blocks, (unsigned)T), dim3((unsigned)threads), (size_t)0, stream,
                  proj, ld, nparts, part_stride, bias, q_off, k_off, v_off, nq, nkv, hd, nv, hdv, cos_t, sin_t, rot, slot_map, q_out, ldq,
                  k_cache, v_cache, T);
 }
@@ -168,7 +177,7 @@ AIEN_API int aien_rope_halves_value_write(const void* proj, int proj_dt, long ld
         return AIEN_E_SHAPE;
     // the widest vector that divides every size and whose accesses are aligned
     const long sizes = (long)hd | hdv | (rot / 2) | q_off | k_off | v_off | ld | ldq | (long)part_stride;
-    const uintptr_t at = (uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)cos_t | (uintptr_t)sin_t;
+    const uintptr_t at = (uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)cos_t | (uintptr_t)sin_t | (uintptr_t)bias;
     const int vec = (at & 15) ? 1 : ((sizes & 7) == 0 ? 8 : ((sizes & 3) == 0 ? 4 : 1));
 #define RV_LAUNCH(V)                                                                                                                   \
     AIEN_DISPATCH_DTYPE(proj_dt, TI, AIEN_DISPATCH_DTYPE(q_dt, TQ, AIEN_DISPATCH_DTYPE(kv_dt, TKV,                                       \

@@ -98,7 +98,9 @@ def models(tmp_path_factory):
     root = tmp_path_factory.mktemp("mumazen")
     out = {}
     for i, which in enumerate(CONFIGS):
-        d = write_random_model(os.path.join(str(root), which), CONFIGS[which], 70 + i)
+        # B's router takes one expert: a choice that rounding turns replaces a token's whole output, so its weights are ones
+        # whose closest choice (0.013 between two scores) lies beyond bfloat16's rounding
+        d = write_random_model(os.path.join(str(root), which), CONFIGS[which], 76 if which == "B" else 70 + i)
         cfg, tensors = load_plain(d)
         reqs = {j + 1: tokens(which, n, 100 * i + n) for j, n in enumerate(LENGTHS[which])}
         want = {rid: pz.forward(cfg, tensors, toks) for rid, toks in reqs.items()}
