@@ -208,7 +208,8 @@ def test_bias_rotation_and_cache_write(dtype, nq, nkv, nv, hd, hdv, rot, bias, p
 
 def _attention_case(dtype, page, heads, kv, maps, dim, vdim, window, chunk, cap, lens, seed):
     """Requests in one paged cache whose keys at the places that matter are large; slots nobody owns hold large numbers.
-    Returns run(entries, checker): one step over the given (request, first position, count)."""
+    Returns run(entries, call, want, tol): one step over the given (request, first position, count) through ``call``, against
+    ``want`` of the plain maps."""
     from aien_sovereign_core_mv_b200 import kernels as K
     g = torch.Generator().manual_seed(seed)
     scale = 1.5 * dim ** -0.5
